@@ -15,8 +15,10 @@ LIB_PATH = os.environ.get("FUSEKIT_CUDA_LIB") or os.path.join(_HERE, "libfusekit
 (TASK_STEP_INIT, TASK_EMBED_LOOKUP_DECODE, TASK_RMSNORM_QKV, TASK_QK_NORM_ROPE_STORE, TASK_SDPA_DECODE,
  TASK_LINEAR_RESIDUAL, TASK_RMSNORM_GATEUP_ACT, TASK_FINAL_RMSNORM_LM_HEAD, TASK_ARGMAX_FINALIZE,
  TASK_ALLREDUCE, TASK_RESIDUAL_ADD, TASK_RMSNORM_ROWS, TASK_ROPE_STORE_ROWS, TASK_ARGMAX_ROWS, TASK_KV_STORE_QUANT,
- TASK_SDPA_DECODE_QUANT) = range(16)
+ TASK_SDPA_DECODE_QUANT, TASK_EMBED_ROWS, TASK_RESIDUAL_NORM_ROWS, TASK_LINEAR_ROWS, TASK_QK_NORM_STORE_ROWS, TASK_ATTENTION_ROWS,
+ TASK_MOE_ROUTE_ROWS, TASK_NORM_LINEAR, TASK_ATTENTION_DECODE, TASK_MOE_UP, TASK_MOE_DOWN, TASK_ARGMAX_ROW) = range(27)
 ACT_SWIGLU, ACT_GEGLU_TANH = 0, 1
+ACT_NONE, ACT_RELU_SQUARED = 0, 2
 
 
 class RoleBinding(C.Structure):
@@ -65,7 +67,7 @@ def lib():
         "fk_memset": [u64, u64, i32, sz], "fk_sync": [u64], "fk_kv_cache_alloc": [u64, i32, i32, i32, P(u64), P(u64)],
         "fk_weight_alloc": [u64, i64, i64, i32, P(u64)], "fk_weight_upload_rows": [u64, u64, i64, i64, vp, vp, vp],
         "fk_weight_synth_rows": [u64, u64, i64, i64, u64, f32, i64, i64, i64], "fk_weight_finalize": [u64, u64],
-        "fk_weight_set_rows": [u64, u64, i32, i32, i32], "fk_weight_pair": [u64, u64, u64, P(u64)],
+        "fk_weight_set_rows": [u64, u64, i32, i32, i32], "fk_weight_pair": [u64, u64, u64, P(u64)], "fk_weight_keep_rows": [u64, u64],
         "fk_weight_dequant": [u64, u64, i64, i64, vp], "fk_weight_nbytes": [u64, u64, P(u64)],
         "fk_synth_normal_bf16": [u64, u64, u64, u64, u64, f32, f32],
         "fk_launch": [u64, P(Task)], "fk_launch_batch": [u64, P(Task), i32], "fk_smoke": [u64, vp, vp, vp, i32],

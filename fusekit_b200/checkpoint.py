@@ -26,7 +26,7 @@ import struct
 
 import numpy as np
 
-from .model_spec import ModelSpec
+from .model_spec import AttentionSpec, LayeredSpec, LayerSpec, LoopSpec, ModelSpec, MoeSpec
 
 _DT = {"U32": (np.uint32, 4), "I32": (np.int32, 4), "BF16": (np.uint16, 2), "F16": (np.float16, 2), "F32": (np.float32, 4),
        "U8": (np.uint8, 1), "I64": (np.int64, 8), "U16": (np.uint16, 2)}
@@ -152,6 +152,33 @@ def spec_from_config(cfg: dict, name: str = "checkpoint") -> ModelSpec:
                      window=window, global_every=every)
 
 
+LAYERED_ARCHITECTURES = ("Fatulix",)
+
+
+def layered_spec_from_config(cfg: dict, name: str = "checkpoint") -> LayeredSpec:
+    """config.json of a layered decoder: ``architecture``, ``width``, ``vocab``, ``norm.eps``, ``layers`` (each ``type``, ``mixer``,
+    ``mlp`` or null) and an optional ``loop``.  Anything this build has no mechanism for is refused by name."""
+    arch = cfg.get("architecture")
+    if arch not in LAYERED_ARCHITECTURES:
+        raise ValueError(f"architecture {arch!r} has no decode path here ({', '.join(LAYERED_ARCHITECTURES)})")
+    layers = []
+    for i, e in enumerate(cfg["layers"]):
+        if e["type"] != "attention":
+            raise ValueError(f"layer {i}: mixer type {e['type']!r} is not supported (attention)")
+        m, f = e["mixer"], e.get("mlp")
+        mixer = AttentionSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]), float(m["diff"]))
+        mlp = None
+        if f is not None:
+            if f["kind"] != "moe":
+                raise ValueError(f"layer {i}: feed-forward kind {f['kind']!r} is not supported (moe)")
+            shared = f.get("shared")
+            mlp = MoeSpec(int(f["router"]["experts"]), int(f["router"]["top"]), int(f["expert"]["ff"]), int(shared["ff"]) if shared else 0)
+        layers.append(LayerSpec(mixer, mlp))
+    lp = cfg.get("loop")
+    loop = LoopSpec(int(lp["start"]), int(lp["stop"]), int(lp["times"])) if lp else None
+    return LayeredSpec(name=name, arch=arch, hidden=int(cfg["width"]), vocab=int(cfg["vocab"]), layers=tuple(layers), eps=float(cfg["norm"]["eps"]), loop=loop)
+
+
 _W = {"q_proj": "self_attn.q_proj", "k_proj": "self_attn.k_proj", "v_proj": "self_attn.v_proj", "o_proj": "self_attn.o_proj",
       "gate_proj": "mlp.gate_proj", "up_proj": "mlp.up_proj", "down_proj": "mlp.down_proj"}
 _V = {"input_norm": "input_layernorm.weight", "post_attention_norm": "post_attention_layernorm.weight",
@@ -160,16 +187,16 @@ _V = {"input_norm": "input_layernorm.weight", "post_attention_norm": "post_atten
       "q_bias": "self_attn.q_proj.bias", "k_bias": "self_attn.k_proj.bias", "v_bias": "self_attn.v_proj.bias"}
 
 
-class Checkpoint:
-    """A model directory: config.json plus one or more safetensors shards."""
+class TensorFiles:
+    """config.json plus one or more safetensors shards of a model directory: tensors by name."""
 
     def __init__(self, path: str):
         self.dir = path
         with open(os.path.join(path, "config.json")) as f:
             self.config = json.load(f)
-        self.spec = spec_from_config(self.config, os.path.basename(os.path.normpath(path)))
         self.files: list[SafetensorsFile] = []
         self.where: dict[str, SafetensorsFile] = {}
+        self.lossy: list[str] = []                                  # tensors converted from fp16 / fp32 to bf16
         idx = os.path.join(path, "model.safetensors.index.json")
         shards = sorted(f for f in os.listdir(path) if f.endswith(".safetensors"))
         if os.path.exists(idx):
@@ -182,16 +209,6 @@ class Checkpoint:
             self.files.append(sf)
             for n in sf.names():
                 self.where[n] = sf
-        emb = [n for n in self.where if n.endswith("embed_tokens.weight")]
-        if len(emb) != 1:
-            raise ValueError(f"{path}: expected one embed_tokens.weight, found {emb}")
-        self.prefix = emb[0][: -len("embed_tokens.weight")]          # "model." or "language_model.model."
-        self.head_prefix = self.prefix[: -len("model.")] if self.prefix.endswith("model.") else ""
-        self.tied = (self.head_prefix + "lm_head.weight") not in self.where
-        self.lossy: list[str] = []                                  # tensors converted from fp16 / fp32 to bf16
-        self.embed_bits = self.spec.bits if (self.prefix + "embed_tokens.scales") in self.where else 16
-        # Gemma-family RMSNorm multiplies by (1 + weight); the runtime takes the effective weight
-        self.norm_offset = 1.0 if self.spec.arch == "gemma3" else 0.0
 
     def has(self, name: str) -> bool:
         return name in self.where
@@ -214,6 +231,27 @@ class Checkpoint:
                 self.lossy.append(name)
             return f16_to_bf16_bits(a) if dt == "F16" else f32_to_bf16_bits(a)
         raise ValueError(f"{name}: dtype {dt} is not a floating type")
+
+    def close(self):
+        for f in self.files:
+            f.close()
+
+
+class Checkpoint(TensorFiles):
+    """An mlx-lm style model directory."""
+
+    def __init__(self, path: str):
+        super().__init__(path)
+        self.spec = spec_from_config(self.config, os.path.basename(os.path.normpath(path)))
+        emb = [n for n in self.where if n.endswith("embed_tokens.weight")]
+        if len(emb) != 1:
+            raise ValueError(f"{path}: expected one embed_tokens.weight, found {emb}")
+        self.prefix = emb[0][: -len("embed_tokens.weight")]          # "model." or "language_model.model."
+        self.head_prefix = self.prefix[: -len("model.")] if self.prefix.endswith("model.") else ""
+        self.tied = (self.head_prefix + "lm_head.weight") not in self.where
+        self.embed_bits = self.spec.bits if (self.prefix + "embed_tokens.scales") in self.where else 16
+        # Gemma-family RMSNorm multiplies by (1 + weight); the runtime takes the effective weight
+        self.norm_offset = 1.0 if self.spec.arch == "gemma3" else 0.0
 
     def _linear_base(self, leaf: str, layer: int) -> str:
         if leaf == "lm_head":
@@ -272,13 +310,36 @@ class Checkpoint:
         return {"bits": self.embed_bits, "packed": self.raw(base + ".weight"), "scales": self.bf16(base + ".scales"),
                 "biases": self.bf16(base + ".biases")}
 
-    def close(self):
-        for f in self.files:
-            f.close()
+
+class LayeredCheckpoint(TensorFiles):
+    """A model directory of a layered decoder: tensors ``embed``, ``head``, ``final.norm`` and ``l<i>.<name>``, bf16."""
+
+    def __init__(self, path: str):
+        super().__init__(path)
+        self.spec = layered_spec_from_config(self.config, os.path.basename(os.path.normpath(path)))
+
+    def provider(self):
+        """For LayeredEngine.load_from: bf16 bits of a tensor, its shape checked against the configuration."""
+        def prov(name, shape):
+            a = self.bf16(name)
+            if tuple(a.shape) != tuple(shape):
+                raise ValueError(f"{self.dir}: tensor {name} has shape {list(a.shape)}, the configuration says {list(shape)}")
+            return a
+        return prov
 
 
 def load_engine(path: str, capacity: int, device: int = 0, tp_rank: int = 0, tp_size: int = 1, **kw):
     """Open a checkpoint directory and return (engine, checkpoint) with all tensors resident on the GPU."""
+    with open(os.path.join(path, "config.json")) as f:
+        layered = "architecture" in json.load(f)
+    if layered:
+        from .layered import LayeredEngine
+        if tp_size != 1:
+            raise ValueError("layered decoders run on one GPU")
+        lck = LayeredCheckpoint(path)
+        leng = LayeredEngine(lck.spec, capacity, device=device, **kw)
+        leng.load_from(lck.provider())
+        return leng, lck
     from .runtime import DecodeEngine
     ck = Checkpoint(path)
     eng = DecodeEngine(ck.spec, capacity, device=device, tp_rank=tp_rank, tp_size=tp_size, **kw)

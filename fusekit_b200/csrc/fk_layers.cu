@@ -1,0 +1,209 @@
+// Host side of the layered decoders' kernels: argument checks and launches, one case per task kind.
+#include "fk_layers.h"
+#include "fk_layers.cuh"
+#include <stdarg.h>
+#include <stdio.h>
+#include <string.h>
+
+bool fkl_owns(int kind) { return kind >= FK_TASK_EMBED_ROWS && kind <= FK_TASK_ARGMAX_ROW; }
+
+template <typename K> static cudaError_t big_smem(K kern) {
+    cudaFuncAttributes fa; cudaError_t e = cudaFuncGetAttributes(&fa, kern);
+    if (e != cudaSuccess) return e;
+    return cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024 - (int)fa.sharedSizeBytes);
+}
+template <typename... KA, typename... A>
+static cudaError_t launch(FklEnv &c, void (*kern)(KA...), dim3 grid, dim3 block, size_t smem, A... args) {
+    cudaLaunchConfig_t cfg; memset(&cfg, 0, sizeof cfg);
+    cfg.gridDim = grid; cfg.blockDim = block; cfg.dynamicSmemBytes = smem; cfg.stream = c.stream;
+    cudaLaunchAttribute at[1];
+    at[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    at[0].val.programmaticStreamSerializationAllowed = 1;
+    cfg.attrs = at; cfg.numAttrs = c.pdl ? 1 : 0;
+    ++*c.launches;
+    return cudaLaunchKernelEx(&cfg, kern, KA(args)...);
+}
+// CALL with VPL = values per lane of the attention kernel (a power of two covering vpad)
+#define VPL_SWITCH(vpad, CALL)                                   \
+    do {                                                         \
+        if ((vpad) <= 32) { constexpr int VPL = 1; CALL; }       \
+        else if ((vpad) <= 64) { constexpr int VPL = 2; CALL; }  \
+        else if ((vpad) <= 128) { constexpr int VPL = 4; CALL; } \
+        else if ((vpad) <= 256) { constexpr int VPL = 8; CALL; } \
+        else { constexpr int VPL = 16; CALL; }                   \
+    } while (0)
+
+cudaError_t fkl_init() {
+    cudaError_t e = cudaSuccess, r;
+#define TRY(x) do { r = (x); if (e == cudaSuccess) e = r; } while (0)
+#define ATT(VPL) TRY(big_smem(k_attention<uint16_t, float, VPL, true>)); TRY(big_smem(k_attention<float, float, VPL, true>)); \
+                 TRY(big_smem(k_attention<uint16_t, uint16_t, VPL, false>)); TRY(big_smem(k_attention<float, float, VPL, false>))
+    ATT(1); ATT(2); ATT(4); ATT(8); ATT(16);
+    TRY(big_smem(k_residual_norm_rows<uint16_t>)); TRY(big_smem(k_residual_norm_rows<float>));
+    TRY(big_smem(k_gemv<FKL_GV_LINEAR>)); TRY(big_smem(k_gemv<FKL_GV_MOE_UP>)); TRY(big_smem(k_gemv<FKL_GV_MOE_DOWN>));
+#undef ATT
+#undef TRY
+    return e;
+}
+
+static fk_status bad(char *err, size_t cap, const char *fmt, ...) {
+    va_list ap; va_start(ap, fmt); vsnprintf(err, cap, fmt, ap); va_end(ap);
+    return FK_ERR_VALUE;
+}
+static int round_up(int v, int m) { return (v + m - 1) / m * m; }
+
+// Blocks and K split of a matrix-vector product: as few warps per row group as reach every SM twice with one group each.
+static cudaError_t launch_gemv(FklEnv &c, int mode, GemvArgs &a) {
+    const int groups = (a.n + FKL_GV_R - 1) / FKL_GV_R, slots = c.sm_count * 2;
+    int ks = 1;
+    while (ks < FKL_GV_WARPS && ks * 2 <= a.nchunks && (long long)groups * ks < (long long)slots * FKL_GV_WARPS) ks *= 2;
+    a.kslices = ks;
+    const int spb = FKL_GV_WARPS / ks, blocks = (groups + spb - 1) / spb, grid = blocks < slots ? blocks : slots;
+    const size_t smem = gv_smem_bytes(a.nchunks);
+    const dim3 g(grid), b(FKL_GV_WARPS * 32);
+    if (mode == FKL_GV_LINEAR) return launch(c, k_gemv<FKL_GV_LINEAR>, g, b, smem, c.state, a);
+    if (mode == FKL_GV_MOE_UP) return launch(c, k_gemv<FKL_GV_MOE_UP>, g, b, smem, c.state, a);
+    return launch(c, k_gemv<FKL_GV_MOE_DOWN>, g, b, smem, c.state, a);
+}
+static bool gv_fits(int nchunks) { return nchunks > 0 && gv_smem_bytes(nchunks) <= 200 * 1024; }
+
+fk_status fkl_run(FklEnv &c, const fk_task &t, char *err, size_t ecap) {
+    const uint64_t *b = t.buf; const int32_t *i = t.iarg; const float *f = t.farg;
+    cudaError_t e = cudaSuccess;
+    FklWeight w, w2;
+    switch (t.kind) {
+    case FK_TASK_EMBED_ROWS: {
+        if (!b[0] || !b[1] || i[0] <= 0 || i[1] <= 0 || i[2] <= 0 || (!b[2] && i[1] > FK_MAX_ROWS)) return bad(err, ecap, "embed_rows: bad arguments");
+        EmbedRowsArgs a{(const uint16_t *)b[0], (float *)b[1], (const uint32_t *)b[2], i[0], i[2]};
+        e = launch(c, k_embed_rows, dim3(i[1]), dim3(256), 0, c.state, a);
+        break;
+    }
+    case FK_TASK_RESIDUAL_NORM_ROWS: {
+        if (!b[0] || !b[5] || !b[6] || i[0] <= 0 || i[1] <= 0 || i[3] < i[0] || ((b[1] || b[8]) && (!b[2] || i[5] < i[0])) || (b[8] && (!b[9] || !b[10] || i[4] <= 0)))
+            return bad(err, ecap, "residual_norm_rows: bad arguments");
+        if ((size_t)i[0] * 4 > 200 * 1024) return bad(err, ecap, "residual_norm_rows: width above 51200");
+        ResNormArgs a{(const float *)b[0], (const void *)b[1], (const uint16_t *)b[2], (const float *)b[3], (float *)b[4], (const uint16_t *)b[5], (void *)b[6],
+                      (const uint32_t *)b[7], (const void *)b[8], (const int *)b[9], (const float *)b[10], i[0], i[3], i[4], i[5], f[0]};
+        const dim3 g(i[1]), blk(i[0] >= 2048 ? 512 : 256);
+        e = i[2] ? launch(c, k_residual_norm_rows<float>, g, blk, (size_t)i[0] * 4, (const FkState *)c.state, a)
+                 : launch(c, k_residual_norm_rows<uint16_t>, g, blk, (size_t)i[0] * 4, (const FkState *)c.state, a);
+        break;
+    }
+    case FK_TASK_LINEAR_ROWS: {
+        const int M = i[0], row0 = i[1], N = i[2], ldx = i[3], ldy = i[4], f32 = i[5], act = i[6] & 255, outf = (i[6] >> 8) & 1, E = i[7];
+        if (!c.weight(c.owner, b[1], &w)) return bad(err, ecap, "linear_rows: weight missing or not kept as rows");
+        if (!b[0] || !b[2] || M <= 0 || N <= 0 || row0 < 0 || ldx < w.k || ldx % 8 || ldy < N || (b[3] && E <= 0)) return bad(err, ecap, "linear_rows: bad arguments");
+        if (b[3] ? w.n != (long long)E * N : row0 + N > w.n) return bad(err, ecap, "linear_rows: shape mismatch");
+        LinRowsArgs a{(const void *)b[0], w.rows + (size_t)row0 * w.k, (void *)b[2], (const int *)b[3], M, N, (int)w.k, ldx, (int)w.k, ldy, act, outf};
+        const dim3 g((N + 63) / 64, (M + 63) / 64, b[3] ? E : 1);
+        if (g.y > 65535 || g.z > 65535) return bad(err, ecap, "linear_rows: too many rows");
+        e = f32 ? launch(c, k_linear_rows<float>, g, dim3(256), 0, (const FkState *)c.state, a) : launch(c, k_linear_rows<uint16_t>, g, dim3(256), 0, (const FkState *)c.state, a);
+        break;
+    }
+    case FK_TASK_QK_NORM_STORE_ROWS: {
+        QkStoreArgs a{(const void *)b[0], (const uint16_t *)b[1], (const uint16_t *)b[2], (void *)b[3], (void *)b[4], (void *)b[5],
+                      i[0], i[1], i[6] >> 8, i[2], i[3], round_up(i[2], 8), round_up(i[3], 8), i[4], i[5], i[7], f[0]};
+        for (int q = 0; q < 6; ++q) if (!b[q]) return bad(err, ecap, "qk_norm_store_rows: missing buffer %d", q);
+        if (a.H <= 0 || a.G <= 0 || a.H % a.G || a.dim <= 0 || a.vdim <= 0 || a.cap <= 0 || a.rows <= 0 || (a.maps != 1 && a.maps != 2) ||
+            a.ld < (a.H + a.G) * a.maps * a.dim + a.G * a.vdim) return bad(err, ecap, "qk_norm_store_rows: bad arguments");
+        const dim3 g(a.rows, ((a.H + a.G) * a.maps + a.G + 3) / 4);
+        e = (i[6] & 1) ? launch(c, k_qk_norm_store_rows<float>, g, dim3(128), 0, c.state, a) : launch(c, k_qk_norm_store_rows<uint16_t>, g, dim3(128), 0, c.state, a);
+        break;
+    }
+    case FK_TASK_ATTENTION_ROWS: case FK_TASK_ATTENTION_DECODE: {
+        const bool dec = t.kind == FK_TASK_ATTENTION_DECODE;
+        AttnArgs a; memset(&a, 0, sizeof a);
+        a.H = i[0]; a.G = i[1]; a.dim = i[2]; a.vdim = i[3]; a.cap = i[4]; a.maps = i[6] >> 8;
+        const int f32 = i[6] & 1, rows = dec ? 1 : i[5];
+        a.scale = f[0]; a.lambda = f[1]; a.diff = f[2]; a.eps = f[3];
+        if (a.H <= 0 || a.G <= 0 || a.H % a.G || a.dim <= 0 || a.vdim <= 0 || a.vdim > 512 || a.cap <= 0 || rows <= 0 || rows > 65535 || (a.maps != 1 && a.maps != 2))
+            return bad(err, ecap, "attention: bad arguments (value size up to 512)");
+        a.dpad = round_up(a.dim, 8); a.vpad = round_up(a.vdim, 8);
+        a.tiles = (a.H / a.G * a.maps + FKL_ATT_ROWS - 1) / FKL_ATT_ROWS; a.splits = 1;
+        const size_t smem = attn_smem_floats(a.dpad, a.vpad) * 4;
+        if (smem > 220 * 1024) return bad(err, ecap, "attention: head size too large");
+        if (dec) {
+            for (int q = 0; q < 8; ++q) if (!b[q]) return bad(err, ecap, "attention_decode: missing buffer %d", q);
+            a.qkv = (const float *)b[0]; a.qn = (const uint16_t *)b[1]; a.kn = (const uint16_t *)b[2]; a.ck = (void *)b[3]; a.cv = (void *)b[4]; a.out = (void *)b[5];
+            a.part = (float *)b[6]; a.counter = (uint32_t *)b[7];
+            a.gate = i[5] ? (const void *)(a.qkv + (a.H + a.G) * a.maps * a.dim + a.G * a.vdim) : nullptr;
+            a.splits = i[7];
+            if (a.splits <= 0 || a.splits > 8 * a.vpad || a.splits > 256) return bad(err, ecap, "attention_decode: bad number of key splits");
+            const dim3 g(a.splits, a.G * a.tiles, 1), blk(FKL_ATT_WARPS * 32);
+            if (f32) VPL_SWITCH(a.vpad, e = launch(c, (k_attention<float, float, VPL, true>), g, blk, smem, c.state, a));
+            else VPL_SWITCH(a.vpad, e = launch(c, (k_attention<uint16_t, float, VPL, true>), g, blk, smem, c.state, a));
+        } else {
+            for (int q = 0; q < 4; ++q) if (!b[q]) return bad(err, ecap, "attention_rows: missing buffer %d", q);
+            a.q = (const void *)b[0]; a.ck = (void *)b[1]; a.cv = (void *)b[2]; a.out = (void *)b[3]; a.gate = (const void *)b[4];
+            a.ldo = round_up(a.H * a.vdim, 64); a.ldg = i[7];
+            const dim3 g(1, a.G * a.tiles, rows), blk(FKL_ATT_WARPS * 32);
+            if (f32) VPL_SWITCH(a.vpad, e = launch(c, (k_attention<float, float, VPL, false>), g, blk, smem, c.state, a));
+            else VPL_SWITCH(a.vpad, e = launch(c, (k_attention<uint16_t, uint16_t, VPL, false>), g, blk, smem, c.state, a));
+        }
+        break;
+    }
+    case FK_TASK_MOE_ROUTE_ROWS: {
+        RouteArgs a; memset(&a, 0, sizeof a);
+        for (int q = 0; q < 9; ++q) if (!b[q]) return bad(err, ecap, "moe_route_rows: missing buffer %d", q);
+        a.logits = (const float *)b[0]; a.h = (const void *)b[1]; a.weight = (float *)b[2]; a.expert = (int *)b[3]; a.rank = (int *)b[4]; a.count = (int *)b[5];
+        a.slot = (int *)b[6]; a.offsets = (int *)b[7]; a.hp = (void *)b[8];
+        a.rows = i[0]; a.E = i[1]; a.top = i[2]; a.ldl = i[3]; a.ld = i[4];
+        if (a.rows <= 0 || a.E <= 0 || a.E > FKL_MAX_EXPERTS || a.top <= 0 || a.top > FKL_MAX_TOP || a.top > a.E || a.ldl < a.E || a.ld <= 0 || a.ld % 8)
+            return bad(err, ecap, "moe_route_rows: bad arguments (at most %d experts, %d chosen)", FKL_MAX_EXPERTS, FKL_MAX_TOP);
+        e = cudaMemsetAsync(a.count, 0, (size_t)a.E * 4, c.stream);
+        if (e == cudaSuccess) e = launch(c, k_moe_route, dim3((a.rows + 3) / 4), dim3(128), 0, (const FkState *)c.state, a);
+        if (e == cudaSuccess) e = i[5] ? launch(c, k_moe_gather<float>, dim3(a.rows * a.top), dim3(256), 0, (const FkState *)c.state, a)
+                                       : launch(c, k_moe_gather<uint16_t>, dim3(a.rows * a.top), dim3(256), 0, (const FkState *)c.state, a);
+        break;
+    }
+    case FK_TASK_NORM_LINEAR: {
+        if (!c.weight(c.owner, b[6], &w)) return bad(err, ecap, "norm_linear: weight missing or not kept as rows");
+        GemvArgs a; memset(&a, 0, sizeof a);
+        a.x = (const float *)b[0]; a.pend = (const float *)b[1]; a.post_w = (const uint16_t *)b[2]; a.add = (const float *)b[3]; a.x_out = (float *)b[4];
+        a.norm_w = (const uint16_t *)b[5]; a.y = (float *)b[7]; a.h_out = (float *)b[8]; a.amax = (unsigned long long *)b[9]; a.counter = (uint32_t *)b[10];
+        a.w = w.rows; a.k = i[0]; a.n = i[1]; a.act = i[2]; a.act_row0 = i[3]; a.ldk = (int)w.k; a.eps = f[0]; a.history = c.history;
+        if (!a.x || !a.y || a.k <= 0 || a.k > w.k || a.n <= 0 || a.n > w.n || (a.pend && (!a.post_w || !a.norm_w)) || (a.amax && !a.counter) ||
+            (a.x_out && a.x_out == a.x)) return bad(err, ecap, "norm_linear: bad arguments");
+        a.nchunks = gv_chunks(a.ldk);
+        if (!gv_fits(a.nchunks)) return bad(err, ecap, "norm_linear: input of %d values is too long", a.k);
+        e = launch_gemv(c, FKL_GV_LINEAR, a);
+        break;
+    }
+    case FK_TASK_MOE_UP: {
+        if (!c.weight(c.owner, b[2], &w)) return bad(err, ecap, "moe_up: weight missing or not kept as rows");
+        GemvArgs a; memset(&a, 0, sizeof a);
+        a.logits = (const float *)b[0]; a.x = (const float *)b[1]; a.w = w.rows; a.y = (float *)b[3]; a.sel = (int *)b[4]; a.wts = (float *)b[5];
+        a.k = i[0]; a.E = i[1]; a.top = i[2]; a.ff = i[3]; a.act = i[4]; a.ldk = (int)w.k; a.n = a.top * a.ff;
+        if (!a.logits || !a.x || !a.y || !a.sel || !a.wts || a.k <= 0 || a.k > w.k || a.E <= 0 || a.E > FKL_MAX_EXPERTS || a.top <= 0 || a.top > FKL_MAX_TOP || a.top > a.E ||
+            a.ff <= 0 || w.n != (long long)a.E * a.ff) return bad(err, ecap, "moe_up: bad arguments");
+        a.nchunks = gv_chunks(a.ldk);
+        if (!gv_fits(a.nchunks)) return bad(err, ecap, "moe_up: input of %d values is too long", a.k);
+        e = launch_gemv(c, FKL_GV_MOE_UP, a);
+        break;
+    }
+    case FK_TASK_MOE_DOWN: {
+        if (!c.weight(c.owner, b[3], &w)) return bad(err, ecap, "moe_down: weight missing or not kept as rows");
+        GemvArgs a; memset(&a, 0, sizeof a);
+        a.x = (const float *)b[0]; a.sel = (int *)b[1]; a.wts = (float *)b[2]; a.w = w.rows; a.sact = (const float *)b[4]; a.y = (float *)b[6];
+        a.n = i[0]; a.E = i[1]; a.top = i[2]; a.ff = i[3]; a.ffs = i[4]; a.ldff = (int)w.k;
+        if (!a.x || !a.sel || !a.wts || !a.y || a.n <= 0 || a.E <= 0 || a.top <= 0 || a.top > FKL_MAX_TOP || a.ff <= 0 || a.ff > a.ldff || w.n != (long long)a.E * a.n)
+            return bad(err, ecap, "moe_down: bad arguments");
+        a.nchunks = a.top * gv_chunks(a.ldff);
+        if (a.ffs > 0) {
+            if (!c.weight(c.owner, b[5], &w2) || w2.n != a.n || w2.k < a.ffs || !a.sact) return bad(err, ecap, "moe_down: shared weight missing or of another shape");
+            a.w2 = w2.rows; a.ldffs = (int)w2.k; a.nchunks += gv_chunks(a.ldffs);
+        }
+        if (!gv_fits(a.nchunks)) return bad(err, ecap, "moe_down: the chosen experts' activations do not fit in shared memory");
+        e = launch_gemv(c, FKL_GV_MOE_DOWN, a);
+        break;
+    }
+    case FK_TASK_ARGMAX_ROW: {
+        if (!b[0] || i[0] <= 0 || i[1] < 0) return bad(err, ecap, "argmax_row: bad arguments");
+        e = launch(c, k_argmax_row_f32, dim3(1), dim3(1024), 0, c.state, (const float *)b[0], c.history, i[0], i[1]);
+        break;
+    }
+    default: return bad(err, ecap, "unknown task kind %d", t.kind);
+    }
+    if (e != cudaSuccess) { snprintf(err, ecap, "launch of task kind %d failed: %s", t.kind, cudaGetErrorString(e)); return FK_ERR_CUDA; }
+    return FK_OK;
+}

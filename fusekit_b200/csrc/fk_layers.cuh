@@ -1,0 +1,646 @@
+// Kernels of the layered decoders: a residual stream in fp32, norms before and after every sublayer, (differential)
+// attention with per-head q/k norm and an output gate, mixture-of-experts feed-forward with a shared expert.
+//
+// Two families.  The *row* kernels work on M consecutive positions (prompt portions); activations between the matrix
+// products are T = bf16 or float, everything a norm, a router, a softmax or the residual touches is fp32.  The *decode*
+// kernels work on one position with fp32 activations throughout: they are bound by the weights they stream, so the wider
+// activations cost nothing.  Weights are bf16 rows [n, k] with k padded by zeros to a multiple of 64, so no product has a
+// ragged K; activation buffers carry the same zero padding.
+#pragma once
+#include "fk_common.cuh"
+#include <math.h>
+
+#define FKL_MAX_EXPERTS 1024
+#define FKL_MAX_TOP 64
+#define FKL_ERR_TOKEN 0x20000u
+#define FKL_ERR_CAPACITY 0x100000u
+#define FKL_ERR_TC_WAIT 0x200000u
+
+enum { FKL_ACT_NONE = 0, FKL_ACT_RELU2 = 2 };
+
+__device__ __forceinline__ float ldT(const uint16_t *p) { return bf2f(*p); }
+__device__ __forceinline__ float ldT(const float *p) { return *p; }
+__device__ __forceinline__ void stT(uint16_t *p, float v) { *p = f2bf(v); }
+__device__ __forceinline__ void stT(float *p, float v) { *p = v; }
+__device__ __forceinline__ float act_apply(float v, int act) { if (act == FKL_ACT_RELU2) { v = fmaxf(v, 0.0f); v *= v; } return v; }
+__device__ __forceinline__ float inv_rms(float ss, int n, float eps) { return __fdiv_rn(1.0f, __fsqrt_rn(ss / (float)n + eps)); }
+__device__ __forceinline__ float sigmoid_f(float z) { return __fdiv_rn(1.0f, 1.0f + expf(-z)); }
+__device__ __forceinline__ void unpack8f(uint4 v, float (&f)[8]) {
+    f[0] = bf_lo(v.x); f[1] = bf_hi(v.x); f[2] = bf_lo(v.y); f[3] = bf_hi(v.y); f[4] = bf_lo(v.z); f[5] = bf_hi(v.z); f[6] = bf_lo(v.w); f[7] = bf_hi(v.w);
+}
+__device__ __forceinline__ void load8(const uint16_t *p, float (&f)[8]) { unpack8f(__ldcg(reinterpret_cast<const uint4 *>(p)), f); }
+__device__ __forceinline__ void load8(const float *p, float (&f)[8]) {
+    const float4 a = __ldcg(reinterpret_cast<const float4 *>(p)), b = __ldcg(reinterpret_cast<const float4 *>(p) + 1);
+    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
+}
+
+// ---------------------------------------------------------------- embedding rows, fp32
+struct EmbedRowsArgs { const uint16_t *table; float *x; const uint32_t *tokens; int d, vocab; };
+__global__ void k_embed_rows(FkState *st, EmbedRowsArgs a) {
+    pdl_wait(); pdl_launch_dependents();
+    const int m = blockIdx.x;
+    uint32_t tok = a.tokens ? __ldcg(a.tokens + m) : st->token[m];
+    if (tok >= (uint32_t)a.vocab) { if (threadIdx.x == 0) atomicOr(&st->error, FKL_ERR_TOKEN); tok = 0; }
+    const uint16_t *src = a.table + (size_t)tok * a.d; float *dst = a.x + (size_t)m * a.d;
+    for (int i = threadIdx.x; i < a.d; i += blockDim.x) dst[i] = bf2f(src[i]);
+}
+
+// ---------------------------------------------------------------- residual add with post-norm, then the next pre-norm
+// x <- x + norm(y) * post_w (+ add), h <- norm(x) * norm_w, per row.  y is a product's rows, or the rows of a mixture of
+// experts: y (shared expert, may be absent) + sum_j weight[j] * moe_y[slot[j]].  `index` picks the rows that are wanted
+// (final norm): output row r comes from row index[r] and x is not written.
+struct ResNormArgs {
+    const float *x; const void *y; const uint16_t *post_w; const float *add; float *x_out; const uint16_t *norm_w; void *h; const uint32_t *index;
+    const void *moe_y; const int *slot; const float *weight; int d, ldh, top, ldy; float eps;
+};
+template <typename T>
+__global__ void __launch_bounds__(512) k_residual_norm_rows(const FkState *st, ResNormArgs a) {
+    extern __shared__ float xs[];                       // [d]
+    __shared__ float red[40];
+    pdl_wait(); pdl_launch_dependents();
+    const size_t row = a.index ? a.index[blockIdx.x] : blockIdx.x;
+    const float *x = a.x + row * a.d;
+    float ry = 0.0f;
+    const bool pend = a.y || a.moe_y;
+    if (pend) {
+        float ss = 0.0f;
+        for (int i = threadIdx.x; i < a.d; i += blockDim.x) {
+            float v = a.y ? ldT((const T *)a.y + row * a.ldy + i) : 0.0f;
+            if (a.moe_y) for (int j = 0; j < a.top; ++j) v = fmaf(a.weight[row * a.top + j], ldT((const T *)a.moe_y + (size_t)a.slot[row * a.top + j] * a.ldy + i), v);
+            xs[i] = v; ss = fmaf(v, v, ss);
+        }
+        ry = inv_rms(block_sum(ss, red), a.d, a.eps);
+    }
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < a.d; i += blockDim.x) {
+        float v = x[i];
+        if (pend) v = fmaf(xs[i] * ry, bf2f(a.post_w[i]), v);
+        if (a.add) v += a.add[row * a.d + i];
+        xs[i] = v; ss = fmaf(v, v, ss);
+        if (a.x_out) a.x_out[row * a.d + i] = v;
+    }
+    const float r = inv_rms(block_sum(ss, red), a.d, a.eps);
+    T *h = (T *)a.h + (size_t)blockIdx.x * a.ldh;
+    for (int i = threadIdx.x; i < a.d; i += blockDim.x) stT(h + i, xs[i] * r * bf2f(a.norm_w[i]));
+}
+
+// ---------------------------------------------------------------- matrix product on rows, CUDA cores
+// Y[m, n] = act(sum_k X[m, k] W[row0 + n, k]); with `offsets` the rows of X are grouped by expert (expert e owns rows
+// offsets[e] .. offsets[e + 1] - 1 and the weight rows e * N ..).  fp32 arithmetic: the product of the 32-bit mode.
+struct LinRowsArgs { const void *x; const uint16_t *w; void *y; const int *offsets; int m, n, k, ldx, ldw, ldy, act, out_f32; };
+template <typename T>
+__global__ void __launch_bounds__(256) k_linear_rows(const FkState *st, LinRowsArgs a) {
+    __shared__ float As[16][68], Bs[16][68];
+    pdl_wait(); pdl_launch_dependents();
+    int m0 = blockIdx.y * 64, mend = a.m; const uint16_t *w = a.w;
+    if (a.offsets) {
+        const int e = blockIdx.z, o = a.offsets[e];
+        m0 += o; mend = a.offsets[e + 1]; w += (size_t)e * a.n * a.ldw;
+    }
+    if (m0 >= mend) return;
+    const int n0 = blockIdx.x * 64, tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    float acc[4][4] = {};
+    const int lr = tid >> 2, lk = (tid & 3) * 4;        // 64 rows x 16 k, four k per thread
+    for (int k0 = 0; k0 < a.k; k0 += 16) {
+        const int mr = m0 + lr, nr = n0 + lr;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            As[lk + j][lr] = mr < mend ? ldT((const T *)a.x + (size_t)mr * a.ldx + k0 + lk + j) : 0.0f;
+            Bs[lk + j][lr] = nr < a.n ? bf2f(w[(size_t)nr * a.ldw + k0 + lk + j]) : 0.0f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < 16; ++k) {
+            const float4 av = *reinterpret_cast<const float4 *>(&As[k][ty * 4]), bv = *reinterpret_cast<const float4 *>(&Bs[k][tx * 4]);
+            const float am[4] = {av.x, av.y, av.z, av.w}, bn[4] = {bv.x, bv.y, bv.z, bv.w};
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(am[i], bn[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+    for (int i = 0; i < 4; ++i) for (int j = 0; j < 4; ++j) {
+        const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
+        if (m >= mend || n >= a.n) continue;
+        const float v = act_apply(acc[i][j], a.act);
+        if (a.out_f32) ((float *)a.y)[(size_t)m * a.ldy + n] = v; else stT((T *)a.y + (size_t)m * a.ldy + n, v);
+    }
+}
+
+// ---------------------------------------------------------------- q/k norm and the cache store of M positions
+// Input rows q | k | v (| gate), heads laid out head by head with `maps` sub-heads of `dim` each.  q is normalised into a
+// buffer of its own, k into the cache [G * maps, capacity, dpad], v is copied into [G, capacity, vpad] (padding stays zero).
+struct QkStoreArgs { const void *qkv; const uint16_t *qn, *kn; void *q, *ck, *cv; int H, G, maps, dim, vdim, dpad, vpad, cap, rows, ld; float eps; };
+template <typename T>
+__global__ void __launch_bounds__(128) k_qk_norm_store_rows(FkState *st, QkStoreArgs a) {
+    pdl_wait(); pdl_launch_dependents();
+    const int lane = threadIdx.x & 31, item = blockIdx.y * 4 + (threadIdx.x >> 5), row = blockIdx.x;
+    const int nq = a.H * a.maps, nk = a.G * a.maps;
+    if (item >= nq + nk + a.G) return;
+    const uint32_t pos = st->offset + (uint32_t)row;
+    if (pos >= (uint32_t)a.cap) { if (lane == 0) atomicOr(&st->error, FKL_ERR_CAPACITY); return; }
+    const T *src = (const T *)a.qkv + (size_t)row * a.ld;
+    if (item >= nq + nk) {
+        const int g = item - nq - nk;
+        src += (nq + nk) * a.dim + g * a.vdim;
+        T *dst = (T *)a.cv + ((size_t)g * a.cap + pos) * a.vpad;
+        for (int i = lane; i < a.vdim; i += 32) dst[i] = src[i];
+        return;
+    }
+    src += item * a.dim;
+    const bool is_q = item < nq;
+    T *dst = is_q ? (T *)a.q + ((size_t)row * nq + item) * a.dpad : (T *)a.ck + ((size_t)(item - nq) * a.cap + pos) * a.dpad;
+    const uint16_t *w = is_q ? a.qn : a.kn;
+    float ss = 0.0f;
+    for (int i = lane; i < a.dim; i += 32) { const float v = ldT(src + i); ss = fmaf(v, v, ss); }
+    const float r = inv_rms(warp_sum(ss), a.dim, a.eps);
+    for (int i = lane; i < a.dim; i += 32) stT(dst + i, ldT(src + i) * r * bf2f(w[i]));
+}
+
+// ---------------------------------------------------------------- attention on CUDA cores (decode, and rows in 32-bit)
+// One block per (key split, kv head x tile of 8 query rows, position).  The query rows of a kv head are its H / G heads
+// times `maps`; all maps of a head sit in one tile.  A warp takes 32 keys at a time: scores with the lanes spread over
+// (key, 8-wide slice of dim), online softmax with one key per lane, then the values with the lanes spread over vdim.
+// Differential maps are combined at the end: a1 - lambda a2, unit rms over vdim, times 1 - diff; then the output gate.
+// DECODE: one position; q and k come raw from the projection (fp32) and are normalised here, the new key and value go into
+// the cache, and the keys are split over blocks (partials in global memory, the last block of a tile merges them).
+#define FKL_ATT_ROWS 8
+#define FKL_ATT_WARPS 8
+struct AttnArgs {
+    const float *qkv; const uint16_t *qn, *kn; const void *q; void *ck, *cv, *out; const void *gate; float *part; uint32_t *counter;
+    int H, G, maps, dim, vdim, dpad, vpad, cap, ldo, ldg, splits, tiles; float scale, lambda, diff, eps;
+};
+__host__ __device__ inline size_t attn_smem_floats(int dpad, int vpad) {
+    return (size_t)FKL_ATT_ROWS * dpad + FKL_ATT_WARPS * 32 * FKL_ATT_ROWS + FKL_ATT_WARPS * FKL_ATT_ROWS * ((size_t)vpad + 2) + FKL_ATT_ROWS * ((size_t)vpad + 2);
+}
+template <typename T, typename A, int VPL, bool DECODE>      // T: cache and q type; A: gate and output type
+__global__ void __launch_bounds__(FKL_ATT_WARPS * 32) k_attention(FkState *st, AttnArgs a) {
+    extern __shared__ float sm[];
+    constexpr int RT = FKL_ATT_ROWS, NW = FKL_ATT_WARPS;
+    float *qs = sm, *sc0 = qs + RT * a.dpad, *ow = sc0 + NW * 32 * RT, *mw = ow + (size_t)NW * RT * a.vpad, *of = mw + NW * RT * 2, *mf = of + RT * a.vpad;
+    __shared__ int s_last;
+    pdl_wait(); pdl_launch_dependents();
+    const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, row = blockIdx.z;
+    const int g = blockIdx.y / a.tiles, tile = blockIdx.y - g * a.tiles, group = a.H / a.G, nrow_kv = group * a.maps;
+    const int r0 = tile * RT, nr = min(RT, nrow_kv - r0);
+    const uint32_t pos = st->offset + (uint32_t)row;
+    if (pos >= (uint32_t)a.cap) { if (tid == 0) atomicOr(&st->error, FKL_ERR_CAPACITY); return; }
+    const int n = (int)pos + 1, per = ((n + a.splits - 1) / a.splits + 31) / 32 * 32;
+    const int k0 = blockIdx.x * per, k1 = min(n, k0 + per);
+    T *ck = (T *)a.ck + (size_t)g * a.maps * a.cap * a.dpad, *cv = (T *)a.cv + (size_t)g * a.cap * a.vpad;
+    // ---- the query rows (normalised), and in decode the new key and value
+    for (int i = tid; i < RT * a.dpad; i += NW * 32) qs[i] = 0.0f;
+    __syncthreads();
+    if (DECODE) {
+        const bool mine = (int)pos >= k0 && (int)pos < k1;
+        const int items = nr + (mine ? a.maps + 1 : 0);
+        for (int it = wid; it < items; it += NW) {
+            if (it == nr + a.maps) {
+                const float *src = a.qkv + (a.H + a.G) * a.maps * a.dim + g * a.vdim;
+                for (int i = lane; i < a.vdim; i += 32) stT(cv + (size_t)pos * a.vpad + i, src[i]);
+                continue;
+            }
+            const bool is_q = it < nr;
+            const float *src = a.qkv + (is_q ? (g * nrow_kv + r0 + it) : (a.H * a.maps + g * a.maps + (it - nr))) * a.dim;
+            const uint16_t *w = is_q ? a.qn : a.kn;
+            float ss = 0.0f;
+            for (int i = lane; i < a.dim; i += 32) ss = fmaf(src[i], src[i], ss);
+            const float r = inv_rms(warp_sum(ss), a.dim, a.eps);
+            for (int i = lane; i < a.dim; i += 32) {
+                const float v = src[i] * r * bf2f(w[i]);
+                if (is_q) qs[it * a.dpad + i] = v; else stT(ck + ((size_t)(it - nr) * a.cap + pos) * a.dpad + i, v);
+            }
+        }
+    } else {
+        const T *q = (const T *)a.q + ((size_t)row * a.H * a.maps + g * nrow_kv + r0) * a.dpad;
+        for (int i = tid; i < nr * a.dpad; i += NW * 32) qs[i] = ldT(q + i);
+    }
+    __syncthreads();
+    // ---- keys
+    int lpk = 1; while (lpk < 32 && lpk * 8 < a.dpad) lpk <<= 1;
+    const int kpp = 32 / lpk, sub = lane & (lpk - 1), kin = lane / lpk;
+    float *sc = sc0 + wid * 32 * RT;                   // [32 keys][RT]
+    float mrow[RT], lrow[RT], o[RT][VPL];
+#pragma unroll
+    for (int r = 0; r < RT; ++r) { mrow[r] = -INFINITY; lrow[r] = 0.0f; for (int i = 0; i < VPL; ++i) o[r][i] = 0.0f; }
+    for (int kb = k0 + wid * 32; kb < k1; kb += NW * 32) {
+        const int nk = min(32, k1 - kb);
+        for (int p0 = 0; p0 < nk; p0 += kpp) {
+            const int kk = p0 + kin; const bool kv = kk < nk;
+            for (int m = 0; m < a.maps; ++m) {
+                const T *krow = ck + ((size_t)m * a.cap + kb + (kv ? kk : 0)) * a.dpad;
+                float dot[RT] = {};
+                for (int d = sub * 8; d < a.dpad; d += lpk * 8) {
+                    float kf[8]; load8(krow + d, kf);
+#pragma unroll
+                    for (int r = 0; r < RT; ++r) if (r < nr && (r0 + r) % a.maps == m) {
+                        const float4 q0 = *reinterpret_cast<const float4 *>(qs + r * a.dpad + d), q1 = *reinterpret_cast<const float4 *>(qs + r * a.dpad + d + 4);
+                        dot[r] = fmaf(q0.x, kf[0], fmaf(q0.y, kf[1], fmaf(q0.z, kf[2], fmaf(q0.w, kf[3], dot[r]))));
+                        dot[r] = fmaf(q1.x, kf[4], fmaf(q1.y, kf[5], fmaf(q1.z, kf[6], fmaf(q1.w, kf[7], dot[r]))));
+                    }
+                }
+#pragma unroll
+                for (int r = 0; r < RT; ++r) if (r < nr && (r0 + r) % a.maps == m) {
+                    float v = dot[r];
+                    for (int s = lpk >> 1; s > 0; s >>= 1) v += __shfl_xor_sync(0xffffffffu, v, s);
+                    if (sub == 0 && kv) sc[kk * RT + r] = v;
+                }
+            }
+        }
+        __syncwarp();
+#pragma unroll
+        for (int r = 0; r < RT; ++r) if (r < nr) {
+            const float s = lane < nk ? sc[lane * RT + r] * a.scale : -INFINITY;
+            const float mn = fmaxf(mrow[r], warp_max(s)), corr = expf(mrow[r] - mn), p = expf(s - mn);
+            lrow[r] = lrow[r] * corr + warp_sum(p); mrow[r] = mn;
+            sc[lane * RT + r] = p;
+#pragma unroll
+            for (int i = 0; i < VPL; ++i) o[r][i] *= corr;
+        }
+        __syncwarp();
+        for (int k = 0; k < nk; ++k) {
+            float v[VPL];
+            const T *vrow = cv + (size_t)(kb + k) * a.vpad;
+#pragma unroll
+            for (int i = 0; i < VPL; ++i) { const int d = lane * VPL + i; v[i] = d < a.vpad ? ldT(vrow + d) : 0.0f; }
+#pragma unroll
+            for (int r = 0; r < RT; ++r) {
+                const float p = r < nr ? sc[k * RT + r] : 0.0f;
+#pragma unroll
+                for (int i = 0; i < VPL; ++i) o[r][i] = fmaf(p, v[i], o[r][i]);
+            }
+        }
+        __syncwarp();
+    }
+    // ---- fold the warps
+#pragma unroll
+    for (int r = 0; r < RT; ++r) {
+#pragma unroll
+        for (int i = 0; i < VPL; ++i) { const int d = lane * VPL + i; if (d < a.vpad) ow[((size_t)wid * RT + r) * a.vpad + d] = o[r][i]; }
+        if (lane == 0) { mw[(wid * RT + r) * 2] = mrow[r]; mw[(wid * RT + r) * 2 + 1] = lrow[r]; }
+    }
+    __syncthreads();
+    for (int i = tid; i < nr * a.vpad; i += NW * 32) {
+        const int r = i / a.vpad, d = i - r * a.vpad;
+        float mx = -INFINITY;
+        for (int w = 0; w < NW; ++w) mx = fmaxf(mx, mw[(w * RT + r) * 2]);
+        float s = 0.0f, l = 0.0f;
+        for (int w = 0; w < NW; ++w) {
+            const float f = mx == -INFINITY ? 0.0f : expf(mw[(w * RT + r) * 2] - mx);
+            s = fmaf(f, ow[((size_t)w * RT + r) * a.vpad + d], s); l = fmaf(f, mw[(w * RT + r) * 2 + 1], l);
+        }
+        of[r * a.vpad + d] = a.splits > 1 ? s : s / l;
+        if (d == 0) { mf[r * 2] = mx; mf[r * 2 + 1] = l; }
+    }
+    __syncthreads();
+    if (a.splits > 1) {
+        const size_t stride = (size_t)RT * (a.vpad + 2);
+        float *mine = a.part + ((size_t)blockIdx.y * a.splits + blockIdx.x) * stride;
+        for (int i = tid; i < nr * a.vpad; i += NW * 32) __stcg(mine + i, of[i]);
+        for (int i = tid; i < nr * 2; i += NW * 32) __stcg(mine + RT * a.vpad + i, mf[i]);
+        __threadfence();
+        __syncthreads();
+        if (tid == 0) { s_last = atomicAdd(a.counter + blockIdx.y, 1u) == (uint32_t)a.splits - 1u; if (s_last) a.counter[blockIdx.y] = 0u; }
+        __syncthreads();
+        if (!s_last) return;
+        __threadfence();
+        const float *base = a.part + (size_t)blockIdx.y * a.splits * stride;
+        // factor of every (split, row): exp(m - max), into shared memory reused from the warp partials
+        float *fac = ow;                                // [splits][RT]
+        for (int i = tid; i < a.splits * nr; i += NW * 32) fac[(i / nr) * RT + i % nr] = __ldcg(base + (size_t)(i / nr) * stride + RT * a.vpad + (i % nr) * 2);
+        __syncthreads();
+        if (tid < nr) {
+            float mx = -INFINITY, l = 0.0f;
+            for (int s = 0; s < a.splits; ++s) mx = fmaxf(mx, fac[s * RT + tid]);
+            for (int s = 0; s < a.splits; ++s) {
+                const float f = expf(fac[s * RT + tid] - mx);
+                fac[s * RT + tid] = f; l = fmaf(f, __ldcg(base + (size_t)s * stride + RT * a.vpad + tid * 2 + 1), l);
+            }
+            mf[tid * 2 + 1] = l;
+        }
+        __syncthreads();
+        for (int i = tid; i < nr * a.vpad; i += NW * 32) {
+            const int r = i / a.vpad;
+            float s = 0.0f;
+            for (int p = 0; p < a.splits; ++p) s = fmaf(fac[p * RT + r], __ldcg(base + (size_t)p * stride + i), s);
+            of[i] = s / mf[r * 2 + 1];
+        }
+        __syncthreads();
+    }
+    // ---- combine the maps, gate, store
+    for (int hh = wid; hh < nr / a.maps; hh += NW) {
+        const int head = g * group + r0 / a.maps + hh;
+        const float *o1 = of + hh * a.maps * a.vpad, *o2 = o1 + a.vpad;
+        float f = 1.0f;
+        if (a.maps == 2) {
+            float ss = 0.0f;
+            for (int d = lane; d < a.vdim; d += 32) { const float v = o1[d] - a.lambda * o2[d]; ss = fmaf(v, v, ss); }
+            f = inv_rms(warp_sum(ss), a.vdim, a.eps) * (1.0f - a.diff);
+        }
+        if (a.gate) f *= sigmoid_f(ldT((const A *)a.gate + (size_t)row * a.ldg + head));
+        A *out = (A *)a.out + (size_t)row * a.ldo + head * a.vdim;
+        for (int d = lane; d < a.vdim; d += 32) stT(out + d, (a.maps == 2 ? o1[d] - a.lambda * o2[d] : o1[d]) * f);
+    }
+}
+
+// ---------------------------------------------------------------- mixture of experts: choice and grouping of M rows
+// The `top` largest logits of z[0 .. E) by one warp (lowest index first among equals), into idx / val (lane 0 of the warp
+// and everyone else sees them after a __syncwarp).
+__device__ __forceinline__ void warp_top(const float *z, int E, int top, int *idx, float *val, int lane) {
+    // a candidate is taken strictly after the previous one in (value descending, index ascending) order
+    float pv = INFINITY; int pi = -1;
+    for (int j = 0; j < top; ++j) {
+        float bv = -INFINITY; int bi = 0x7fffffff;
+        for (int e = lane; e < E; e += 32) {
+            const float v = z[e];
+            const bool after = v < pv || (v == pv && e > pi);
+            if (after && (v > bv || (v == bv && e < bi))) { bv = v; bi = e; }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, bv, o); const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+            if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+        }
+        if (bi >= E) { bi = min(pi + 1, E - 1); bv = z[bi]; }      // only with NaN logits: keep the index in range
+        if (lane == 0) { idx[j] = bi; val[j] = bv; }
+        pv = bv; pi = bi;
+    }
+    __syncwarp();
+}
+// softmax over the chosen logits, in place (one warp; val[0] is the largest)
+__device__ __forceinline__ void warp_top_softmax(float *val, int top, int lane) {
+    const float mx = val[0];
+    float s = 0.0f;
+    for (int j = lane; j < top; j += 32) s += expf(val[j] - mx);
+    s = warp_sum(s);
+    __syncwarp();
+    for (int j = lane; j < top; j += 32) val[j] = expf(val[j] - mx) / s;
+    __syncwarp();
+}
+struct RouteArgs {
+    const float *logits; const void *h; float *weight; int *expert, *rank, *count, *slot, *offsets; void *hp; int rows, E, top, ldl, ld;
+};
+// each row's experts, weights, and its rank among the rows of that expert (the order inside an expert does not matter: every
+// row of a grouped product is computed by itself)
+__global__ void __launch_bounds__(128) k_moe_route(const FkState *st, RouteArgs a) {
+    __shared__ int idx[4][FKL_MAX_TOP]; __shared__ float val[4][FKL_MAX_TOP];
+    pdl_wait(); pdl_launch_dependents();
+    const int wid = threadIdx.x >> 5, lane = threadIdx.x & 31, row = blockIdx.x * 4 + wid;
+    if (row >= a.rows) return;
+    warp_top(a.logits + (size_t)row * a.ldl, a.E, a.top, idx[wid], val[wid], lane);
+    warp_top_softmax(val[wid], a.top, lane);
+    for (int j = lane; j < a.top; j += 32) {
+        const int s = row * a.top + j, e = idx[wid][j];
+        a.weight[s] = val[wid][j]; a.expert[s] = e; a.rank[s] = atomicAdd(a.count + e, 1);
+    }
+}
+// rows grouped by expert: slot of every (row, choice), expert offsets, and the copied activations
+template <typename T>
+__global__ void __launch_bounds__(256) k_moe_gather(const FkState *st, RouteArgs a) {
+    __shared__ int off[FKL_MAX_EXPERTS + 1]; __shared__ int wsum[8];
+    pdl_wait(); pdl_launch_dependents();
+    const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
+    int carry = 0;
+    for (int base = 0; base < a.E; base += 256) {       // exclusive scan of the counts
+        const int e = base + tid, c = e < a.E ? a.count[e] : 0;
+        int v = c;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) { const int t = __shfl_up_sync(0xffffffffu, v, o); if (lane >= o) v += t; }
+        if (lane == 31) wsum[wid] = v;
+        __syncthreads();
+        int before = carry, total = 0;
+        for (int w = 0; w < 8; ++w) { if (w < wid) before += wsum[w]; total += wsum[w]; }
+        if (e < a.E) off[e] = before + v - c;
+        carry += total;
+        __syncthreads();
+    }
+    if (tid == 0) off[a.E] = carry;
+    __syncthreads();
+    if (blockIdx.x == 0) for (int e = tid; e <= a.E; e += 256) a.offsets[e] = off[e];
+    const int s = blockIdx.x, row = s / a.top, dst = off[a.expert[s]] + a.rank[s];
+    if (tid == 0) a.slot[s] = dst;
+    const uint4 *src = reinterpret_cast<const uint4 *>((const T *)a.h + (size_t)row * a.ld);
+    uint4 *d = reinterpret_cast<uint4 *>((T *)a.hp + (size_t)dst * a.ld);
+    for (int i = tid; i < a.ld * (int)sizeof(T) / 16; i += 256) d[i] = __ldcg(src + i);
+}
+
+// ---------------------------------------------------------------- one row: matrix-vector products over bf16 rows
+// A warp owns R = 2 weight rows at a time and streams them in chunks of 256 weights (16 bytes per lane and row), two batches
+// of U = 4 chunks in registers: one being multiplied, one in flight.  The activations sit in shared memory as fp32, in the
+// order the lanes read them without bank conflicts.  With few rows, 2 .. 8 warps of a block share a row group and split K.
+// A chunk is described by (base of row 0, row stride, weights in it), which also expresses the concatenated K ranges of a
+// mixture's down projection.  The first batch is fetched before the dependency wait where the rows do not depend on it.
+#define FKL_GV_R 2
+#define FKL_GV_U 4
+#define FKL_GV_WARPS 8
+enum { FKL_GV_LINEAR = 0, FKL_GV_MOE_UP = 1, FKL_GV_MOE_DOWN = 2 };
+struct GvChunk { const uint16_t *base; int stride, len; };
+struct GemvArgs {
+    // input vector: x, or with norm_w set: x' = x + norm(pend) * post_w (+ add) -> x_out, then norm(x') * norm_w (-> h_out)
+    const float *x, *pend; const uint16_t *post_w; const float *add; float *x_out; const uint16_t *norm_w; float *h_out;
+    const uint16_t *w; float *y; int k, ldk, n, act, act_row0; float eps;
+    unsigned long long *amax; uint32_t *counter, *history;             // greedy choice over y (the last block advances the state)
+    // mixture of experts
+    const float *logits; int *sel; float *wts; const float *sact; const uint16_t *w2; int E, top, ff, ldff, ffs, ldffs;
+    int kslices, nchunks;
+};
+__host__ __device__ inline int gv_chunks(int ldk) { return (ldk + 255) / 256; }
+__host__ __device__ inline size_t gv_smem_bytes(int nchunks) { return (size_t)nchunks * (256 * 4 + sizeof(GvChunk)); }
+__device__ __forceinline__ int gv_place(int i) { const int j = i & 7; return (i & ~255) + (j >> 2) * 128 + ((i & 255) >> 3) * 4 + (j & 3); }
+__device__ __forceinline__ uint4 ldg_stream(const uint16_t *p) {
+    uint4 v; asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p)); return v;
+}
+template <int MODE>
+__global__ void __launch_bounds__(FKL_GV_WARPS * 32, 2) k_gemv(FkState *st, GemvArgs a) {
+    extern __shared__ __align__(16) unsigned char gv_smem[];
+    constexpr int R = FKL_GV_R, U = FKL_GV_U, NT = FKL_GV_WARPS * 32;
+    float *xs = reinterpret_cast<float *>(gv_smem); GvChunk *tab = reinterpret_cast<GvChunk *>(gv_smem + (size_t)a.nchunks * 1024);
+    __shared__ float red[40], part[FKL_GV_WARPS][R], tval[FKL_MAX_TOP]; __shared__ int tsel[FKL_MAX_TOP];
+    __shared__ unsigned long long wbest[FKL_GV_WARPS]; __shared__ int is_last;
+    const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, KS = a.kslices, spb = FKL_GV_WARPS / KS, ksl = wid % KS, slot = wid / KS;
+    const int c0 = a.nchunks * ksl / KS, c1 = a.nchunks * (ksl + 1) / KS, nb = (c1 - c0 + U - 1) / U;
+    const int groups = (a.n + R - 1) / R, gstride = gridDim.x * spb;
+    int g = blockIdx.x * spb + slot;
+    size_t roff[R];                                    // rows of the current fetch group: index into the chunk's rows
+    auto set_rows = [&](int gg) {
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+            int row = gg * R + r; row = row < a.n ? row : a.n - 1;
+            if (MODE == FKL_GV_MOE_UP) { const int j = row / a.ff; row = tsel[j] * a.ff + (row - j * a.ff); }
+            roff[r] = (size_t)row;
+        }
+    };
+    uint4 nxt[U][R];
+    auto fetch = [&](int c) {
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            if (c + u < c1) {
+                const GvChunk ch = tab[c + u];
+#pragma unroll
+                for (int r = 0; r < R; ++r) nxt[u][r] = lane * 8 < ch.len ? ldg_stream(ch.base + roff[r] * ch.stride + lane * 8) : make_uint4(0, 0, 0, 0);
+            } else {
+#pragma unroll
+                for (int r = 0; r < R; ++r) nxt[u][r] = make_uint4(0, 0, 0, 0);
+            }
+        }
+    };
+    for (int i = tid; i < a.nchunks * 256; i += NT) xs[i] = 0.0f;
+    if (MODE != FKL_GV_MOE_DOWN) {
+        for (int c = tid; c < a.nchunks; c += NT) tab[c] = GvChunk{a.w + c * 256, a.ldk, min(256, a.ldk - c * 256)};
+        __syncthreads();
+        if (MODE == FKL_GV_LINEAR && g < groups && nb > 0) { set_rows(g); fetch(c0); }
+    }
+    pdl_wait(); pdl_launch_dependents();
+    // ---- the input vector
+    if (MODE == FKL_GV_MOE_DOWN) {
+        const int nce = gv_chunks(a.ldff), nshared = a.nchunks - a.top * nce;
+        for (int j = tid; j < a.top; j += NT) { tsel[j] = a.sel[j]; tval[j] = a.wts[j]; }
+        __syncthreads();
+        for (int c = tid; c < a.nchunks; c += NT) {
+            const int j = c / nce, cc = c - j * nce;
+            if (j < a.top) tab[c] = GvChunk{a.w + (size_t)tsel[j] * a.n * a.ldff + cc * 256, a.ldff, min(256, a.ldff - cc * 256)};
+            else { const int cs = c - a.top * nce; tab[c] = GvChunk{a.w2 + cs * 256, a.ldffs, min(256, a.ldffs - cs * 256)}; }
+        }
+        (void)nshared;
+        for (int i = tid; i < a.top * a.ff; i += NT) { const int j = i / a.ff, q = i - j * a.ff; xs[gv_place(j * nce * 256 + q)] = tval[j] * __ldcg(a.x + i); }
+        for (int i = tid; i < a.ffs; i += NT) xs[gv_place(a.top * nce * 256 + i)] = __ldcg(a.sact + i);
+        __syncthreads();
+        if (g < groups && nb > 0) { set_rows(g); fetch(c0); }
+    } else if (MODE == FKL_GV_MOE_UP) {
+        if (wid == 0) {
+            warp_top(a.logits, a.E, a.top, tsel, tval, lane);
+            if (blockIdx.x == 0) {
+                warp_top_softmax(tval, a.top, lane);
+                for (int j = lane; j < a.top; j += 32) { a.sel[j] = tsel[j]; a.wts[j] = tval[j]; }
+            }
+        }
+        for (int i = tid; i < a.k; i += NT) xs[gv_place(i)] = __ldcg(a.x + i);
+        __syncthreads();
+        if (g < groups && nb > 0) { set_rows(g); fetch(c0); }
+    } else if (a.norm_w) {
+        __syncthreads();
+        float ry = 0.0f;
+        if (a.pend) {
+            float ss = 0.0f;
+            for (int i = tid; i < a.k; i += NT) { const float v = __ldcg(a.pend + i); ss = fmaf(v, v, ss); }
+            ry = inv_rms(block_sum(ss, red), a.k, a.eps);
+        }
+        float ss = 0.0f;
+        for (int i = tid; i < a.k; i += NT) {
+            float v = __ldcg(a.x + i);
+            if (a.pend) v = fmaf(__ldcg(a.pend + i) * ry, bf2f(a.post_w[i]), v);
+            if (a.add) v += __ldcg(a.add + i);
+            xs[gv_place(i)] = v; ss = fmaf(v, v, ss);
+            if (a.x_out && blockIdx.x == 0) a.x_out[i] = v;
+        }
+        const float r = inv_rms(block_sum(ss, red), a.k, a.eps);
+        for (int i = tid; i < a.k; i += NT) {
+            const float v = xs[gv_place(i)] * r * bf2f(a.norm_w[i]);
+            xs[gv_place(i)] = v;
+            if (a.h_out && blockIdx.x == 0) a.h_out[i] = v;
+        }
+        __syncthreads();
+    } else {
+        __syncthreads();
+        for (int i = tid; i < a.k; i += NT) xs[gv_place(i)] = __ldcg(a.x + i);
+        __syncthreads();
+    }
+    // ---- rows
+    unsigned long long best = 0ull;
+    const int rounds = (groups + gstride - 1) / gstride;          // the same for all blocks and warps (K split: barriers inside)
+    for (int rd = 0; rd < rounds; ++rd, g += gstride) {
+        if (KS == 1 && g >= groups) break;
+        const bool live = g < groups;
+        float acc[R] = {};
+        if (live) for (int b = 0; b < nb; ++b) {
+            uint4 cur[U][R];
+#pragma unroll
+            for (int u = 0; u < U; ++u)
+#pragma unroll
+                for (int r = 0; r < R; ++r) cur[u][r] = nxt[u][r];
+            if (b + 1 < nb) fetch(c0 + (b + 1) * U);
+            else if (g + gstride < groups) { set_rows(g + gstride); fetch(c0); }
+#pragma unroll
+            for (int u = 0; u < U; ++u) {
+                const int c = c0 + b * U + u;
+                if (c < c1) {
+                    const float4 x0 = *reinterpret_cast<const float4 *>(xs + c * 256 + lane * 4), x1 = *reinterpret_cast<const float4 *>(xs + c * 256 + 128 + lane * 4);
+#pragma unroll
+                    for (int r = 0; r < R; ++r) {
+                        float f[8]; unpack8f(cur[u][r], f);
+                        acc[r] = fmaf(f[0], x0.x, fmaf(f[1], x0.y, fmaf(f[2], x0.z, fmaf(f[3], x0.w, acc[r]))));
+                        acc[r] = fmaf(f[4], x1.x, fmaf(f[5], x1.y, fmaf(f[6], x1.z, fmaf(f[7], x1.w, acc[r]))));
+                    }
+                }
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < R; ++r) acc[r] = warp_sum(acc[r]);
+        if (KS > 1) {
+            if (lane == 0) for (int r = 0; r < R; ++r) part[wid][r] = acc[r];
+            __syncthreads();
+            if (ksl == 0) for (int r = 0; r < R; ++r) for (int q = 1; q < KS; ++q) acc[r] += part[wid + q][r];
+            __syncthreads();
+        }
+        if (live && ksl == 0) {
+#pragma unroll
+            for (int r = 0; r < R; ++r) {
+                const int row = g * R + r;
+                if (row < a.n) {
+                    const float v = row >= a.act_row0 ? act_apply(acc[r], a.act) : acc[r];
+                    if (lane == 0) a.y[row] = v;
+                    if (a.amax) {
+                        const uint32_t u = __float_as_uint(v), key = (u & 0x80000000u) ? ~u : u | 0x80000000u;
+                        const unsigned long long kk = ((unsigned long long)key << 32) | (unsigned long long)(0xffffffffu - (uint32_t)row);
+                        best = kk > best ? kk : best;
+                    }
+                }
+            }
+        }
+    }
+    if (MODE != FKL_GV_LINEAR || !a.amax) return;
+    if (lane == 0) wbest[wid] = best;
+    __syncthreads();
+    if (tid == 0) {
+        for (int i = 1; i < FKL_GV_WARPS; ++i) best = wbest[i] > best ? wbest[i] : best;
+        a.amax[blockIdx.x] = best;
+        __threadfence();
+        is_last = atomicAdd(a.counter, 1u) == gridDim.x - 1;
+        if (is_last) *a.counter = 0u;
+    }
+    __syncthreads();
+    if (!is_last || wid != 0) return;
+    __threadfence();
+    unsigned long long b = 0ull;
+    for (int i = lane; i < (int)gridDim.x; i += 32) { const unsigned long long v = __ldcg(a.amax + i); b = v > b ? v : b; }
+    b = warp_max_u64(b);
+    if (lane == 0) {
+        const uint32_t next = 0xffffffffu - (uint32_t)(b & 0xffffffffull);
+        st->token[0] = next;
+        if (a.history && st->hist_counter < st->hist_cap) a.history[st->hist_counter] = next;
+        st->hist_counter += 1; st->offset += 1; st->epoch += 1;
+    }
+}
+
+// greedy token of one row of fp32 logits, ties to the lowest index; advances the position by `advance` (end of a portion)
+__global__ void __launch_bounds__(1024) k_argmax_row_f32(FkState *st, const float *logits, uint32_t *history, int v, int advance) {
+    __shared__ unsigned long long wbest[32];
+    pdl_wait(); pdl_launch_dependents();
+    unsigned long long best = 0ull;
+    for (int i = threadIdx.x; i < v; i += blockDim.x) {
+        const uint32_t u = __float_as_uint(__ldcg(logits + i)), key = (u & 0x80000000u) ? ~u : u | 0x80000000u;
+        const unsigned long long kk = ((unsigned long long)key << 32) | (unsigned long long)(0xffffffffu - (uint32_t)i);
+        best = kk > best ? kk : best;
+    }
+    best = warp_max_u64(best);
+    if ((threadIdx.x & 31) == 0) wbest[threadIdx.x >> 5] = best;
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        for (int i = 1; i < (int)(blockDim.x >> 5); ++i) best = wbest[i] > best ? wbest[i] : best;
+        const uint32_t next = 0xffffffffu - (uint32_t)(best & 0xffffffffull);
+        st->token[0] = next;
+        if (history && st->hist_counter < st->hist_cap) history[st->hist_counter] = next;
+        st->hist_counter += 1; st->offset += (uint32_t)advance; st->epoch += 1;
+    }
+}

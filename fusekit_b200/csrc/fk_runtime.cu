@@ -9,6 +9,7 @@
 #include "fk_qmm.cuh"
 #include "fk_qmm_tc.cuh"
 #include "fk_json.h"
+#include "fk_layers.h"
 #include <chrono>
 #include <thread>
 
@@ -162,6 +163,7 @@ extern "C" fk_status fk_open(int device, fk_handle *out) {
     CU(big_smem(k_linear_residual<4>)); CU(big_smem(k_linear_residual<8>)); CU(big_smem(k_linear_residual<16>));
     CU(big_smem(k_rmsnorm_gateup_act<4>)); CU(big_smem(k_rmsnorm_gateup_act<8>)); CU(big_smem(k_rmsnorm_gateup_act<16>));
     CU(big_smem(k_final_head<4>)); CU(big_smem(k_final_head<8>)); CU(big_smem(k_final_head<16>));
+    CU(fkl_init());
     c->open = true;
     std::lock_guard<std::mutex> lk(g_mu);
     g_ctx.push_back(c); *out = g_ctx.size();
@@ -201,7 +203,9 @@ static const char *kKernelNames[FK_TASK_KIND_COUNT] = {
     "fusekit_step_init", "fusekit_embed_lookup_decode", "fusekit_rmsnorm_qkv", "fusekit_qk_norm_rope_store",
     "fusekit_sdpa_decode", "fusekit_linear_residual", "fusekit_rmsnorm_gateup_act", "fusekit_final_rmsnorm_lm_head",
     "fusekit_argmax_finalize", "fusekit_allreduce", "fusekit_residual_add", "fusekit_rmsnorm_rows", "fusekit_rope_store_rows",
-    "fusekit_argmax_rows", "fusekit_kv_store_quant", "fusekit_sdpa_decode_quant"};
+    "fusekit_argmax_rows", "fusekit_kv_store_quant", "fusekit_sdpa_decode_quant", "fusekit_embed_rows", "fusekit_residual_norm_rows",
+    "fusekit_linear_rows", "fusekit_qk_norm_store_rows", "fusekit_attention_rows", "fusekit_moe_route_rows", "fusekit_norm_linear",
+    "fusekit_attention_decode", "fusekit_moe_up", "fusekit_moe_down", "fusekit_argmax_row"};
 extern "C" fk_status fk_kernel_names(char *buf, size_t cap) {
     if (!buf || cap == 0) return fail(FK_ERR_VALUE, "buf is null");
     std::string s;
@@ -334,6 +338,16 @@ extern "C" fk_status fk_weight_finalize(fk_handle h, fk_weight wid) {
         drop_rows(w);
     } else { w->rows_kind = FK_ROWS_PLAIN; }
     w->finalized = true;
+    return FK_OK;
+}
+// Freezes a dense weight as the rows it was uploaded as: the layout of the layered decoders' kernels (matrix-vector products and
+// tensor-core tiles read the same rows).
+extern "C" fk_status fk_weight_keep_rows(fk_handle h, fk_weight wid) {
+    CTX(h); Weight *w = get_w(c, wid);
+    if (!w) return fail(FK_ERR_VALUE, "bad weight id");
+    if (w->finalized) return w->tiled ? fail(FK_ERR_STATE, "weight already repacked") : FK_OK;
+    if (w->bits != 16) return fail(FK_ERR_VALUE, "only dense bf16 weights are kept as rows");
+    w->rows_kind = FK_ROWS_PLAIN; w->finalized = true;
     return FK_OK;
 }
 extern "C" fk_status fk_weight_pair(fk_handle h, fk_weight gate, fk_weight up, fk_weight *out) {
@@ -534,7 +548,20 @@ static fk_status make_xchg(Ctx *c, int site_plus1, PeerXchg *x, const char *what
     x->map = c->peers; x->site = FK_PEER_SITE0 + site_plus1 - 1;
     return FK_OK;
 }
+static bool rows_weight(void *owner, uint64_t id, FklWeight *out) {
+    const Weight *w = get_w((Ctx *)owner, id);
+    if (!w || !w->finalized || w->tiled || w->bits != 16 || !w->w) return false;
+    *out = FklWeight{(const uint16_t *)w->w, w->n, w->k};
+    return true;
+}
 static fk_status run_task(Ctx *c, const fk_task &t, const Weight *nextw = nullptr) {
+    if (fkl_owns(t.kind)) {
+        FklEnv env{c->stream, c->pdl, c->sm_count, c->state, c->history, &c->launches, c, rows_weight};
+        if (t.kind == FK_TASK_EMBED_ROWS && t.iarg[2] > 0) c->vocab = (uint32_t)t.iarg[2];
+        char err[256] = "";
+        fk_status s = fkl_run(env, t, err, sizeof err);
+        return s ? fail(s, "%s", err) : FK_OK;
+    }
     const uint64_t *b = t.buf; const int32_t *i = t.iarg; const float *f = t.farg;
     cudaError_t e = cudaSuccess;
     switch (t.kind) {

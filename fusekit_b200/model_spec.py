@@ -73,6 +73,123 @@ class ModelSpec:
         return self.weight_bytes_per_token() + self.kv_bytes_per_token(ctx)
 
 
+# ---------------------------------------------------------------- decoders described layer by layer
+@dataclass(frozen=True)
+class AttentionSpec:
+    """Attention with an RMS norm on every q/k (sub-)head, no rotation and a sigmoid output gate per head.  ``diff`` set:
+    differential attention -- every head has two query/key maps over the same values, combined as a1 - lambda a2."""
+    heads: int
+    kv_heads: int
+    dim: int                  # query/key size of a map
+    vdim: int
+    scale: float              # score = (q . k) * scale
+    diff: float | None = None
+
+    @property
+    def maps(self) -> int:
+        return 1 if self.diff is None else 2
+
+    @property
+    def q_rows(self) -> int:
+        return self.heads * self.maps * self.dim
+
+    @property
+    def k_rows(self) -> int:
+        return self.kv_heads * self.maps * self.dim
+
+    @property
+    def v_rows(self) -> int:
+        return self.kv_heads * self.vdim
+
+    @property
+    def rows(self) -> int:    # q | k | v | gate, the fused projection
+        return self.q_rows + self.k_rows + self.v_rows + self.heads
+
+
+@dataclass(frozen=True)
+class MoeSpec:
+    """Mixture of ``experts`` feed-forward layers W_down relu(W_up h)^2, ``top`` per token weighted by the softmax over the
+    chosen router logits, plus a shared one of size ``shared_ff`` (0: none)."""
+    experts: int
+    top: int
+    ff: int
+    shared_ff: int = 0
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    mixer: AttentionSpec
+    mlp: MoeSpec | None = None
+
+
+@dataclass(frozen=True)
+class LoopSpec:
+    """Layers start .. stop - 1 run ``times`` times in a row; the embedding output is added to x before each repetition."""
+    start: int
+    stop: int
+    times: int
+
+
+@dataclass(frozen=True)
+class LayeredSpec:
+    """A decoder whose layers are listed one by one: norms before and after each sublayer, an fp32 residual stream, layers of
+    unequal sizes, a looped range.  A *run* is one execution of a layer; every run has its own cache."""
+    name: str
+    arch: str
+    hidden: int
+    vocab: int
+    layers: tuple
+    eps: float = 1e-6
+    loop: LoopSpec | None = None
+    seed: int = 20240531
+    bits: int = 16
+
+    def __post_init__(self):
+        lp = self.loop
+        if lp is not None and not (0 <= lp.start < lp.stop <= len(self.layers) and lp.times >= 1):
+            raise ValueError(f"{self.name}: loop {lp} does not fit {len(self.layers)} layers")
+        for i, l in enumerate(self.layers):
+            m, f = l.mixer, l.mlp
+            if min(m.heads, m.kv_heads, m.dim, m.vdim) < 1 or m.heads % m.kv_heads:
+                raise ValueError(f"{self.name}: layer {i}: attention sizes {m}")
+            if f is not None and not (1 <= f.top <= f.experts and f.ff >= 1 and f.shared_ff >= 0):
+                raise ValueError(f"{self.name}: layer {i}: expert sizes {f}")
+
+    def runs(self) -> list:
+        """(layer, the embedding output is added first) in execution order."""
+        lp, n = self.loop, len(self.layers)
+        if lp is None:
+            return [(i, False) for i in range(n)]
+        body = [(i, k > 0 and i == lp.start) for k in range(lp.times) for i in range(lp.start, lp.stop)]
+        return [(i, False) for i in range(lp.start)] + body + [(i, False) for i in range(lp.stop, n)]
+
+    # ---- algorithmic bytes of a decode step at bf16: every weight that is used once, and the keys and values
+    def weight_bytes_per_token(self) -> int:
+        tot = self.hidden * self.vocab
+        for i, _ in self.runs():
+            m, f = self.layers[i].mixer, self.layers[i].mlp
+            tot += m.rows * self.hidden + self.hidden * m.heads * m.vdim
+            if f is not None:
+                tot += self.hidden * (f.experts + 2 * f.shared_ff + 2 * f.top * f.ff)
+        return 2 * tot
+
+    def kv_bytes_per_token(self, ctx: int) -> int:
+        return sum(2 * ctx * (self.layers[i].mixer.k_rows + self.layers[i].mixer.v_rows) for i, _ in self.runs())
+
+    def bytes_per_token(self, ctx: int) -> int:
+        return self.weight_bytes_per_token() + self.kv_bytes_per_token(ctx)
+
+    def flops_per_token(self, ctx: float) -> float:
+        """Multiply-adds x 2 of one position that sees ``ctx`` keys, the head left out (prompt positions need no logits)."""
+        w = self.weight_bytes_per_token() // 2 - self.hidden * self.vocab
+        att = sum(self.layers[i].mixer.heads * self.layers[i].mixer.maps * (self.layers[i].mixer.dim + self.layers[i].mixer.vdim) for i, _ in self.runs())
+        return 2.0 * (w + att * ctx)
+
+
+def _fatulix(name, hidden, vocab, n_layers, attn, mlp, loop=None):
+    return LayeredSpec(name, "Fatulix", hidden, vocab, tuple(LayerSpec(attn, mlp) for _ in range(n_layers)), loop=loop)
+
+
 CONFIGS = {
     # Qwen2.5-0.5B-shaped (CPU-reference-sized parity config)
     "qwen2.5-0.5b": ModelSpec("qwen2.5-0.5b", "qwen2", 24, 896, 14, 2, 64, 4864, 151936),
@@ -86,6 +203,23 @@ CONFIGS = {
     "tiny-qwen": ModelSpec("tiny-qwen", "qwen2", 2, 256, 4, 2, 64, 512, 1024),
     "tiny-gemma": ModelSpec("tiny-gemma", "gemma3", 3, 256, 4, 2, 64, 512, 1024, window=16, global_every=3),
 }
+
+
+LAYERED_CONFIGS = {
+    # looped mixture-of-experts decoders with differential attention, at sizes of a small and a mid-size model's layers
+    "fatulix-2048": _fatulix("fatulix-2048", 2048, 65536, 8, AttentionSpec(16, 4, 64, 128, 0.125, 0.3), MoeSpec(32, 4, 1024, 2048), LoopSpec(2, 6, 2)),
+    "fatulix-3584": _fatulix("fatulix-3584", 3584, 152064, 8, AttentionSpec(28, 4, 64, 128, 0.125, 0.3), MoeSpec(16, 2, 4736, 9472)),
+    "tiny-fatulix": _fatulix("tiny-fatulix", 128, 320, 3, AttentionSpec(6, 2, 24, 32, 0.2, 0.4), MoeSpec(5, 2, 64, 128), LoopSpec(1, 3, 2)),
+}
+
+
+def config(name: str):
+    """The registered shape called ``name``: a ModelSpec or a LayeredSpec."""
+    if name in CONFIGS:
+        return CONFIGS[name]
+    if name in LAYERED_CONFIGS:
+        return LAYERED_CONFIGS[name]
+    raise KeyError(f"no configuration {name!r}; known: {sorted(CONFIGS) + sorted(LAYERED_CONFIGS)}")
 
 
 # ---- tensor naming / stream ids (FNV-1a 64 of the name, xor a mix of the seed) ----

@@ -18,7 +18,7 @@ import numpy as np
 
 from . import _native as N
 from . import task_graph
-from .model_spec import ModelSpec, stream_id, tensor_name
+from .model_spec import LayeredSpec, ModelSpec, stream_id, tensor_name
 
 FK_CHUNK = 64          # tokens pre-submitted per chunk (reference FK_CHUNK, dispatch.py:1103)
 
@@ -90,6 +90,9 @@ class Runtime:
 
     def weight_synth_rows(self, wid, dst_row0, nrows, stream, std, k_global, src_row0, k0):
         N.check(self.L.fk_weight_synth_rows(self.h, wid, dst_row0, nrows, stream, std, k_global, src_row0, k0), "fk_weight_synth_rows")
+
+    def weight_keep_rows(self, wid):
+        N.check(self.L.fk_weight_keep_rows(self.h, wid), "fk_weight_keep_rows")
 
     def weight_finalize(self, wid):
         N.check(self.L.fk_weight_finalize(self.h, wid), "fk_weight_finalize")
@@ -181,7 +184,143 @@ def check_tp(spec: ModelSpec, world: int):
         raise ValueError("tensor parallelism is wired for the Qwen-shaped layer only")
 
 
-class DecodeEngine:
+class EngineBase:
+    """What every decode engine shares: a task graph whose roles ``_resolve`` turns into addresses, its capture as one CUDA
+    graph per token, and the greedy / sampled loops over replays.  An engine sets ``rt``, ``graph`` and ``logits``."""
+
+    def task_graph(self) -> dict:
+        raise NotImplementedError
+
+    def _resolve(self, role: str) -> int:
+        raise NotImplementedError
+
+    def last_logits(self) -> np.ndarray:
+        raise NotImplementedError
+
+    def dispatches_from(self, graph: dict) -> list:
+        """Resolve a task graph document (from task_graph.emit or read back from JSON) to the fk_task list, in
+        decode_pipeline order (the reference's replay order, src/codegen/task_graph_json.rs:1619-1664)."""
+        if graph.get("version") != task_graph.VERSION:
+            raise ValueError(f"task graph version {graph.get('version')} (this runtime reads {task_graph.VERSION})")
+        if graph.get("active_m", 1) != 1:
+            raise ValueError("only batch-1 decode graphs are dispatchable")
+        if not graph["decode_capabilities"]["dispatchable"]:
+            raise ValueError("task graph is not dispatchable: " + "; ".join(graph["decode_capabilities"]["reasons"]))
+        by_id = {t["id"]: t for t in graph["tasks"]}
+        out = []
+        for tid in graph["decode_pipeline"]:
+            t = by_id[tid]
+            bufs = {slot: self._resolve(role) for slot, role in task_graph.task_slots(t).items()}
+            out.append(N.Task.make(t["kind"], t.get("layer_idx", -1), bufs, t["iargs"], t["fargs"]))
+        return out
+
+    def role_table(self, graph: dict) -> list:
+        """(role, address-or-weight-id) for every explicit binding of the document: the table the library's own JSON reader
+        (fk_tasks_from_json / fk_graph_capture_json) resolves role strings through."""
+        roles = sorted({b["role"] for t in graph["tasks"] for b in t["extra_bindings"] if b["slot"] < 100})
+        return [(r, self._resolve(r)) for r in roles]
+
+    def dispatches_from_json(self, text: str, table=None) -> list:
+        """The fk_task list of a task_graph.json text as the library parses it (no Python between the file and the records)."""
+        import json
+        table = self.role_table(json.loads(text)) if table is None else table
+        L = N.lib()
+        arr = (N.RoleBinding * max(1, len(table)))(*[N.RoleBinding(r.encode(), int(v)) for r, v in table])
+        n = C.c_int32()
+        N.check(L.fk_tasks_from_json(text.encode(), arr, len(table), None, 0, C.byref(n)), "fk_tasks_from_json")
+        out = (N.Task * max(1, n.value))()
+        N.check(L.fk_tasks_from_json(text.encode(), arr, len(table), out, n.value, C.byref(n)), "fk_tasks_from_json")
+        return list(out)[: n.value]
+
+    def capture_json(self, text: str) -> int:
+        """Capture the decode step straight from a task_graph.json text (reference: load_dispatcher + build_icb,
+        python_runtime/src/lib.rs:115-169, 459-570)."""
+        import json
+        table = self.role_table(json.loads(text))
+        arr = (N.RoleBinding * len(table))(*[N.RoleBinding(r.encode(), int(v)) for r, v in table])
+        g = C.c_uint64()
+        N.check(self.rt.L.fk_graph_capture_json(self.rt.h, text.encode(), arr, len(table), C.byref(g)), "fk_graph_capture_json")
+        self.tasks = self.replay = self.dispatches_from_json(text, table)
+        self.graph = g.value
+        return self.graph
+
+    def build_dispatches(self) -> list:
+        """The per-token kernel list in replay order (reference order: embed -> per layer RmsNormQkv,
+        SDPA, LinearResidual, gate/up chain, LinearResidual -> final head -> argmax;
+        src/codegen/task_graph_json.rs:1619-1664, dispatch.py:3163-3611)."""
+        return self.dispatches_from(self.task_graph())
+
+    # ------------------------------------------------------------------ replay
+    def capture(self) -> int:
+        """Capture the per-token task list once as a CUDA graph (reference: build_icb, lib.rs:459-570)."""
+        self.tasks = self.replay = self.build_dispatches()
+        arr = (N.Task * len(self.replay))(*self.replay)
+        g = C.c_uint64()
+        N.check(self.rt.L.fk_graph_capture(self.rt.h, arr, len(self.replay), C.byref(g)), "fk_graph_capture")
+        self.graph = g.value
+        return self.graph
+
+    def run_eager(self, token: int, offset: int):
+        """One token through the task list without a graph (verification path)."""
+        self.rt.state_set(token, offset)
+        self.rt.launch_batch(self.build_dispatches())
+        return self.rt.state_get()[0]
+
+    def decode_chunk(self, base_offset: int, seed_token: int, count: int):
+        """`count` greedy tokens with on-device token feedback; returns (tokens, gpu_seconds)."""
+        if not self.graph:
+            self.capture()
+        out = np.empty(count, np.uint32)
+        secs = C.c_double()
+        N.check(self.rt.L.fk_decode_chunk(self.rt.h, self.graph, base_offset, seed_token, count, out.ctypes.data, C.byref(secs)), "fk_decode_chunk")
+        return out, secs.value
+
+    def generate(self, seed_token: int, base_offset: int, max_tokens: int, chunk: int = FK_CHUNK):
+        """Greedy loop in chunks of `chunk` tokens (reference: _fast_generate_step)."""
+        toks, secs, tok, off = [], 0.0, seed_token, base_offset
+        while len(toks) < max_tokens:
+            n = min(chunk, max_tokens - len(toks))
+            out, t = self.decode_chunk(off, tok, n)
+            toks.extend(int(v) for v in out); secs += t; tok = int(out[-1]); off += n
+        return np.array(toks, np.uint32), secs
+
+    def generate_sampled(self, seed_token: int, base_offset: int, max_tokens: int, temperature: float = 1.0, top_k: int = 0,
+                         top_p: float = 1.0, seed: int = 0):
+        """Sampling beyond greedy, the way the reference does it: the fused step still runs on the GPU, the logits of every
+        step come back to the host and the sampler picks the next token there (the reference hands logits to mlx-lm's
+        sampler whenever the request is not greedy, python/fusekit_runtime/__init__.py:4782-4843).  Needs an engine created
+        with want_logits=True.  Returns the sampled tokens."""
+        if not self.logits:
+            raise N.FusekitError("sampling needs an engine created with want_logits=True")
+        rng = np.random.default_rng(seed)
+        toks, tok = [], int(seed_token)
+        for i in range(max_tokens):
+            self.decode_chunk(base_offset + i, tok, 1)
+            tok = sample_logits(self.last_logits(), temperature, top_k, top_p, rng)
+            toks.append(tok)
+        return np.array(toks, np.uint32)
+
+    def profile_nodes(self, repeats: int = 3):
+        if not self.graph:
+            self.capture()
+        n = len(self.replay)
+        out = (C.c_double * n)()
+        cnt = C.c_int()
+        N.check(self.rt.L.fk_graph_profile_nodes(self.rt.h, self.graph, repeats, out, n, C.byref(cnt)), "fk_graph_profile_nodes")
+        return [(self.replay[i].kind, self.replay[i].layer, out[i]) for i in range(n)]
+
+    def time_tasks(self, tasks, repeats: int = 5) -> float:
+        """Seconds per pass of `tasks` launched back to back (CUDA events on the library's stream)."""
+        arr = (N.Task * len(tasks))(*tasks)
+        secs = C.c_double()
+        N.check(self.rt.L.fk_time_tasks(self.rt.h, arr, len(tasks), repeats, C.byref(secs)), "fk_time_tasks")
+        return secs.value
+
+    def close(self):
+        self.rt.close()
+
+
+class DecodeEngine(EngineBase):
     """One model instance (or one tensor-parallel slice of it) resident on a GPU."""
 
     def __init__(self, spec: ModelSpec, capacity: int, device: int = 0, tp_rank: int = 0, tp_size: int = 1,
@@ -422,125 +561,6 @@ class DecodeEngine:
                     "o_buf": self.o_buf, "silu_up_digits": getattr(self, "act_digits", 0)}[p[1]]
         raise KeyError(f"unknown task-graph role {role!r}")
 
-    def dispatches_from(self, graph: dict) -> list:
-        """Resolve a task graph document (from task_graph.emit or read back from JSON) to the fk_task list, in
-        decode_pipeline order (the reference's replay order, src/codegen/task_graph_json.rs:1619-1664)."""
-        if graph.get("version") != task_graph.VERSION:
-            raise ValueError(f"task graph version {graph.get('version')} (this runtime reads {task_graph.VERSION})")
-        if graph.get("active_m", 1) != 1:
-            raise ValueError("only batch-1 decode graphs are dispatchable")
-        if not graph["decode_capabilities"]["dispatchable"]:
-            raise ValueError("task graph is not dispatchable: " + "; ".join(graph["decode_capabilities"]["reasons"]))
-        by_id = {t["id"]: t for t in graph["tasks"]}
-        out = []
-        for tid in graph["decode_pipeline"]:
-            t = by_id[tid]
-            bufs = {slot: self._resolve(role) for slot, role in task_graph.task_slots(t).items()}
-            out.append(N.Task.make(t["kind"], t.get("layer_idx", -1), bufs, t["iargs"], t["fargs"]))
-        return out
-
-    def role_table(self, graph: dict) -> list:
-        """(role, address-or-weight-id) for every explicit binding of the document: the table the library's own JSON reader
-        (fk_tasks_from_json / fk_graph_capture_json) resolves role strings through."""
-        roles = sorted({b["role"] for t in graph["tasks"] for b in t["extra_bindings"] if b["slot"] < 100})
-        return [(r, self._resolve(r)) for r in roles]
-
-    def dispatches_from_json(self, text: str, table=None) -> list:
-        """The fk_task list of a task_graph.json text as the library parses it (no Python between the file and the records)."""
-        import json
-        table = self.role_table(json.loads(text)) if table is None else table
-        L = N.lib()
-        arr = (N.RoleBinding * max(1, len(table)))(*[N.RoleBinding(r.encode(), int(v)) for r, v in table])
-        n = C.c_int32()
-        N.check(L.fk_tasks_from_json(text.encode(), arr, len(table), None, 0, C.byref(n)), "fk_tasks_from_json")
-        out = (N.Task * max(1, n.value))()
-        N.check(L.fk_tasks_from_json(text.encode(), arr, len(table), out, n.value, C.byref(n)), "fk_tasks_from_json")
-        return list(out)[: n.value]
-
-    def capture_json(self, text: str) -> int:
-        """Capture the decode step straight from a task_graph.json text (reference: load_dispatcher + build_icb,
-        python_runtime/src/lib.rs:115-169, 459-570)."""
-        import json
-        table = self.role_table(json.loads(text))
-        arr = (N.RoleBinding * len(table))(*[N.RoleBinding(r.encode(), int(v)) for r, v in table])
-        g = C.c_uint64()
-        N.check(self.rt.L.fk_graph_capture_json(self.rt.h, text.encode(), arr, len(table), C.byref(g)), "fk_graph_capture_json")
-        self.tasks = self.replay = self.dispatches_from_json(text, table)
-        self.graph = g.value
-        return self.graph
-
-    def build_dispatches(self) -> list:
-        """The per-token kernel list in replay order (reference order: embed -> per layer RmsNormQkv,
-        SDPA, LinearResidual, gate/up chain, LinearResidual -> final head -> argmax;
-        src/codegen/task_graph_json.rs:1619-1664, dispatch.py:3163-3611)."""
-        return self.dispatches_from(self.task_graph())
-
-    # ------------------------------------------------------------------ replay
-    def capture(self) -> int:
-        """Capture the per-token task list once as a CUDA graph (reference: build_icb, lib.rs:459-570)."""
-        self.tasks = self.replay = self.build_dispatches()
-        arr = (N.Task * len(self.replay))(*self.replay)
-        g = C.c_uint64()
-        N.check(self.rt.L.fk_graph_capture(self.rt.h, arr, len(self.replay), C.byref(g)), "fk_graph_capture")
-        self.graph = g.value
-        return self.graph
-
-    def run_eager(self, token: int, offset: int):
-        """One token through the task list without a graph (verification path)."""
-        self.rt.state_set(token, offset)
-        self.rt.launch_batch(self.build_dispatches())
-        return self.rt.state_get()[0]
-
-    def decode_chunk(self, base_offset: int, seed_token: int, count: int):
-        """`count` greedy tokens with on-device token feedback; returns (tokens, gpu_seconds)."""
-        if not self.graph:
-            self.capture()
-        out = np.empty(count, np.uint32)
-        secs = C.c_double()
-        N.check(self.rt.L.fk_decode_chunk(self.rt.h, self.graph, base_offset, seed_token, count, out.ctypes.data, C.byref(secs)), "fk_decode_chunk")
-        return out, secs.value
-
-    def generate(self, seed_token: int, base_offset: int, max_tokens: int, chunk: int = FK_CHUNK):
-        """Greedy loop in chunks of `chunk` tokens (reference: _fast_generate_step)."""
-        toks, secs, tok, off = [], 0.0, seed_token, base_offset
-        while len(toks) < max_tokens:
-            n = min(chunk, max_tokens - len(toks))
-            out, t = self.decode_chunk(off, tok, n)
-            toks.extend(int(v) for v in out); secs += t; tok = int(out[-1]); off += n
-        return np.array(toks, np.uint32), secs
-
-    def generate_sampled(self, seed_token: int, base_offset: int, max_tokens: int, temperature: float = 1.0, top_k: int = 0,
-                         top_p: float = 1.0, seed: int = 0):
-        """Sampling beyond greedy, the way the reference does it: the fused step still runs on the GPU, the logits of every
-        step come back to the host and the sampler picks the next token there (the reference hands logits to mlx-lm's
-        sampler whenever the request is not greedy, python/fusekit_runtime/__init__.py:4782-4843).  Needs an engine created
-        with want_logits=True.  Returns the sampled tokens."""
-        if not self.logits:
-            raise N.FusekitError("sampling needs an engine created with want_logits=True")
-        rng = np.random.default_rng(seed)
-        toks, tok = [], int(seed_token)
-        for i in range(max_tokens):
-            self.decode_chunk(base_offset + i, tok, 1)
-            tok = sample_logits(self.last_logits(), temperature, top_k, top_p, rng)
-            toks.append(tok)
-        return np.array(toks, np.uint32)
-
-    def profile_nodes(self, repeats: int = 3):
-        if not self.graph:
-            self.capture()
-        n = len(self.replay)
-        out = (C.c_double * n)()
-        cnt = C.c_int()
-        N.check(self.rt.L.fk_graph_profile_nodes(self.rt.h, self.graph, repeats, out, n, C.byref(cnt)), "fk_graph_profile_nodes")
-        return [(self.replay[i].kind, self.replay[i].layer, out[i]) for i in range(n)]
-
-    def time_tasks(self, tasks, repeats: int = 5) -> float:
-        """Seconds per pass of `tasks` launched back to back (CUDA events on the library's stream)."""
-        arr = (N.Task * len(tasks))(*tasks)
-        secs = C.c_double()
-        N.check(self.rt.L.fk_time_tasks(self.rt.h, arr, len(tasks), repeats, C.byref(secs)), "fk_time_tasks")
-        return secs.value
-
     def hidden_states(self) -> np.ndarray:
         """Residual stream after every layer of the last decoded token, [n_layers, H] bf16 bits."""
         s = self.spec
@@ -587,14 +607,11 @@ class DecodeEngine:
         self.tp_exchange = "allreduce"
         N.check(self.rt.L.fk_peer_arena_close(self.rt.h), "fk_peer_arena_close")
 
-    def close(self):
-        self.rt.close()
-
-
-def sample_logits(logits_bf16: np.ndarray, temperature: float = 1.0, top_k: int = 0, top_p: float = 1.0, rng=None) -> int:
-    """One token from bf16 logits (bit patterns): temperature scaling, then top-k and nucleus (top-p) filtering, then a draw.
+def sample_logits(logits: np.ndarray, temperature: float = 1.0, top_k: int = 0, top_p: float = 1.0, rng=None) -> int:
+    """One token from logits (float32 values, or uint16 bit patterns of bf16): temperature scaling, then top-k and nucleus (top-p) filtering, then a draw.
     temperature <= 0 or top_k == 1 is the greedy choice with ties to the lowest index, like the on-device argmax."""
-    x = (np.asarray(logits_bf16, np.uint16).astype(np.uint32) << 16).view(np.float32).astype(np.float64)
+    x = np.asarray(logits)
+    x = (x if x.dtype == np.float32 else (x.astype(np.uint16).astype(np.uint32) << 16).view(np.float32)).astype(np.float64)
     if temperature <= 0.0 or top_k == 1:
         return int(np.argmax(x))                  # first maximum = lowest index
     x = x / temperature
@@ -631,7 +648,10 @@ def comm_unique_id() -> bytes:
     return buf.raw
 
 
-def attach(spec: ModelSpec, capacity: int, device: int = 0, **kw) -> DecodeEngine:
+def attach(spec, capacity: int, device: int = 0, **kw) -> EngineBase:
     """Counterpart of ``fusekit_runtime.attach`` (python/fusekit_runtime/__init__.py:3101-3156):
-    returns an engine whose decode calls run on the CUDA runtime."""
+    returns an engine whose decode calls run on the CUDA runtime; the class follows the kind of ``spec``."""
+    if isinstance(spec, LayeredSpec):
+        from .layered import LayeredEngine
+        return LayeredEngine(spec, capacity, device, **kw)
     return DecodeEngine(spec, capacity, device, **kw)

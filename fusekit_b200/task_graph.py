@@ -17,10 +17,12 @@ from .model_spec import ModelSpec
 VERSION = 2
 KINDS = ["step_init", "embed_lookup_decode", "rmsnorm_qkv", "qk_norm_rope_store", "sdpa_decode", "linear_residual",
          "rmsnorm_gateup_act", "final_rmsnorm_lm_head", "argmax_finalize", "allreduce", "residual_add", "rmsnorm_rows",
-         "rope_store_rows", "argmax_rows", "kv_store_quant", "sdpa_decode_quant"]
+         "rope_store_rows", "argmax_rows", "kv_store_quant", "sdpa_decode_quant", "embed_rows", "residual_norm_rows", "linear_rows",
+         "qk_norm_store_rows", "attention_rows", "moe_route_rows", "norm_linear", "attention_decode", "moe_up", "moe_down", "argmax_row"]
 KERNEL = {k: "fusekit_" + k for k in KINDS}
 (K_STEP, K_EMBED, K_QKV, K_QKNORM, K_SDPA, K_LIN, K_GATEUP, K_HEAD, K_ARGMAX, K_ALLREDUCE, K_RESADD, K_NORMROWS, K_ROPEROWS,
- K_ARGMAXROWS, K_KVQ, K_SDPAQ) = range(16)
+ K_ARGMAXROWS, K_KVQ, K_SDPAQ, K_EMBEDROWS, K_RESNORM, K_LINROWS, K_QKSTORE, K_ATTROWS, K_ROUTE, K_NORMLIN, K_ATTDEC, K_MOEUP,
+ K_MOEDOWN, K_ARGMAXROW) = range(27)
 
 
 def _bf16_round(v: float) -> float:
@@ -162,9 +164,14 @@ def emit(spec: ModelSpec, capacity: int, tp_rank: int = 0, tp_size: int = 1, fus
         add(K_ALLREDUCE, -1, {0: "global_scratch.argmax_scratch"}, [1, 1])
         add(K_ARGMAX, -1, {4: "global_scratch.argmax_scratch"}, [1])
 
-    # ---- v2 envelope: tasks with bindings, a linear event chain, layer groups, the decode pipeline
     out_slots = {K_EMBED: [1], K_QKV: [4, 5, 6, 7, 8, 11], K_QKNORM: [0, 5, 6], K_SDPA: [3, 4, 5], K_LIN: [3, 4], K_GATEUP: [4, 5, 11],
                  K_HEAD: [3, 4, 5, 11], K_ARGMAX: [], K_ALLREDUCE: [0], K_RESADD: [2], K_KVQ: [0, 3, 4, 5, 6, 7, 8], K_SDPAQ: [3, 4, 5]}
+    return _envelope(tasks, out_slots, {"chip": "b200", "arch": "sm_100a", "tensor_parallel": tp_size, "rank": tp_rank, "bits": s.bits,
+                                        "launch": "grid and block sizes are chosen by the runtime from the SM count (plan_shape)"})
+
+
+def _envelope(tasks: list, out_slots: dict, target: dict) -> dict:
+    """The v2 document around a task list: tasks with bindings, a linear event chain, layer groups, the decode pipeline."""
     jtasks, groups = [], {}
     for i, t in enumerate(tasks):
         ins, outs, extra = [], [], []
@@ -177,8 +184,8 @@ def emit(spec: ModelSpec, capacity: int, tp_rank: int = 0, tp_size: int = 1, fus
                 ins.append({"role": "scratch", "scratch_id": slot, "role_name": role})
             extra.append({"slot": slot, "role": role})
         if t["kind"] not in (K_ALLREDUCE, K_RESADD):
-            extra += [{"slot": 100, "role": "token_id_in" if t["kind"] == K_EMBED else "layer_offset"}]
-        if t["kind"] in (K_HEAD, K_ARGMAX):
+            extra += [{"slot": 100, "role": "token_id_in" if t["kind"] in (K_EMBED, K_EMBEDROWS) else "layer_offset"}]
+        if t["kind"] in (K_HEAD, K_ARGMAX) or (t["kind"] == K_NORMLIN and 9 in t["bufs"]):
             extra += [{"slot": 101, "role": "next_token_out"}]
         jt = {"id": i, "fusion_id": i, "kernel": KERNEL[KINDS[t["kind"]]], "kind": t["kind"], "grid_threads": [0, 1, 1], "threadgroup": [0, 1, 1],
               "inputs": ins, "outputs": outs, "extra_bindings": extra, "depends_on": [i - 1] if i else [], "trigger_event": i,
@@ -186,7 +193,7 @@ def emit(spec: ModelSpec, capacity: int, tp_rank: int = 0, tp_size: int = 1, fus
         if t["layer"] >= 0:
             jt["layer_idx"] = t["layer"]
         jtasks.append(jt)
-        region = "embed" if t["kind"] == K_EMBED else (f"layer.{t['layer']}" if t["layer"] >= 0 else "post")
+        region = "embed" if t["kind"] in (K_EMBED, K_EMBEDROWS) else (f"layer.{t['layer']}" if t["layer"] >= 0 else "post")
         groups.setdefault(region, []).append(i)
     return {
         "version": VERSION, "active_m": 1, "tasks": jtasks,
@@ -195,9 +202,119 @@ def emit(spec: ModelSpec, capacity: int, tp_rank: int = 0, tp_size: int = 1, fus
         "layer_groups": [{"region": r, "task_ids": ids} for r, ids in groups.items()],
         "decode_pipeline": list(range(len(jtasks))),
         "decode_capabilities": {"dispatchable": True, "reasons": []},
-        "target": {"chip": "b200", "arch": "sm_100a", "tensor_parallel": tp_size, "rank": tp_rank, "bits": s.bits,
-                   "launch": "grid and block sizes are chosen by the runtime from the SM count (plan_shape)"},
+        "target": target,
     }
+
+
+# ------------------------------------------------------------------ layered decoders (model_spec.LayeredSpec)
+def round_up(v: int, m: int) -> int:
+    return (v + m - 1) // m * m
+
+
+def _task(tasks, kind, layer, bufs, iargs, fargs=()):
+    tasks.append({"kind": kind, "layer": layer, "bufs": {int(k): v for k, v in bufs.items() if v}, "iargs": [int(v) for v in iargs],
+                  "fargs": [float(v) for v in fargs]})
+
+
+def key_splits(mixer, capacity: int, sm: int) -> int:
+    """Blocks the keys of a decode step are split over: two blocks per SM over all kv heads, at least 64 keys of capacity each."""
+    tiles = -(-(mixer.heads // mixer.kv_heads * mixer.maps) // 8)
+    return max(1, min(-(-2 * sm // (mixer.kv_heads * tiles)), -(-capacity // 64), 8 * round_up(mixer.vdim, 8), 256))
+
+
+def layered_decode_tasks(spec, capacity: int, lambdas: dict, dtype: int = 0, sm: int = 148) -> list:
+    """One decoded position: per layer run q|k|v|gate projection (previous sublayer's post-norm, residual add and this one's
+    pre-norm in its prologue), attention with the q/k norm and the cache store in its prologue, output projection, router and
+    shared up-projection in one product, the chosen experts' up- and down-projections; then the head with the greedy choice."""
+    D, eps, t = spec.hidden, spec.eps, []
+    x = lambda r: f"global_scratch.x_in.{r}"
+    _task(t, K_EMBEDROWS, -1, {0: "param.embed_tokens", 1: x(0)}, [D, 1, spec.vocab])
+    cur, pend, post = x(0), None, None
+    for run, (i, again) in enumerate(spec.runs()):
+        m, f, lp = spec.layers[i].mixer, spec.layers[i].mlp, f"layer_param.{i}."
+        xo = x(run) if run else None
+        _task(t, K_NORMLIN, run, {0: cur, 1: pend, 2: post, 3: x(0) if again else None, 4: xo, 5: lp + "norm1", 6: lp + "mix.qkvg", 7: "layer_scratch.qkvg"},
+              [D, m.rows, 0, 0], [eps])
+        cur = xo or cur
+        _task(t, K_ATTDEC, run, {0: "layer_scratch.qkvg", 1: lp + "mix.q.norm", 2: lp + "mix.k.norm", 3: f"layer_cache_k.{run}", 4: f"layer_cache_v.{run}",
+                                 5: "layer_scratch.attention", 6: "global_scratch.attention_partials", 7: "global_scratch.attention_counters"},
+              [m.heads, m.kv_heads, m.dim, m.vdim, capacity, 1, dtype | m.maps << 8, key_splits(m, capacity, sm)], [m.scale, lambdas[i], m.diff or 0.0, eps])
+        _task(t, K_NORMLIN, run, {0: "layer_scratch.attention", 6: lp + "mix.o", 7: "layer_scratch.mixer_out"}, [m.heads * m.vdim, D, 0, 0], [eps])
+        pend, post = "layer_scratch.mixer_out", lp + "norm1b"
+        if f is None:
+            continue
+        act = 2
+        _task(t, K_NORMLIN, run, {0: cur, 1: pend, 2: post, 4: f"layer_scratch.{run}.h_attn", 5: lp + "norm2", 6: lp + "mlp.router_shared",
+                                  7: "layer_scratch.router_shared", 8: "layer_scratch.ff_in"}, [D, f.experts + f.shared_ff, act, f.experts], [eps])
+        cur = f"layer_scratch.{run}.h_attn"
+        _task(t, K_MOEUP, run, {0: "layer_scratch.router_shared", 1: "layer_scratch.ff_in", 2: lp + "mlp.experts_up", 3: "layer_scratch.expert_act",
+                                4: "layer_scratch.chosen", 5: "layer_scratch.chosen_weight"}, [D, f.experts, f.top, f.ff, act])
+        _task(t, K_MOEDOWN, run, {0: "layer_scratch.expert_act", 1: "layer_scratch.chosen", 2: "layer_scratch.chosen_weight", 3: lp + "mlp.experts_down",
+                                  4: f"layer_scratch.shared_act.{i}" if f.shared_ff else None, 5: lp + "mlp.shared_down" if f.shared_ff else None,
+                                  6: "layer_scratch.ff_out"}, [D, f.experts, f.top, f.ff, f.shared_ff])
+        pend, post = "layer_scratch.ff_out", lp + "norm2b"
+    _task(t, K_NORMLIN, -1, {0: cur, 1: pend, 2: post, 4: x(len(spec.runs())), 5: "param.final_norm", 6: "param.lm_head", 7: "global_scratch.logits",
+                             9: "global_scratch.argmax_scratch", 10: "global_scratch.head_counter"}, [D, spec.vocab, 0, 0], [eps])
+    return t
+
+
+def layered_rows_tasks(spec, capacity: int, lambdas: dict, rows: int, wanted: int, greedy: bool, dtype: int = 0) -> list:
+    """``rows`` consecutive positions: the same layers on row kernels; logits of the ``wanted`` rows of the index buffer, and with
+    ``greedy`` the token after the first of them (the position then advances by ``rows``)."""
+    D, V, M, eps, t = spec.hidden, spec.vocab, rows, spec.eps, []
+    ld = round_up(D, 64)
+    emb, xb, h = "rows_scratch.embedding", "rows_scratch.x", "rows_scratch.h"
+    _task(t, K_EMBEDROWS, -1, {0: "param.embed_tokens", 1: emb, 2: "rows_scratch.tokens"}, [D, M, V])
+    cur, pend, post, top = emb, {}, None, 0
+
+    def linear(run, x, w, y, n, ldx, ldy, act=0, row0=0, f32=0, m=M, grouped=None, experts=0):
+        _task(t, K_LINROWS, run, {0: x, 1: w, 2: y, 3: grouped}, [m, row0, n, ldx, ldy, dtype, act | f32 << 8, experts])
+
+    for run, (i, again) in enumerate(spec.runs()):
+        m, f, lp = spec.layers[i].mixer, spec.layers[i].mlp, f"layer_param.{i}."
+        _task(t, K_RESNORM, run, {0: cur, 2: post, 3: emb if again else None, 4: xb if run else None, 5: lp + "norm1", 6: h, **pend},
+              [D, M, dtype, ld, top, ld], [eps])
+        cur = xb if run else cur
+        ldq, ldo = round_up(m.rows, 64), round_up(m.heads * m.vdim, 64)
+        linear(run, h, lp + "mix.qkvg", "rows_scratch.qkvg", m.rows, ld, ldq)
+        _task(t, K_QKSTORE, run, {0: "rows_scratch.qkvg", 1: lp + "mix.q.norm", 2: lp + "mix.k.norm", 3: "rows_scratch.q", 4: f"layer_cache_k.{run}", 5: f"layer_cache_v.{run}"},
+              [m.heads, m.kv_heads, m.dim, m.vdim, capacity, M, dtype | m.maps << 8, ldq], [eps])
+        _task(t, K_ATTROWS, run, {0: "rows_scratch.q", 1: f"layer_cache_k.{run}", 2: f"layer_cache_v.{run}", 3: "rows_scratch.attention", 4: f"rows_scratch.gate.{i}"},
+              [m.heads, m.kv_heads, m.dim, m.vdim, capacity, M, dtype | m.maps << 8, ldq], [m.scale, lambdas[i], m.diff or 0.0, eps])
+        linear(run, "rows_scratch.attention", lp + "mix.o", "rows_scratch.y", D, ldo, ld)
+        pend, post, top = {1: "rows_scratch.y"}, lp + "norm1b", 0
+        if f is None:
+            continue
+        _task(t, K_RESNORM, run, {0: cur, 2: post, 4: xb, 5: lp + "norm2", 6: h, **pend}, [D, M, dtype, ld, 0, ld], [eps])
+        cur, act, lde, lds, lff = xb, 2, round_up(f.experts, 64), round_up(max(f.shared_ff, 1), 64), round_up(f.ff, 64)
+        linear(run, h, lp + "mlp.router_shared", "rows_scratch.router", f.experts, ld, lde, f32=1)
+        _task(t, K_ROUTE, run, {0: "rows_scratch.router", 1: h, 2: "rows_scratch.chosen_weight", 3: "rows_scratch.chosen", 4: "rows_scratch.rank", 5: "rows_scratch.count",
+                                6: "rows_scratch.slot", 7: "rows_scratch.offsets", 8: "rows_scratch.h_grouped"}, [M, f.experts, f.top, lde, ld, dtype])
+        linear(run, "rows_scratch.h_grouped", lp + "mlp.experts_up", "rows_scratch.act_grouped", f.ff, ld, lff, act=act, m=M * f.top,
+               grouped="rows_scratch.offsets", experts=f.experts)
+        linear(run, "rows_scratch.act_grouped", lp + "mlp.experts_down", "rows_scratch.y_grouped", D, lff, ld, m=M * f.top, grouped="rows_scratch.offsets",
+               experts=f.experts)
+        pend = {8: "rows_scratch.y_grouped", 9: "rows_scratch.slot", 10: "rows_scratch.chosen_weight"}
+        if f.shared_ff:
+            linear(run, h, lp + "mlp.router_shared", "rows_scratch.shared_act", f.shared_ff, ld, lds, act=act, row0=f.experts)
+            linear(run, "rows_scratch.shared_act", lp + "mlp.shared_down", "rows_scratch.y", D, lds, ld)
+            pend[1] = "rows_scratch.y"
+        post, top = lp + "norm2b", f.top
+    if wanted:
+        _task(t, K_RESNORM, -1, {0: cur, 2: post, 5: "param.final_norm", 6: "rows_scratch.h_wanted", 7: "rows_scratch.index", **pend},
+              [D, wanted, dtype, ld, top, ld], [eps])
+        linear(-1, "rows_scratch.h_wanted", "param.lm_head", "rows_scratch.logits", V, ld, V, f32=1, m=wanted)
+        if greedy:
+            _task(t, K_ARGMAXROW, -1, {0: "rows_scratch.logits"}, [V, M])
+    return t
+
+
+def emit_layered(spec, capacity: int, lambdas: dict, dtype: int = 0, sm: int = 148) -> dict:
+    """The decode step of a layered decoder as a v2 document (``lambdas``: layer -> combination constant of its two maps)."""
+    out_slots = {K_EMBEDROWS: [1], K_NORMLIN: [4, 7, 8, 9, 10], K_ATTDEC: [3, 4, 5, 6, 7], K_MOEUP: [3, 4, 5], K_MOEDOWN: [6]}
+    return _envelope(layered_decode_tasks(spec, capacity, lambdas, dtype, sm), out_slots,
+                     {"chip": "b200", "arch": "sm_100a", "tensor_parallel": 1, "rank": 0, "bits": 32 if dtype else 16,
+                      "launch": "grid and block sizes are chosen by the runtime from the SM count"})
 
 
 def task_slots(jtask: dict) -> dict:

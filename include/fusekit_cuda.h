@@ -55,11 +55,25 @@ enum {
     FK_TASK_ARGMAX_ROWS = 13,          /* batch: greedy token of every sequence + position advance (argmax_logits_scan.rs:83-124) */
     FK_TASK_KV_STORE_QUANT = 14,       /* kernels/rope_kv_cache_store_decode_quant.rs (fused form rmsnorm_qkv.rs:435-612): RoPE + quantised KV store */
     FK_TASK_SDPA_DECODE_QUANT = 15,    /* kernels/sdpa_decode_quant.rs:301-680: attention over the quantised cache */
-    FK_TASK_KIND_COUNT = 16
+    /* layered decoders (no reference counterpart): fp32 residual, differential attention, mixture of experts, looped layers */
+    FK_TASK_EMBED_ROWS = 16,
+    FK_TASK_RESIDUAL_NORM_ROWS = 17,
+    FK_TASK_LINEAR_ROWS = 18,
+    FK_TASK_QK_NORM_STORE_ROWS = 19,
+    FK_TASK_ATTENTION_ROWS = 20,
+    FK_TASK_MOE_ROUTE_ROWS = 21,
+    FK_TASK_NORM_LINEAR = 22,
+    FK_TASK_ATTENTION_DECODE = 23,
+    FK_TASK_MOE_UP = 24,
+    FK_TASK_MOE_DOWN = 25,
+    FK_TASK_ARGMAX_ROW = 26,
+    FK_TASK_KIND_COUNT = 27
 };
 
 /* activation selector for FK_TASK_RMSNORM_GATEUP_ACT */
 enum { FK_ACT_SWIGLU = 0, FK_ACT_GEGLU_TANH = 1 };
+/* activation selector of the layered decoders' products: none, square of relu */
+enum { FK_ACT_NONE = 0, FK_ACT_RELU_SQUARED = 2 };
 
 /*
  * One entry of the per-token dispatch list (reference: the (kernel, buffers,
@@ -136,6 +150,38 @@ enum { FK_ACT_SWIGLU = 0, FK_ACT_GEGLU_TANH = 1 };
  *                      shapes, python/fusekit_runtime/__init__.py:2825-2850, src/commands/patch.rs:112-152) sharing one cache
  *                      [n_kv, capacity, hd]; row m attends keys 0 .. offset + m.  ARGMAX_ROWS i2: positions the step advances
  *                      by (default 1; M for such a chunk)
+ * Layered decoders.  A = bf16 or (dtype = 1) fp32 activations; weights are dense rows kept as uploaded (fk_weight_keep_rows), K
+ * padded with zeros to a multiple of 64; `maps` = 2 for differential attention (two sub-heads per head), else 1; dpad / vpad =
+ * dim / vdim rounded up to 8.  ROWS tasks work on M consecutive positions offset .. offset + M - 1 of one sequence.
+ * EMBED_ROWS           buf0 table T[V,D]  buf1 x f32[M,D]  buf2 token ids u32[M] | 0 (the decode state's)   i0 D  i1 M  i2 V
+ * RESIDUAL_NORM_ROWS   x' = x + norm(y) * post (+ add), h = norm(x') * w.  buf0 x f32[M,D]  buf1 y A[M,ldy]|0  buf2 post T[D]
+ *                      buf3 add f32[M,D]|0  buf4 x' out|0 (may be buf0)  buf5 w T[D]  buf6 h A[M,ldh]  buf7 row index u32|0 (output
+ *                      row r is input row index[r])  buf8 grouped expert rows A[M*top,ldy]|0  buf9 slots  buf10 expert weights
+ *                      (y += sum_j weight[j] * buf8[slot[j]])   i0 D  i1 output rows  i2 dtype  i3 ldh  i4 top  i5 ldy   f0 eps
+ * LINEAR_ROWS          buf0 x A[M,ldx]  buf1 weight  buf2 y [M,ldy]  buf3 expert offsets i32[E+1]|0 (rows grouped by expert, weight
+ *                      rows e*N ..)   i0 M  i1 first weight row  i2 N  i3 ldx  i4 ldy  i5 dtype  i6 act | 256 (y is fp32)  i7 E
+ * QK_NORM_STORE_ROWS   buf0 q|k|v rows A[M,ld]  buf1 q norm T[dim]  buf2 k norm  buf3 q out A[M,H*maps,dpad]  buf4 cache k
+ *                      A[G*maps,capacity,dpad]  buf5 cache v A[G,capacity,vpad]   i0 H  i1 G  i2 dim  i3 vdim  i4 capacity  i5 M
+ *                      i6 dtype | maps << 8  i7 ld   f0 eps
+ * ATTENTION_ROWS       causal attention of M positions.  buf0 q  buf1 cache k  buf2 cache v  buf3 out A[M, round64(H*vdim)]  buf4 gate
+ *                      logits A|0   i0..i6 as above  i7 ld of the gate rows   f0 scale  f1 lambda  f2 diff  f3 eps
+ * MOE_ROUTE_ROWS       buf0 router logits f32[M,ldl]  buf1 h A[M,ld]  buf2 weights f32[M*top] out  buf3 experts i32 out  buf4 ranks i32
+ *                      out  buf5 counts i32[E]  buf6 slots i32 out  buf7 offsets i32[E+1] out  buf8 h rows grouped by expert A[M*top,ld]
+ *                      i0 M  i1 E  i2 top  i3 ldl  i4 ld  i5 dtype
+ * NORM_LINEAR          one row, fp32 activations: y = act(W h), h = norm(x') * w with x' as in RESIDUAL_NORM_ROWS, or h = x when buf5 = 0.
+ *                      buf0 x f32[K]  buf1 pending y f32|0  buf2 post  buf3 add|0  buf4 x' out|0 (not buf0)  buf5 w|0  buf6 weight
+ *                      buf7 y f32[N]  buf8 h out f32|0  buf9 argmax scratch u64[2*SMs]|0  buf10 counter   i0 K  i1 N  i2 act  i3 first row with
+ *                      act   f0 eps      (with buf9 the last block picks the greedy token of y and advances the decode state)
+ * ATTENTION_DECODE     one position: q/k norm, cache store, attention.  buf0 q|k|v|gate f32  buf1 q norm  buf2 k norm  buf3 cache k
+ *                      buf4 cache v  buf5 out f32[H*vdim]  buf6 partials f32  buf7 counters (zero before first use)   i0 H  i1 G  i2 dim
+ *                      i3 vdim  i4 capacity  i5 gate present  i6 dtype | maps << 8 (dtype of the caches)  i7 key splits
+ *                      partials: G * ceil(H/G*maps/8) * splits * 8 * (vpad + 2) floats   f0 scale  f1 lambda  f2 diff  f3 eps
+ * MOE_UP               buf0 router logits f32[E]  buf1 h f32[D]  buf2 weight [E*ff, D]  buf3 act out f32[top*ff]  buf4 chosen i32 out
+ *                      buf5 weights f32 out   i0 D  i1 E  i2 top  i3 ff  i4 act
+ * MOE_DOWN             buf0 act f32[top*ff]  buf1 chosen  buf2 weights  buf3 weight [E*D, ff]  buf4 shared act f32|0  buf5 shared weight [D, ffs]
+ *                      buf6 y f32[D]   i0 D  i1 E  i2 top  i3 ff  i4 ffs
+ * ARGMAX_ROW           buf0 logits f32[V]   i0 V  i1 positions to advance by
+ *
  * Batch decode (M = 2..16 independent sequences at one position): EMBED with i1 = M, LINEAR_RESIDUAL / RMSNORM_GATEUP_ACT
  * with their row counts, SDPA_DECODE with i5 = M (q and out T[M, n_q*hd], caches [M, n_kv, capacity, hd]).
  */
@@ -186,6 +232,8 @@ fk_status fk_weight_set_rows(fk_handle h, fk_weight w, int kind, int head_dim, i
 /* Freezes the object; 4- and 8-bit rows are repacked into the streaming layout (16 rows x 8 groups per
  * 4608-byte unit, lane-ordered) and the MLX-layout copy is released. */
 fk_status fk_weight_finalize(fk_handle h, fk_weight w);
+/* Freezes a dense (16-bit) object as the rows it was uploaded as: the form the layered decoders' tasks read. */
+fk_status fk_weight_keep_rows(fk_handle h, fk_weight w);
 /* Interleaves a gate and an up projection (same shape, not yet finalized) into one weight whose tiles hold
  * 8 gate rows and the 8 matching up rows; consumes both inputs.  RMSNORM_GATEUP_ACT takes it in buf2 (buf3 0). */
 fk_status fk_weight_pair(fk_handle h, fk_weight gate, fk_weight up, fk_weight *out);
