@@ -1,6 +1,8 @@
 // Host side of the layered decoders' kernels: argument checks and launches, one case per task kind.
 #include "fk_layers.h"
 #include "fk_layers.cuh"
+#include "fk_gemm_tc.cuh"
+#include "fk_flash.cuh"
 #include <stdarg.h>
 #include <stdio.h>
 #include <string.h>
@@ -23,6 +25,8 @@ static cudaError_t launch(FklEnv &c, void (*kern)(KA...), dim3 grid, dim3 block,
     ++*c.launches;
     return cudaLaunchKernelEx(&cfg, kern, KA(args)...);
 }
+#define FKL_FLASH_MIN_ROWS 8          // up to this many positions one block per (position, kv head) on CUDA cores does better
+
 // CALL with VPL = values per lane of the attention kernel (a power of two covering vpad)
 #define VPL_SWITCH(vpad, CALL)                                   \
     do {                                                         \
@@ -41,6 +45,12 @@ cudaError_t fkl_init() {
     ATT(1); ATT(2); ATT(4); ATT(8); ATT(16);
     TRY(big_smem(k_residual_norm_rows<uint16_t>)); TRY(big_smem(k_residual_norm_rows<float>));
     TRY(big_smem(k_gemv<FKL_GV_LINEAR>)); TRY(big_smem(k_gemv<FKL_GV_MOE_UP>)); TRY(big_smem(k_gemv<FKL_GV_MOE_DOWN>));
+    TRY(cudaFuncSetAttribute(k_gemm_tc<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TcTile<64>::SMEM));
+    TRY(cudaFuncSetAttribute(k_gemm_tc<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TcTile<128>::SMEM));
+    TRY(cudaFuncSetAttribute(k_gemm_tc<256>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TcTile<256>::SMEM));
+#define FL(KD) TRY(big_smem(k_flash_rows<KD, 64>)); TRY(big_smem(k_flash_rows<KD, 128>)); TRY(big_smem(k_flash_rows<KD, 256>))
+    FL(32); FL(64); FL(128);
+#undef FL
 #undef ATT
 #undef TRY
     return e;
@@ -64,6 +74,36 @@ static cudaError_t launch_gemv(FklEnv &c, int mode, GemvArgs &a) {
     if (mode == FKL_GV_LINEAR) return launch(c, k_gemv<FKL_GV_LINEAR>, g, b, smem, c.state, a);
     if (mode == FKL_GV_MOE_UP) return launch(c, k_gemv<FKL_GV_MOE_UP>, g, b, smem, c.state, a);
     return launch(c, k_gemv<FKL_GV_MOE_DOWN>, g, b, smem, c.state, a);
+}
+// bf16 rows [rows, k] (row stride ld elements) in boxes of 64 columns x box_rows, 128-byte swizzle
+typedef CUresult (*EncodeTiled)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *, const cuuint32_t *, const cuuint32_t *,
+                                CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
+static bool tensor_map(CUtensorMap *m, const void *p, long long rows, long long k, long long ld, int box_rows) {
+    static EncodeTiled fn = nullptr;
+    if (!fn) {
+        void *f = nullptr; cudaDriverEntryPointQueryResult qr;
+        if (cudaGetDriverEntryPointByVersion("cuTensorMapEncodeTiled", &f, 12000, cudaEnableDefault, &qr) != cudaSuccess || qr != cudaDriverEntryPointSuccess) return false;
+        fn = (EncodeTiled)f;
+    }
+    const cuuint64_t dims[2] = {(cuuint64_t)k, (cuuint64_t)rows}, strides[1] = {(cuuint64_t)ld * 2};
+    const cuuint32_t box[2] = {FKL_TC_BK, (cuuint32_t)box_rows}, es[2] = {1, 1};
+    return fn(m, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, (void *)p, dims, strides, box, es, CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+              CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+// the widest tile that still gives (almost) every SM one
+static int tc_tile(int sm, long long mtiles, int n) {
+    if (mtiles * ((n + 255) / 256) * 10 >= sm * 9) return 256;
+    if (mtiles * ((n + 127) / 128) * 10 >= sm * 7) return 128;
+    return 64;
+}
+template <int BN> static cudaError_t launch_tc(FklEnv &c, int grid, const CUtensorMap &mx, const CUtensorMap &mw, const TcGemmArgs &a) {
+    return launch(c, k_gemm_tc<BN>, dim3(grid), dim3(FKL_TC_THREADS), TcTile<BN>::SMEM, c.state, mx, mw, a);
+}
+template <int KD> static cudaError_t launch_flash(FklEnv &c, const FlashArgs &a) {
+    const dim3 g(a.H, (a.rows + 63) / 64), b(128 * a.maps);
+    if (a.vdim <= 64) return launch(c, k_flash_rows<KD, 64>, g, b, flash_smem_bytes<KD, 64>(a.maps), c.state, a);
+    if (a.vdim <= 128) return launch(c, k_flash_rows<KD, 128>, g, b, flash_smem_bytes<KD, 128>(a.maps), c.state, a);
+    return launch(c, k_flash_rows<KD, 256>, g, b, flash_smem_bytes<KD, 256>(a.maps), c.state, a);
 }
 static bool gv_fits(int nchunks) { return nchunks > 0 && gv_smem_bytes(nchunks) <= 200 * 1024; }
 
@@ -94,10 +134,22 @@ fk_status fkl_run(FklEnv &c, const fk_task &t, char *err, size_t ecap) {
         if (!c.weight(c.owner, b[1], &w)) return bad(err, ecap, "linear_rows: weight missing or not kept as rows");
         if (!b[0] || !b[2] || M <= 0 || N <= 0 || row0 < 0 || ldx < w.k || ldx % 8 || ldy < N || (b[3] && E <= 0)) return bad(err, ecap, "linear_rows: bad arguments");
         if (b[3] ? w.n != (long long)E * N : row0 + N > w.n) return bad(err, ecap, "linear_rows: shape mismatch");
-        LinRowsArgs a{(const void *)b[0], w.rows + (size_t)row0 * w.k, (void *)b[2], (const int *)b[3], M, N, (int)w.k, ldx, (int)w.k, ldy, act, outf};
+        if (!f32) {           // tensor cores
+            if (ldx % 64 || (b[0] & 15)) return bad(err, ecap, "linear_rows: bf16 rows need a stride in multiples of 64 and 16-byte alignment");
+            TcGemmArgs a{(void *)b[2], (const int *)b[3], M, N, (int)(w.k / FKL_TC_BK), row0, ldy, act, outf, E};
+            const long long mt = b[3] ? (M < E ? M : E) + M / 128 : (M + 127) / 128;
+            const int bn = tc_tile(c.sm_count, mt, N);
+            const long long tiles = mt * ((N + bn - 1) / bn);
+            const int grid = tiles < c.sm_count ? (int)tiles : c.sm_count;
+            CUtensorMap mx, mw;
+            if (!tensor_map(&mx, (const void *)b[0], M, w.k, ldx, 128) || !tensor_map(&mw, w.rows, w.n, w.k, w.k, bn)) return bad(err, ecap, "linear_rows: tensor map refused");
+            e = bn == 256 ? launch_tc<256>(c, grid, mx, mw, a) : bn == 128 ? launch_tc<128>(c, grid, mx, mw, a) : launch_tc<64>(c, grid, mx, mw, a);
+            break;
+        }
+        LinRowsArgs a{(const float *)b[0], w.rows + (size_t)row0 * w.k, (float *)b[2], (const int *)b[3], M, N, (int)w.k, ldx, (int)w.k, ldy, act};
         const dim3 g((N + 63) / 64, (M + 63) / 64, b[3] ? E : 1);
         if (g.y > 65535 || g.z > 65535) return bad(err, ecap, "linear_rows: too many rows");
-        e = f32 ? launch(c, k_linear_rows<float>, g, dim3(256), 0, (const FkState *)c.state, a) : launch(c, k_linear_rows<uint16_t>, g, dim3(256), 0, (const FkState *)c.state, a);
+        e = launch(c, k_linear_rows, g, dim3(256), 0, (const FkState *)c.state, a);
         break;
     }
     case FK_TASK_QK_NORM_STORE_ROWS: {
@@ -136,6 +188,12 @@ fk_status fkl_run(FklEnv &c, const fk_task &t, char *err, size_t ecap) {
             for (int q = 0; q < 4; ++q) if (!b[q]) return bad(err, ecap, "attention_rows: missing buffer %d", q);
             a.q = (const void *)b[0]; a.ck = (void *)b[1]; a.cv = (void *)b[2]; a.out = (void *)b[3]; a.gate = (const void *)b[4];
             a.ldo = round_up(a.H * a.vdim, 64); a.ldg = i[7];
+            if (!f32 && rows > FKL_FLASH_MIN_ROWS && a.dim <= 128 && a.vdim <= 256) {
+                FlashArgs fa{(const uint16_t *)a.q, (const uint16_t *)a.ck, (const uint16_t *)a.cv, (const uint16_t *)a.gate, (uint16_t *)a.out, a.H, a.G, a.maps, a.vdim,
+                             a.dpad, a.vpad, a.cap, a.ldo, a.ldg, rows, a.scale, a.lambda, a.diff, a.eps};
+                e = a.dim <= 32 ? launch_flash<32>(c, fa) : a.dim <= 64 ? launch_flash<64>(c, fa) : launch_flash<128>(c, fa);
+                break;
+            }
             const dim3 g(1, a.G * a.tiles, rows), blk(FKL_ATT_WARPS * 32);
             if (f32) VPL_SWITCH(a.vpad, e = launch(c, (k_attention<float, float, VPL, false>), g, blk, smem, c.state, a));
             else VPL_SWITCH(a.vpad, e = launch(c, (k_attention<uint16_t, uint16_t, VPL, false>), g, blk, smem, c.state, a));

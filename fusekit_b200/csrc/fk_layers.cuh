@@ -87,8 +87,7 @@ __global__ void __launch_bounds__(512) k_residual_norm_rows(const FkState *st, R
 // ---------------------------------------------------------------- matrix product on rows, CUDA cores
 // Y[m, n] = act(sum_k X[m, k] W[row0 + n, k]); with `offsets` the rows of X are grouped by expert (expert e owns rows
 // offsets[e] .. offsets[e + 1] - 1 and the weight rows e * N ..).  fp32 arithmetic: the product of the 32-bit mode.
-struct LinRowsArgs { const void *x; const uint16_t *w; void *y; const int *offsets; int m, n, k, ldx, ldw, ldy, act, out_f32; };
-template <typename T>
+struct LinRowsArgs { const float *x; const uint16_t *w; float *y; const int *offsets; int m, n, k, ldx, ldw, ldy, act; };
 __global__ void __launch_bounds__(256) k_linear_rows(const FkState *st, LinRowsArgs a) {
     __shared__ float As[16][68], Bs[16][68];
     pdl_wait(); pdl_launch_dependents();
@@ -105,7 +104,7 @@ __global__ void __launch_bounds__(256) k_linear_rows(const FkState *st, LinRowsA
         const int mr = m0 + lr, nr = n0 + lr;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-            As[lk + j][lr] = mr < mend ? ldT((const T *)a.x + (size_t)mr * a.ldx + k0 + lk + j) : 0.0f;
+            As[lk + j][lr] = mr < mend ? a.x[(size_t)mr * a.ldx + k0 + lk + j] : 0.0f;
             Bs[lk + j][lr] = nr < a.n ? bf2f(w[(size_t)nr * a.ldw + k0 + lk + j]) : 0.0f;
         }
         __syncthreads();
@@ -123,8 +122,7 @@ __global__ void __launch_bounds__(256) k_linear_rows(const FkState *st, LinRowsA
     for (int i = 0; i < 4; ++i) for (int j = 0; j < 4; ++j) {
         const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
         if (m >= mend || n >= a.n) continue;
-        const float v = act_apply(acc[i][j], a.act);
-        if (a.out_f32) ((float *)a.y)[(size_t)m * a.ldy + n] = v; else stT((T *)a.y + (size_t)m * a.ldy + n, v);
+        a.y[(size_t)m * a.ldy + n] = act_apply(acc[i][j], a.act);
     }
 }
 

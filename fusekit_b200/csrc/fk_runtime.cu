@@ -79,6 +79,7 @@ struct Weight {
 struct Graph {
     std::vector<fk_task> tasks;
     cudaGraph_t graph = nullptr; cudaGraphExec_t exec = nullptr;
+    uint32_t vocab = 0;                         // rows of the embedding table this graph looks tokens up in (0 = unknown)
 };
 struct Ctx {
     int device = 0; bool open = false;
@@ -557,7 +558,6 @@ static bool rows_weight(void *owner, uint64_t id, FklWeight *out) {
 static fk_status run_task(Ctx *c, const fk_task &t, const Weight *nextw = nullptr) {
     if (fkl_owns(t.kind)) {
         FklEnv env{c->stream, c->pdl, c->sm_count, c->state, c->history, &c->launches, c, rows_weight};
-        if (t.kind == FK_TASK_EMBED_ROWS && t.iarg[2] > 0) c->vocab = (uint32_t)t.iarg[2];
         char err[256] = "";
         fk_status s = fkl_run(env, t, err, sizeof err);
         return s ? fail(s, "%s", err) : FK_OK;
@@ -936,6 +936,8 @@ extern "C" fk_status fk_graph_capture(fk_handle h, const fk_task *tasks, int n, 
     CU(e);
     CU(cudaGraphInstantiate(&g.exec, g.graph, 0));
     CU(cudaGraphUpload(g.exec, c->stream));
+    for (const fk_task &t : g.tasks)
+        if ((t.kind == FK_TASK_EMBED_LOOKUP_DECODE || t.kind == FK_TASK_EMBED_ROWS) && t.iarg[2] > 0) g.vocab = (uint32_t)t.iarg[2];
     c->graphs.push_back(g); *out = c->graphs.size();
     return FK_OK;
 }
@@ -1128,6 +1130,7 @@ extern "C" fk_status fk_decode_chunk(fk_handle h, fk_graph gid, uint32_t base_of
     if (count <= 0 || (uint32_t)count > c->hist_cap) return fail(FK_ERR_VALUE, "count must be in 1..%u", c->hist_cap);
     if (c->pending) return fail(FK_ERR_STATE, "a launch is pending; call fk_wait");
     if (c->comm_lost) return fail(FK_ERR_STATE, "the communicator was aborted after an error; open a new context");
+    if (g->vocab) c->vocab = g->vocab;          // several engines may share a handle
     fk_status s = set_state(c, seed_token, base_offset); if (s) return s;
     CU(cudaEventRecord(c->ev0, c->stream));
     for (int j = 0; j < count; ++j) CU(cudaGraphLaunch(g->exec, c->stream));
@@ -1152,6 +1155,7 @@ extern "C" fk_status fk_decode_chunk_rows(fk_handle h, fk_graph gid, uint32_t ba
     if (!seed_tokens || rows <= 0 || rows > FK_MAX_ROWS) return fail(FK_ERR_VALUE, "rows must be in 1..%d", FK_MAX_ROWS);
     if (count <= 0 || (uint64_t)count * rows > c->hist_cap) return fail(FK_ERR_VALUE, "count * rows must be in 1..%u", c->hist_cap);
     if (c->pending) return fail(FK_ERR_STATE, "a launch is pending; call fk_wait");
+    if (g->vocab) c->vocab = g->vocab;
     for (int m = 0; m < rows; ++m)
         if (c->vocab && seed_tokens[m] >= c->vocab) return fail(FK_ERR_VALUE, "token id %u is outside the embedding table (%u rows)", seed_tokens[m], c->vocab);
     FkState *s0 = (FkState *)c->pinned; memset(s0, 0, sizeof(FkState));

@@ -287,7 +287,7 @@ class LayeredEngine(EngineBase):
         rt.upload(self.scratch["rows_scratch.tokens"], toks)
         if len(want):
             rt.upload(self.scratch["rows_scratch.index"], np.asarray(want, np.uint32))
-        rt.state_set(int(toks[0]), base_offset)
+        rt.state_set(0, base_offset)          # the tokens come from their buffer
         N.check(rt.L.fk_launch_batch(rt.h, arr, len(arr)), "fk_launch_batch")
         token, _, err = rt.state_get()
         if err:
