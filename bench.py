@@ -294,6 +294,143 @@ def run_batch(args, local: int):
     }), flush=True)
 
 
+LAYERED_CTX, LAYERED_PROMPT = 1024, 2048
+
+
+def run_layered(args, local: int):
+    """A layered decoder (random weights) beside the closest older model: a Qwen-shaped bf16 decoder of the same width, heads and
+    feed-forward weights per token, as many layers as the layered one has layers.  One JSON line per shape: decode and prompt
+    throughput of both, and for every kernel the time, the bytes or FLOPs its roofline counts, and the fraction reached, next to
+    the like kernel's.  Kernels are timed over one launch per layer, so every launch reads weights that are not in L2."""
+    import dataclasses
+    from fusekit_b200.batch import PrefillEngine
+    from fusekit_b200.model_spec import LAYERED_CONFIGS, ModelSpec
+    from fusekit_b200 import _native as N
+    from fusekit_b200.runtime import DecodeEngine, EngineBase, attach
+    peak, peak_kind = measured_peak()
+    try:
+        flops_peak = float(json.load(open(os.path.join(ROOT, "MEASURED_PEAKS.json")))["bf16_tflops"])
+    except Exception:
+        flops_peak = 1590.0
+    names = [n for n in LAYERED_CONFIGS if not n.startswith("tiny")] if args.layered == "all" else [args.layered]
+    ctx, P = LAYERED_CTX, LAYERED_PROMPT
+
+    def frac(secs, nbytes, flops=0.0):
+        return max(nbytes / (peak * 1e9), flops / (flops_peak * 1e12)) / secs
+
+    def chunks(eng, seed, base):
+        tok, dev, wall = seed, 0.0, 0.0
+        for i in range(args.warmup + args.steps):
+            t0 = time.perf_counter()
+            out, s = eng.decode_chunk(base, tok, CHUNK)
+            tok = int(out[-1])
+            if i >= args.warmup:
+                dev, wall = dev + s, wall + time.perf_counter() - t0
+        return CHUNK * args.steps / dev, CHUNK * args.steps / wall
+
+    for name in names:
+        spec = LAYERED_CONFIGS[name]
+        m, f, D, L = spec.layers[0].mixer, spec.layers[0].mlp, spec.hidden, len(spec.layers)
+        runs = spec.runs()
+        first = {i: r for r, (i, _) in reversed(list(enumerate(runs)))}       # a layer's first run
+        eng = attach(spec, max(ctx + CHUNK, P) + 8, device=local, max_rows=P)
+        eng.load_synthetic(); eng.prefill_kv_synthetic(ctx); eng.capture()
+        rt = eng.rt
+        sampler = ClockSampler(local); sampler.start()
+        dec, dec_e2e = chunks(eng, 3, ctx)
+        rt.state_set(3, ctx)
+        kv = 2 * ctx * (m.k_rows + m.v_rows)
+        kern = {}
+
+        def add(key, tasks, nbytes, flops=0.0):
+            secs = eng.time_tasks(tasks, 5) / len(tasks)
+            kern[key] = {"us": secs * 1e6, "frac": frac(secs, nbytes, flops), "bytes": nbytes, "flops": flops}
+
+        pick = lambda kind, n=None, of=None: [t for t in (of or eng.replay) if t.kind == kind and t.layer in first.values() and (n is None or t.iarg[1] == n)]
+        add("decode q|k|v|gate", pick(N.TASK_NORM_LINEAR, m.rows), 2 * m.rows * D)
+        add("decode attention", pick(N.TASK_ATTENTION_DECODE), kv)
+        add("decode output projection", [t for t in pick(N.TASK_NORM_LINEAR, D) if t.iarg[0] == m.heads * m.vdim and not t.buf[5]], 2 * D * m.heads * m.vdim)
+        add("decode router + shared up", pick(N.TASK_NORM_LINEAR, f.experts + f.shared_ff), 2 * D * (f.experts + f.shared_ff))
+        add("decode expert up", pick(N.TASK_MOE_UP), 2 * D * f.top * f.ff)
+        add("decode down", pick(N.TASK_MOE_DOWN), 2 * D * (f.top * f.ff + f.shared_ff))
+        add("decode head", [eng.replay[-1]], 2 * D * spec.vocab)
+        rows = eng.rows_dispatches(P, 0, False)
+        rt.upload(eng.scratch["rows_scratch.tokens"], np.random.default_rng(0).integers(0, spec.vocab, P).astype(np.uint32))
+        rt.state_set(0, 0)
+        pre_secs = eng.time_tasks(rows, max(2, args.steps))
+        pr = lambda kind, test=lambda t: True: pick(kind, None, [t for t in rows if test(t)])
+        lin = lambda n, k, mm, grouped=0: (2 * (mm * k + (f.experts if grouped else 1) * n * k + mm * n), 2.0 * mm * n * k)
+        is_lin = lambda wrole, row0=0: pr(N.TASK_LINEAR_ROWS, lambda t: t.iarg[1] == row0 and any(t.buf[1] == eng.W[f"layer_param.{i}.{wrole}"] for i in range(L)))
+        add("rows q|k|v|gate", is_lin("mix.qkvg"), *lin(m.rows, D, P))
+        add("rows attention", pr(N.TASK_ATTENTION_ROWS), 2 * P * (m.q_rows + m.k_rows + m.v_rows + m.heads * m.vdim), m.heads * m.maps * (m.dim + m.vdim) * float(P) * P)
+        add("rows output projection", is_lin("mix.o"), *lin(D, m.heads * m.vdim, P))
+        add("rows router", is_lin("mlp.router_shared"), *lin(f.experts, D, P))
+        add("rows shared up", is_lin("mlp.router_shared", f.experts), *lin(f.shared_ff, D, P))
+        add("rows shared down", is_lin("mlp.shared_down"), *lin(D, f.shared_ff, P))
+        add("rows expert up", is_lin("mlp.experts_up"), *lin(f.ff, D, P * f.top, 1))
+        add("rows expert down", is_lin("mlp.experts_down"), *lin(D, f.ff, P * f.top, 1))
+        add("rows residual + norm", pr(N.TASK_RESIDUAL_NORM_ROWS), P * D * (2 + 2 + 4 + 4))            # y and h in bf16, x read and written
+        add("rows q/k norm + store", pr(N.TASK_QK_NORM_STORE_ROWS), 4 * P * (m.rows - m.heads))
+        add("rows routing", pr(N.TASK_MOE_ROUTE_ROWS), 2 * P * D * (1 + f.top))
+        clocks = sampler.stop()
+        for _ in range(2):
+            t0 = time.perf_counter(); eng.prefill(np.arange(P) % spec.vocab); wall = time.perf_counter() - t0
+        eng.close()
+
+        # ---- the older model of the same size
+        inter = 2 * (f.top * f.ff + f.shared_ff) // 3 // 64 * 64
+        q = ModelSpec(f"qwen-like-{D}", "qwen2", L, D, m.heads, m.kv_heads, 128, inter, spec.vocab, bits=16)
+        old = DecodeEngine(q, ctx + CHUNK + 8, device=local)
+        old.load_synthetic(); old.prefill_kv_synthetic(ctx); old.capture()
+        odec, _ = chunks(old, 3, ctx)
+        old.rt.state_set(3, ctx)
+        like = {}
+
+        def oadd(key, tasks, nbytes, e=old):
+            secs = EngineBase.time_tasks(e, tasks, 5) / len(tasks)
+            like[key] = {"us": secs * 1e6, "frac": frac(secs, nbytes), "bytes": nbytes}
+
+        kinds = lambda k, n=None, e=old: [t for t in e.tasks if t.kind == k and (n is None or (t.iarg[0], t.iarg[1]) == n)]
+        oadd("qkv", kinds(2), q.linear_bytes(D, (q.n_q + 2 * q.n_kv) * 128))
+        oadd("attention", kinds(4), 4 * q.n_kv * 128 * ctx)
+        oadd("o", kinds(5, (q.n_q * 128, D)), q.linear_bytes(q.n_q * 128, D, True))
+        oadd("gate/up", kinds(6), 2 * q.linear_bytes(D, inter))
+        oadd("down", kinds(5, (inter, D)), q.linear_bytes(inter, D, True))
+        oadd("head", kinds(7), q.linear_bytes(D, q.vocab))
+        obytes = q.bytes_per_token(ctx)
+        old.close()
+        q4 = dataclasses.replace(q, bits=4)
+        pre = PrefillEngine(q4, P, 16, device=local)
+        pre.load_synthetic(); pre.capture()
+        osecs = [sum(pre.decode_chunk(c, np.arange(16), 1)[1] for c in range(0, P, 16)) for _ in range(2)][1]
+        pre.rt.state_set(3, P - 16)
+        pk = lambda k, n=None: kinds(k, n, pre)
+        oadd("16 rows qkv", pk(5, (D, (q.n_q + 2 * q.n_kv) * 128)), q4.linear_bytes(D, (q.n_q + 2 * q.n_kv) * 128), pre)
+        oadd("16 rows attention", pk(4), 4 * q.n_kv * 128 * P, pre)
+        oadd("16 rows o", pk(5, (q.n_q * 128, D)), q4.linear_bytes(q.n_q * 128, D), pre)
+        oadd("16 rows gate/up", pk(6), 2 * q4.linear_bytes(D, inter), pre)
+        oadd("16 rows down", pk(5, (inter, D)), q4.linear_bytes(inter, D), pre)
+        oadd("16 rows norm", pk(11), 4 * 16 * D, pre)
+        oadd("16 rows rope + store", pk(12), 4 * 16 * (q.n_q + 2 * q.n_kv) * 128, pre)
+        pre.close()
+        pair = {"decode q|k|v|gate": "qkv", "decode attention": "attention", "decode output projection": "o", "decode router + shared up": "gate/up", "decode expert up": "gate/up",
+                "decode down": "down", "decode head": "head", "rows q|k|v|gate": "16 rows qkv", "rows attention": "16 rows attention", "rows output projection": "16 rows o",
+                "rows router": "16 rows o", "rows shared up": "16 rows gate/up", "rows shared down": "16 rows down", "rows expert up": "16 rows gate/up", "rows expert down": "16 rows down",
+                "rows residual + norm": "16 rows norm", "rows q/k norm + store": "16 rows rope + store"}
+        for k, v in kern.items():
+            if k in pair:
+                v["like"], v["like_frac"], v["like_frac_over_frac"] = pair[k], like[pair[k]]["frac"], like[pair[k]]["frac"] / v["frac"]
+        print(json.dumps({
+            "metric": f"layered decoder {name}: decode tok/s at context {ctx}, prompt tok/s at {P}", "value": dec, "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+            "warmup": args.warmup, "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
+            "config": {"model": name, "runs": len(runs), "l2": "one launch per layer: inputs larger than L2"},
+            "decode": {"tok_s": dec, "e2e_tok_s": dec_e2e, "roofline_frac": spec.bytes_per_token(ctx) * dec / 1e9 / peak, "bytes_per_token": spec.bytes_per_token(ctx)},
+            "prompt": {"tok_s": P / pre_secs, "e2e_tok_s": P / wall, "tflops": spec.flops_per_token(P / 2) * P / pre_secs / 1e12},
+            "like_model": {"model": q.name, "layers": L, "inter": inter, "decode_tok_s_bf16": odec, "decode_roofline_frac": obytes * odec / 1e9 / peak,
+                           "prompt_tok_s_q4_16_rows": P / osecs},
+            "peaks": {"hbm_gbs": peak, "bf16_tflops": flops_peak, "kind": peak_kind}, "clocks": clocks, "kernels": kern, "like_kernels": like}), flush=True)
+
+
 def main():
     global CHUNK
     ap = argparse.ArgumentParser()
@@ -307,6 +444,7 @@ def main():
     ap.add_argument("--no-tp-extra", action="store_true", help="with N > 1 replicas, skip the additional 32B tensor-parallel run")
     ap.add_argument("--batch", type=int, default=1, help="independent sequences decoded together (2..16: the batch decode engine, one GPU)")
     ap.add_argument("--qmm", default="auto", choices=["auto", "tcgen05", "mma"], help="kernel of the several-row projections in batch decode")
+    ap.add_argument("--layered", default=None, metavar="SHAPE", help="measure a layered decoder (a registered shape, or all) beside the closest older model")
     ap.add_argument("--no-cpu-baseline", action="store_true")
     ap.add_argument("--cpu-budget", type=float, default=15.0)
     ap.add_argument("--profile-nodes", type=int, default=5, help="repeats of the per-kernel timing pass (0 = skip)")
@@ -316,6 +454,11 @@ def main():
     local = int(os.environ.get("LOCAL_RANK", 0))
     if args.impl == "reference":
         run_reference(args, rank)
+        return
+
+    if args.layered:
+        if rank == 0:
+            run_layered(args, local)
         return
 
     if args.batch > 1:

@@ -44,7 +44,8 @@ cudaError_t fkl_init() {
                  TRY(big_smem(k_attention<uint16_t, uint16_t, VPL, false>)); TRY(big_smem(k_attention<float, float, VPL, false>))
     ATT(1); ATT(2); ATT(4); ATT(8); ATT(16);
     TRY(big_smem(k_residual_norm_rows<uint16_t>)); TRY(big_smem(k_residual_norm_rows<float>));
-    TRY(big_smem(k_gemv<FKL_GV_LINEAR>)); TRY(big_smem(k_gemv<FKL_GV_MOE_UP>)); TRY(big_smem(k_gemv<FKL_GV_MOE_DOWN>));
+    TRY(big_smem(k_gemv<FKL_GV_LINEAR, 0>)); TRY(big_smem(k_gemv<FKL_GV_LINEAR, 1>)); TRY(big_smem(k_gemv<FKL_GV_LINEAR, 2>)); TRY(big_smem(k_gemv<FKL_GV_LINEAR, 4>));
+    TRY(big_smem(k_gemv<FKL_GV_MOE_UP, 0>)); TRY(big_smem(k_gemv<FKL_GV_MOE_DOWN, 0>)); TRY(big_smem(k_attention_decode));
     TRY(cudaFuncSetAttribute(k_gemm_tc<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TcTile<64>::SMEM));
     TRY(cudaFuncSetAttribute(k_gemm_tc<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TcTile<128>::SMEM));
     TRY(cudaFuncSetAttribute(k_gemm_tc<256>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TcTile<256>::SMEM));
@@ -62,18 +63,23 @@ static fk_status bad(char *err, size_t cap, const char *fmt, ...) {
 }
 static int round_up(int v, int m) { return (v + m - 1) / m * m; }
 
-// Blocks and K split of a matrix-vector product: as few warps per row group as reach every SM twice with one group each.
+// Blocks and K split of a matrix-vector product: one block per SM, and as few warps per row group as give every warp one.
 static cudaError_t launch_gemv(FklEnv &c, int mode, GemvArgs &a) {
-    const int groups = (a.n + FKL_GV_R - 1) / FKL_GV_R, slots = c.sm_count * 2;
+    const int groups = (a.n + FKL_GV_R - 1) / FKL_GV_R, slots = c.sm_count;
     int ks = 1;
     while (ks < FKL_GV_WARPS && ks * 2 <= a.nchunks && (long long)groups * ks < (long long)slots * FKL_GV_WARPS) ks *= 2;
     a.kslices = ks;
     const int spb = FKL_GV_WARPS / ks, blocks = (groups + spb - 1) / spb, grid = blocks < slots ? blocks : slots;
     const size_t smem = gv_smem_bytes(a.nchunks);
     const dim3 g(grid), b(FKL_GV_WARPS * 32);
-    if (mode == FKL_GV_LINEAR) return launch(c, k_gemv<FKL_GV_LINEAR>, g, b, smem, c.state, a);
-    if (mode == FKL_GV_MOE_UP) return launch(c, k_gemv<FKL_GV_MOE_UP>, g, b, smem, c.state, a);
-    return launch(c, k_gemv<FKL_GV_MOE_DOWN>, g, b, smem, c.state, a);
+    if (mode == FKL_GV_MOE_UP) return launch(c, k_gemv<FKL_GV_MOE_UP, 0>, g, b, smem, c.state, a);
+    if (mode == FKL_GV_MOE_DOWN) return launch(c, k_gemv<FKL_GV_MOE_DOWN, 0>, g, b, smem, c.state, a);
+    const bool vec = a.norm_w && a.k % 4 == 0 && (((uintptr_t)a.x | (uintptr_t)a.pend | (uintptr_t)a.add | (uintptr_t)a.x_out | (uintptr_t)a.h_out) & 15) == 0;
+    const int per = FKL_GV_WARPS * 32 * 4;              // values in one register round of a block
+    if (vec && a.k <= per) return launch(c, k_gemv<FKL_GV_LINEAR, 1>, g, b, smem, c.state, a);
+    if (vec && a.k <= 2 * per) return launch(c, k_gemv<FKL_GV_LINEAR, 2>, g, b, smem, c.state, a);
+    if (vec && a.k <= 4 * per) return launch(c, k_gemv<FKL_GV_LINEAR, 4>, g, b, smem, c.state, a);
+    return launch(c, k_gemv<FKL_GV_LINEAR, 0>, g, b, smem, c.state, a);
 }
 // bf16 rows [rows, k] (row stride ld elements) in boxes of 64 columns x box_rows, 128-byte swizzle
 typedef CUresult (*EncodeTiled)(CUtensorMap *, CUtensorMapDataType, cuuint32_t, void *, const cuuint64_t *, const cuuint64_t *, const cuuint32_t *, const cuuint32_t *,
@@ -182,6 +188,8 @@ fk_status fkl_run(FklEnv &c, const fk_task &t, char *err, size_t ecap) {
             a.splits = i[7];
             if (a.splits <= 0 || a.splits > 8 * a.vpad || a.splits > 256) return bad(err, ecap, "attention_decode: bad number of key splits");
             const dim3 g(a.splits, a.G * a.tiles, 1), blk(FKL_ATT_WARPS * 32);
+            const int ad = ad_layout(a.maps, a.dpad, a.vpad).total;
+            if (!f32 && ad <= 200 * 1024) { e = launch(c, k_attention_decode, g, dim3(FKL_AD_THREADS), (size_t)ad, c.state, a); break; }
             if (f32) VPL_SWITCH(a.vpad, e = launch(c, (k_attention<float, float, VPL, true>), g, blk, smem, c.state, a));
             else VPL_SWITCH(a.vpad, e = launch(c, (k_attention<uint16_t, float, VPL, true>), g, blk, smem, c.state, a));
         } else {

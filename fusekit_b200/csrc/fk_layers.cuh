@@ -342,6 +342,210 @@ __global__ void __launch_bounds__(FKL_ATT_WARPS * 32) k_attention(FkState *st, A
     }
 }
 
+// ---------------------------------------------------------------- attention of one position, bf16 caches
+// The same task as the DECODE form above, laid out for latency.  A block takes 64 keys at a time: the maps' keys and the values of
+// a chunk arrive in shared memory by cp.async (two chunks in flight, the first two requested before the dependency wait: the
+// cached rows are older than the kernel before this one), then a thread scores one key against two query rows, a warp runs the
+// softmax of one row, and the threads spread over (value columns, key parts) for the weighted sum.  The new key and value, known
+// only after the wait, go to the cache and straight into the last chunk.  Partials of the blocks meet in global memory; the last
+// block of a (kv head, row tile) folds them, combines the maps and applies the gate.
+#define FKL_AD_KEYS 64
+#define FKL_AD_THREADS 256
+struct AdLayout { int ks, vs, stage, q, sc, pr, nk, nv, of, total; };      // byte offsets; ks / vs: row strides in elements
+__host__ __device__ inline AdLayout ad_layout(int maps, int dpad, int vpad) {
+    AdLayout l; l.ks = ((dpad / 8) | 1) * 8; l.vs = ((vpad / 8) | 1) * 8;           // odd multiples of 16 bytes
+    l.stage = FKL_AD_KEYS * 2 * (maps * l.ks + l.vs);
+    const int red = FKL_AD_THREADS * FKL_ATT_ROWS * 2 * 4;                           // the key parts' sums, over the chunk buffers
+    l.q = 2 * l.stage > red ? 2 * l.stage : red;
+    l.sc = l.q + FKL_ATT_ROWS * dpad * 4; l.pr = l.sc + FKL_ATT_ROWS * (FKL_AD_KEYS + 1) * 4; l.pr = (l.pr + 15) & ~15;
+    l.nk = l.pr + FKL_AD_KEYS * FKL_ATT_ROWS * 4; l.nv = l.nk + ((maps * dpad * 2 + 15) & ~15); l.of = l.nv + ((vpad * 2 + 15) & ~15);
+    l.total = l.of + FKL_ATT_ROWS * vpad * 4;
+    return l;
+}
+__device__ __forceinline__ void cp16_zfill(uint32_t dst, const void *src, bool valid) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+__global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st, AttnArgs a) {
+    extern __shared__ __align__(128) unsigned char ad_smem[];
+    constexpr int RT = FKL_ATT_ROWS, KC = FKL_AD_KEYS, NT = FKL_AD_THREADS;
+    const AdLayout L = ad_layout(a.maps, a.dpad, a.vpad);
+    float *qs = reinterpret_cast<float *>(ad_smem + L.q), *sc = reinterpret_cast<float *>(ad_smem + L.sc), *pr = reinterpret_cast<float *>(ad_smem + L.pr);
+    uint16_t *nk = reinterpret_cast<uint16_t *>(ad_smem + L.nk), *nv = reinterpret_cast<uint16_t *>(ad_smem + L.nv);
+    float *of = reinterpret_cast<float *>(ad_smem + L.of);
+    __shared__ float s_corr[RT], s_m[RT], s_l[RT], s_fac[256 * RT]; __shared__ int s_last;
+    const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
+    const int g = blockIdx.y / a.tiles, tile = blockIdx.y - g * a.tiles, group = a.H / a.G, nrow_kv = group * a.maps, r0 = tile * RT, nr = min(RT, nrow_kv - r0);
+    const uint32_t upos = st->offset;                   // advanced by the head of the token before, long since finished
+    const int pos = (int)upos, n = pos + 1, per = ((n + a.splits - 1) / a.splits + KC - 1) / KC * KC, active = (n + per - 1) / per;
+    const int k0 = blockIdx.x * per, k1 = min(n, k0 + per), nchunk = k1 > k0 ? (k1 - k0 + KC - 1) / KC : 0;
+    const bool fits = upos < (uint32_t)a.cap;
+    uint16_t *ck = (uint16_t *)a.ck + (size_t)g * a.maps * a.cap * a.dpad, *cv = (uint16_t *)a.cv + (size_t)g * a.cap * a.vpad;
+    const uint32_t sbase = (uint32_t)__cvta_generic_to_shared(ad_smem);
+    auto request = [&](int c) {                         // chunk c into stage c & 1; the new position's row comes from registers later
+        const uint32_t kb = sbase + (uint32_t)((c & 1) * L.stage), vb = kb + (uint32_t)(a.maps * KC * L.ks * 2);
+        const int kn = a.dpad / 8, vn = a.vpad / 8, key0 = k0 + c * KC;
+        for (int i = tid; i < a.maps * KC * kn; i += NT) {
+            const int r = i / kn, cc = (i - r * kn) * 8, key = key0 + (r & (KC - 1)); const bool v = key < pos;
+            if (key != pos) cp16_zfill(kb + (uint32_t)((r * L.ks + cc) * 2), v ? ck + ((size_t)(r / KC) * a.cap + key) * a.dpad + cc : ck, v);
+        }
+        for (int i = tid; i < KC * vn; i += NT) {
+            const int r = i / vn, cc = (i - r * vn) * 8, key = key0 + r; const bool v = key < pos;
+            if (key != pos) cp16_zfill(vb + (uint32_t)((r * L.vs + cc) * 2), v ? cv + (size_t)key * a.vpad + cc : cv, v);
+        }
+    };
+    if (fits) for (int c = 0; c < 2; ++c) { if (c < nchunk) request(c); asm volatile("cp.async.commit_group;" ::: "memory"); }
+    pdl_wait(); pdl_launch_dependents();
+    if (!fits) { if (tid == 0) atomicOr(&st->error, FKL_ERR_CAPACITY); return; }
+    if (nchunk == 0) return;                            // more splits than this many keys need
+    // ---- query rows, and where the position falls here the new key and value
+    const bool mine = pos >= k0 && pos < k1;
+    for (int it = wid; it < RT + (mine ? a.maps + 1 : 0); it += NT / 32) {
+        if (it >= nr && it < RT) { for (int i = lane; i < a.dpad; i += 32) qs[it * a.dpad + i] = 0.0f; continue; }
+        if (it == RT + a.maps) {
+            const float *src = a.qkv + (a.H + a.G) * a.maps * a.dim + g * a.vdim;
+            for (int i = lane; i < a.vpad; i += 32) { const uint16_t v = i < a.vdim ? f2bf(__ldcg(src + i)) : (uint16_t)0; nv[i] = v; if (i < a.vdim) cv[(size_t)pos * a.vpad + i] = v; }
+            continue;
+        }
+        const bool is_q = it < RT;
+        const float *src = a.qkv + (is_q ? (g * nrow_kv + r0 + it) : (a.H * a.maps + g * a.maps + (it - RT))) * a.dim;
+        const uint16_t *w = is_q ? a.qn : a.kn;
+        float ss = 0.0f;
+        for (int i = lane; i < a.dim; i += 32) { const float v = __ldcg(src + i); ss = fmaf(v, v, ss); }
+        const float r = inv_rms(warp_sum(ss), a.dim, a.eps);
+        for (int i = lane; i < a.dpad; i += 32) {
+            const float v = i < a.dim ? __ldcg(src + i) * r * bf2f(w[i]) : 0.0f;
+            if (is_q) qs[it * a.dpad + i] = v * a.scale;
+            else { nk[(it - RT) * a.dpad + i] = f2bf(v); if (i < a.dim) ck[((size_t)(it - RT) * a.cap + pos) * a.dpad + i] = f2bf(v); }
+        }
+    }
+    // ---- chunks
+    int tpc = 1; while (tpc < NT && tpc < a.vpad / 2) tpc <<= 1;        // threads over pairs of value columns
+    const int parts = NT / tpc, col = (tid & (tpc - 1)) * 2, part = tid / tpc;
+    float o[RT][2];
+#pragma unroll
+    for (int r = 0; r < RT; ++r) o[r][0] = o[r][1] = 0.0f;
+    float m = -INFINITY, l = 0.0f;                      // row `wid` of the softmax
+    for (int c = 0; c < nchunk; ++c) {
+        asm volatile("cp.async.wait_group 1;" ::: "memory");
+        __syncthreads();
+        const unsigned char *kb = ad_smem + (c & 1) * L.stage; unsigned char *kbw = ad_smem + (c & 1) * L.stage;
+        const uint16_t *ks = reinterpret_cast<const uint16_t *>(kb), *vs = ks + a.maps * KC * L.ks;
+        const int key0 = k0 + c * KC;
+        if (mine && pos >= key0 && pos < key0 + KC) {
+            uint16_t *kw = reinterpret_cast<uint16_t *>(kbw), *vw = kw + a.maps * KC * L.ks;
+            for (int i = tid; i < a.maps * a.dpad; i += NT) { const int mm = i / a.dpad; kw[(mm * KC + pos - key0) * L.ks + i - mm * a.dpad] = nk[i]; }
+            for (int i = tid; i < a.vpad; i += NT) vw[(pos - key0) * L.vs + i] = nv[i];
+            __syncthreads();
+        }
+        {   // scores: key tid % 64, rows tid / 64 and 4 more (of the same map)
+            const int key = tid & (KC - 1), ra = tid / KC, rb = ra + 4, mm = a.maps == 2 ? (ra & 1) : 0;
+            const uint16_t *kr = ks + (mm * KC + key) * L.ks; const float *qa = qs + ra * a.dpad, *qb = qs + rb * a.dpad;
+            float da = 0.0f, db = 0.0f;
+            for (int d = 0; d < a.dpad; d += 8) {
+                float f[8]; unpack8f(*reinterpret_cast<const uint4 *>(kr + d), f);
+                const float4 a0 = *reinterpret_cast<const float4 *>(qa + d), a1 = *reinterpret_cast<const float4 *>(qa + d + 4);
+                const float4 b0 = *reinterpret_cast<const float4 *>(qb + d), b1 = *reinterpret_cast<const float4 *>(qb + d + 4);
+                da = fmaf(a0.x, f[0], fmaf(a0.y, f[1], fmaf(a0.z, f[2], fmaf(a0.w, f[3], fmaf(a1.x, f[4], fmaf(a1.y, f[5], fmaf(a1.z, f[6], fmaf(a1.w, f[7], da))))))));
+                db = fmaf(b0.x, f[0], fmaf(b0.y, f[1], fmaf(b0.z, f[2], fmaf(b0.w, f[3], fmaf(b1.x, f[4], fmaf(b1.y, f[5], fmaf(b1.z, f[6], fmaf(b1.w, f[7], db))))))));
+            }
+            const bool v = key0 + key < k1;
+            sc[ra * (KC + 1) + key] = v ? da : -INFINITY; sc[rb * (KC + 1) + key] = v ? db : -INFINITY;
+        }
+        __syncthreads();
+        {   // softmax of row wid
+            const float s0 = sc[wid * (KC + 1) + lane], s1 = sc[wid * (KC + 1) + lane + 32];
+            const float mn = fmaxf(m, warp_max(fmaxf(s0, s1))), corr = expf(m - mn), p0 = expf(s0 - mn), p1 = expf(s1 - mn);
+            l = l * corr + warp_sum(p0 + p1); m = mn;
+            pr[lane * RT + wid] = p0; pr[(lane + 32) * RT + wid] = p1;
+            if (lane == 0) s_corr[wid] = corr;
+        }
+        __syncthreads();
+        if (col < a.vpad) {
+#pragma unroll
+            for (int r = 0; r < RT; ++r) { const float f = s_corr[r]; o[r][0] *= f; o[r][1] *= f; }
+            const int nkey = min(KC, k1 - key0);
+#pragma unroll 4
+            for (int k = part; k < nkey; k += parts) {
+                const uint32_t vv = *reinterpret_cast<const uint32_t *>(vs + k * L.vs + col);
+                const float v0 = bf_lo(vv), v1 = bf_hi(vv);
+                const float4 pa = *reinterpret_cast<const float4 *>(pr + k * RT), pb = *reinterpret_cast<const float4 *>(pr + k * RT + 4);
+                const float p[RT] = {pa.x, pa.y, pa.z, pa.w, pb.x, pb.y, pb.z, pb.w};
+#pragma unroll
+                for (int r = 0; r < RT; ++r) { o[r][0] = fmaf(p[r], v0, o[r][0]); o[r][1] = fmaf(p[r], v1, o[r][1]); }
+            }
+        }
+        __syncthreads();                                // the stage is free
+        if (c + 2 < nchunk) request(c + 2);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    // ---- fold the key parts (chunk buffers reused; nothing is in flight: the groups above are empty)
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    if (lane == 0) { s_m[wid] = m; s_l[wid] = l; }
+    float *red = reinterpret_cast<float *>(ad_smem);
+    __syncthreads();
+    for (int r = 0; r < RT; ++r) *reinterpret_cast<float2 *>(red + (r * NT + tid) * 2) = make_float2(o[r][0], o[r][1]);
+    __syncthreads();
+    for (int i = tid; i < nr * (a.vpad / 2); i += NT) {
+        const int r = i / (a.vpad / 2), cp = i - r * (a.vpad / 2);
+        float2 s = make_float2(0.0f, 0.0f);
+        for (int p = 0; p < parts; ++p) { const float2 v = *reinterpret_cast<const float2 *>(red + (r * NT + p * tpc + cp) * 2); s.x += v.x; s.y += v.y; }
+        const float f = active > 1 ? 1.0f : 1.0f / s_l[r];
+        *reinterpret_cast<float2 *>(of + r * a.vpad + cp * 2) = make_float2(s.x * f, s.y * f);
+    }
+    __syncthreads();
+    if (active > 1) {
+        const size_t stride = (size_t)RT * (a.vpad + 2);
+        const float *base = a.part + (size_t)blockIdx.y * a.splits * stride;
+        float *mine_p = a.part + ((size_t)blockIdx.y * a.splits + blockIdx.x) * stride;
+        for (int i = tid; i < RT * a.vpad / 4; i += NT) __stcg(reinterpret_cast<float4 *>(mine_p) + i, reinterpret_cast<const float4 *>(of)[i]);
+        if (tid < RT) { __stcg(mine_p + RT * a.vpad + tid * 2, s_m[tid]); __stcg(mine_p + RT * a.vpad + tid * 2 + 1, s_l[tid]); }
+        __threadfence();
+        __syncthreads();
+        if (tid == 0) { s_last = atomicAdd(a.counter + blockIdx.y, 1u) == (uint32_t)active - 1u; if (s_last) a.counter[blockIdx.y] = 0u; }
+        __syncthreads();
+        if (!s_last) return;
+        __threadfence();
+        // factors exp(m - max) / sum of every (split, row), one warp per row
+        for (int r = wid; r < nr; r += NT / 32) {
+            float mx = -INFINITY, ls = 0.0f;
+            for (int p = lane; p < active; p += 32) mx = fmaxf(mx, __ldcg(base + (size_t)p * stride + RT * a.vpad + r * 2));
+            mx = warp_max(mx);
+            for (int p = lane; p < active; p += 32) {
+                const float f = expf(__ldcg(base + (size_t)p * stride + RT * a.vpad + r * 2) - mx);
+                s_fac[p * RT + r] = f; ls = fmaf(f, __ldcg(base + (size_t)p * stride + RT * a.vpad + r * 2 + 1), ls);
+            }
+            ls = warp_sum(ls);
+            __syncwarp();
+            for (int p = lane; p < active; p += 32) s_fac[p * RT + r] /= ls;
+        }
+        __syncthreads();
+        for (int i = tid; i < nr * a.vpad / 4; i += NT) {
+            const int r = i * 4 / a.vpad;
+            float4 s = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 8
+            for (int p = 0; p < active; ++p) {
+                const float4 v = __ldcg(reinterpret_cast<const float4 *>(base + (size_t)p * stride) + i); const float f = s_fac[p * RT + r];
+                s.x = fmaf(f, v.x, s.x); s.y = fmaf(f, v.y, s.y); s.z = fmaf(f, v.z, s.z); s.w = fmaf(f, v.w, s.w);
+            }
+            reinterpret_cast<float4 *>(of)[i] = s;
+        }
+        __syncthreads();
+    }
+    for (int hh = wid; hh < nr / a.maps; hh += NT / 32) {
+        const int head = g * group + r0 / a.maps + hh;
+        const float *o1 = of + hh * a.maps * a.vpad, *o2 = o1 + a.vpad;
+        float f = 1.0f;
+        if (a.maps == 2) {
+            float ss = 0.0f;
+            for (int d = lane; d < a.vdim; d += 32) { const float v = o1[d] - a.lambda * o2[d]; ss = fmaf(v, v, ss); }
+            f = inv_rms(warp_sum(ss), a.vdim, a.eps) * (1.0f - a.diff);
+        }
+        if (a.gate) f *= sigmoid_f(__ldcg((const float *)a.gate + head));
+        float *out = (float *)a.out + head * a.vdim;
+        for (int d = lane; d < a.vdim; d += 32) out[d] = (a.maps == 2 ? o1[d] - a.lambda * o2[d] : o1[d]) * f;
+    }
+}
+
 // ---------------------------------------------------------------- mixture of experts: choice and grouping of M rows
 // The `top` largest logits of z[0 .. E) by one warp (lowest index first among equals), into idx / val (lane 0 of the warp
 // and everyone else sees them after a __syncwarp).
@@ -426,12 +630,12 @@ __global__ void __launch_bounds__(256) k_moe_gather(const FkState *st, RouteArgs
 // ---------------------------------------------------------------- one row: matrix-vector products over bf16 rows
 // A warp owns R = 2 weight rows at a time and streams them in chunks of 256 weights (16 bytes per lane and row), two batches
 // of U = 4 chunks in registers: one being multiplied, one in flight.  The activations sit in shared memory as fp32, in the
-// order the lanes read them without bank conflicts.  With few rows, 2 .. 8 warps of a block share a row group and split K.
+// order the lanes read them without bank conflicts.  With few rows, 2 .. 16 warps of a block share a row group and split K.
 // A chunk is described by (base of row 0, row stride, weights in it), which also expresses the concatenated K ranges of a
 // mixture's down projection.  The first batch is fetched before the dependency wait where the rows do not depend on it.
 #define FKL_GV_R 2
 #define FKL_GV_U 4
-#define FKL_GV_WARPS 8
+#define FKL_GV_WARPS 16
 enum { FKL_GV_LINEAR = 0, FKL_GV_MOE_UP = 1, FKL_GV_MOE_DOWN = 2 };
 struct GvChunk { const uint16_t *base; int stride, len; };
 struct GemvArgs {
@@ -449,13 +653,16 @@ __device__ __forceinline__ int gv_place(int i) { const int j = i & 7; return (i 
 __device__ __forceinline__ uint4 ldg_stream(const uint16_t *p) {
     uint4 v; asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p)); return v;
 }
-template <int MODE>
-__global__ void __launch_bounds__(FKL_GV_WARPS * 32, 2) k_gemv(FkState *st, GemvArgs a) {
+// NV > 0: the norm prologue keeps NV x 4 values per thread in registers (inputs of up to NV * 2048 values, a multiple of 4): one
+// round of loads, the weights' before the dependency wait.  NV = 0: any length, several passes.
+template <int MODE, int NV>
+__global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, GemvArgs a) {
     extern __shared__ __align__(16) unsigned char gv_smem[];
     constexpr int R = FKL_GV_R, U = FKL_GV_U, NT = FKL_GV_WARPS * 32;
     float *xs = reinterpret_cast<float *>(gv_smem); GvChunk *tab = reinterpret_cast<GvChunk *>(gv_smem + (size_t)a.nchunks * 1024);
     __shared__ float red[40], part[FKL_GV_WARPS][R], tval[FKL_MAX_TOP]; __shared__ int tsel[FKL_MAX_TOP];
     __shared__ unsigned long long wbest[FKL_GV_WARPS]; __shared__ int is_last;
+    __shared__ float slog[MODE == FKL_GV_MOE_UP ? FKL_MAX_EXPERTS : 1];
     const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, KS = a.kslices, spb = FKL_GV_WARPS / KS, ksl = wid % KS, slot = wid / KS;
     const int c0 = a.nchunks * ksl / KS, c1 = a.nchunks * (ksl + 1) / KS, nb = (c1 - c0 + U - 1) / U;
     const int groups = (a.n + R - 1) / R, gstride = gridDim.x * spb;
@@ -489,6 +696,15 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 2) k_gemv(FkState *st, Gemv
         __syncthreads();
         if (MODE == FKL_GV_LINEAR && g < groups && nb > 0) { set_rows(g); fetch(c0); }
     }
+    uint2 pw[NV > 0 ? NV : 1], nw[NV > 0 ? NV : 1];
+    if (NV > 0 && a.norm_w) {
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const int i = (v * NT + tid) * 4;
+            nw[v] = i < a.k ? __ldg(reinterpret_cast<const uint2 *>(a.norm_w + i)) : make_uint2(0, 0);
+            pw[v] = a.pend && i < a.k ? __ldg(reinterpret_cast<const uint2 *>(a.post_w + i)) : make_uint2(0, 0);
+        }
+    }
     pdl_wait(); pdl_launch_dependents();
     // ---- the input vector
     if (MODE == FKL_GV_MOE_DOWN) {
@@ -501,21 +717,61 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 2) k_gemv(FkState *st, Gemv
             else { const int cs = c - a.top * nce; tab[c] = GvChunk{a.w2 + cs * 256, a.ldffs, min(256, a.ldffs - cs * 256)}; }
         }
         (void)nshared;
-        for (int i = tid; i < a.top * a.ff; i += NT) { const int j = i / a.ff, q = i - j * a.ff; xs[gv_place(j * nce * 256 + q)] = tval[j] * __ldcg(a.x + i); }
-        for (int i = tid; i < a.ffs; i += NT) xs[gv_place(a.top * nce * 256 + i)] = __ldcg(a.sact + i);
         __syncthreads();
         if (g < groups && nb > 0) { set_rows(g); fetch(c0); }
+        for (int j = 0; j < a.top; ++j) for (int i = tid; i < a.ff; i += NT) xs[gv_place(j * nce * 256 + i)] = tval[j] * __ldcg(a.x + j * a.ff + i);
+        for (int i = tid; i < a.ffs; i += NT) xs[gv_place(a.top * nce * 256 + i)] = __ldcg(a.sact + i);
+        __syncthreads();
     } else if (MODE == FKL_GV_MOE_UP) {
+        for (int i = tid; i < a.k; i += NT) xs[gv_place(i)] = __ldcg(a.x + i);
+        for (int i = tid; i < a.E; i += NT) slog[i] = __ldcg(a.logits + i);
+        __syncthreads();
         if (wid == 0) {
-            warp_top(a.logits, a.E, a.top, tsel, tval, lane);
+            warp_top(slog, a.E, a.top, tsel, tval, lane);
             if (blockIdx.x == 0) {
                 warp_top_softmax(tval, a.top, lane);
                 for (int j = lane; j < a.top; j += 32) { a.sel[j] = tsel[j]; a.wts[j] = tval[j]; }
             }
         }
-        for (int i = tid; i < a.k; i += NT) xs[gv_place(i)] = __ldcg(a.x + i);
         __syncthreads();
         if (g < groups && nb > 0) { set_rows(g); fetch(c0); }
+    } else if (NV > 0 && a.norm_w) {
+        float4 x[NV > 0 ? NV : 1], y[NV > 0 ? NV : 1];
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const int i = (v * NT + tid) * 4;
+            x[v] = y[v] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            if (i < a.k) {
+                x[v] = __ldcg(reinterpret_cast<const float4 *>(a.x + i));
+                if (a.pend) y[v] = __ldcg(reinterpret_cast<const float4 *>(a.pend + i));
+                if (a.add) { const float4 e = __ldcg(reinterpret_cast<const float4 *>(a.add + i)); x[v].x += e.x; x[v].y += e.y; x[v].z += e.z; x[v].w += e.w; }
+            }
+        }
+        if (a.pend) {
+            float ss = 0.0f;
+#pragma unroll
+            for (int v = 0; v < NV; ++v) ss = fmaf(y[v].x, y[v].x, fmaf(y[v].y, y[v].y, fmaf(y[v].z, y[v].z, fmaf(y[v].w, y[v].w, ss))));
+            const float ry = inv_rms(block_sum(ss, red), a.k, a.eps);
+#pragma unroll
+            for (int v = 0; v < NV; ++v) {
+                x[v].x = fmaf(y[v].x * ry, bf_lo(pw[v].x), x[v].x); x[v].y = fmaf(y[v].y * ry, bf_hi(pw[v].x), x[v].y);
+                x[v].z = fmaf(y[v].z * ry, bf_lo(pw[v].y), x[v].z); x[v].w = fmaf(y[v].w * ry, bf_hi(pw[v].y), x[v].w);
+            }
+        }
+        float ss = 0.0f;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) ss = fmaf(x[v].x, x[v].x, fmaf(x[v].y, x[v].y, fmaf(x[v].z, x[v].z, fmaf(x[v].w, x[v].w, ss))));
+        const float r = inv_rms(block_sum(ss, red), a.k, a.eps);
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const int i = (v * NT + tid) * 4;
+            if (i >= a.k) continue;
+            if (a.x_out && blockIdx.x == 0) *reinterpret_cast<float4 *>(a.x_out + i) = x[v];
+            const float4 h = make_float4(x[v].x * r * bf_lo(nw[v].x), x[v].y * r * bf_hi(nw[v].x), x[v].z * r * bf_lo(nw[v].y), x[v].w * r * bf_hi(nw[v].y));
+            *reinterpret_cast<float4 *>(xs + gv_place(i)) = h;          // four neighbours stay neighbours
+            if (a.h_out && blockIdx.x == 0) *reinterpret_cast<float4 *>(a.h_out + i) = h;
+        }
+        __syncthreads();
     } else if (a.norm_w) {
         __syncthreads();
         float ry = 0.0f;

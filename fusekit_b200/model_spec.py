@@ -206,9 +206,10 @@ CONFIGS = {
 
 
 LAYERED_CONFIGS = {
-    # looped mixture-of-experts decoders with differential attention, at sizes of a small and a mid-size model's layers
-    "fatulix-2048": _fatulix("fatulix-2048", 2048, 65536, 8, AttentionSpec(16, 4, 64, 128, 0.125, 0.3), MoeSpec(32, 4, 1024, 2048), LoopSpec(2, 6, 2)),
-    "fatulix-3584": _fatulix("fatulix-3584", 3584, 152064, 8, AttentionSpec(28, 4, 64, 128, 0.125, 0.3), MoeSpec(16, 2, 4736, 9472)),
+    # looped mixture-of-experts decoders with differential attention, at sizes of the layers of a small, a 7B and a 32B model
+    "fatulix-2048": _fatulix("fatulix-2048", 2048, 65536, 16, AttentionSpec(16, 4, 64, 128, 0.125, 0.3), MoeSpec(32, 4, 1024, 2048), LoopSpec(4, 8, 2)),
+    "fatulix-3584": _fatulix("fatulix-3584", 3584, 152064, 8, AttentionSpec(28, 4, 64, 128, 0.125, 0.3), MoeSpec(16, 2, 4672, 9344)),
+    "fatulix-5120": _fatulix("fatulix-5120", 5120, 152064, 6, AttentionSpec(40, 8, 64, 128, 0.125, 0.3), MoeSpec(8, 2, 8192, 8192)),
     "tiny-fatulix": _fatulix("tiny-fatulix", 128, 320, 3, AttentionSpec(6, 2, 24, 32, 0.2, 0.4), MoeSpec(5, 2, 64, 128), LoopSpec(1, 3, 2)),
 }
 

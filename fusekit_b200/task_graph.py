@@ -217,9 +217,10 @@ def _task(tasks, kind, layer, bufs, iargs, fargs=()):
 
 
 def key_splits(mixer, capacity: int, sm: int) -> int:
-    """Blocks the keys of a decode step are split over: two blocks per SM over all kv heads, at least 64 keys of capacity each."""
+    """Blocks the keys of a decode step are split over: two blocks per SM over all kv heads, at most 64 (the last
+    block to finish folds the others' results) and at least 64 keys of capacity each."""
     tiles = -(-(mixer.heads // mixer.kv_heads * mixer.maps) // 8)
-    return max(1, min(-(-2 * sm // (mixer.kv_heads * tiles)), -(-capacity // 64), 8 * round_up(mixer.vdim, 8), 256))
+    return max(1, min(-(-2 * sm // (mixer.kv_heads * tiles)), -(-capacity // 64), 64))
 
 
 def layered_decode_tasks(spec, capacity: int, lambdas: dict, dtype: int = 0, sm: int = 148) -> list:
