@@ -30,7 +30,7 @@ __device__ __forceinline__ void fl_copy16(uint32_t dst, const void *src, bool va
 __device__ __forceinline__ uint32_t fl_pack(float lo, float hi) { const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi); return *reinterpret_cast<const uint32_t *>(&h); }
 
 template <int KD, int VD>
-__global__ void __launch_bounds__(256) k_flash_rows(FkState *st, FlashArgs a) {
+__global__ void __launch_bounds__(256, VD <= 128 && KD <= 64 ? 2 : 1) k_flash_rows(FkState *st, FlashArgs a) {
     extern __shared__ __align__(128) unsigned char fl_smem[];
     constexpr int KS = KD + 8, VS = VD + 8;             // row strides in elements: odd multiples of 16 bytes, so ldmatrix has no conflicts
     const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, g8 = lane >> 2, t4 = lane & 3, map = wid >> 2, nt = blockDim.x;
@@ -79,24 +79,26 @@ __global__ void __launch_bounds__(256) k_flash_rows(FkState *st, FlashArgs a) {
         if (tile + 1 < ntiles) { fetch(tile + 1, (tile + 1) & 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
         else asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
-        if (tile * 64 <= off + wrow + 15) {             // some key of the tile is visible to some row of the warp
-            const uint32_t kb = sbase + (tile & 1) * stage + (uint32_t)(map * 64 * KS * 2), vb = sbase + (tile & 1) * stage + (uint32_t)(a.maps * 64 * KS * 2);
-            float s[8][4];
+        const uint32_t kb = sbase + (tile & 1) * stage + (uint32_t)(map * 64 * KS * 2), vb = sbase + (tile & 1) * stage + (uint32_t)(a.maps * 64 * KS * 2);
+        // 32 keys at a time, as far as some key is visible to some row of the warp
+#pragma unroll 1
+        for (int h0 = 0; h0 < 64 && tile * 64 + h0 <= off + wrow + 15; h0 += 32) {
+            float s[4][4];
 #pragma unroll
-            for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
+            for (int i = 0; i < 4; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
 #pragma unroll
             for (int k = 0; k < KD / 16; ++k)
 #pragma unroll
-                for (int n = 0; n < 4; ++n) {           // 16 keys: matrices (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, ..) x 2
+                for (int n = 0; n < 2; ++n) {           // 16 keys: matrices (keys 0-7, k 0-7), (keys 0-7, k 8-15), (keys 8-15, ..) x 2
                     uint32_t b[4];
-                    fl_ldsm(b, kb + (uint32_t)(((n * 16 + (lane & 7) + ((lane >> 4) << 3)) * KS + k * 16 + ((lane >> 3) & 1) * 8) * 2));
+                    fl_ldsm(b, kb + (uint32_t)(((h0 + n * 16 + (lane & 7) + ((lane >> 4) << 3)) * KS + k * 16 + ((lane >> 3) & 1) * 8) * 2));
                     fl_mma(s[2 * n], qf[k], b[0], b[1]); fl_mma(s[2 * n + 1], qf[k], b[2], b[3]);
                 }
-            const bool edge = tile * 64 + 63 > off + wrow;
+            const bool edge = tile * 64 + h0 + 31 > off + wrow;
             float x0 = -INFINITY, x1 = -INFINITY;
 #pragma unroll
-            for (int i = 0; i < 8; ++i) {
-                const int key = tile * 64 + i * 8 + t4 * 2;
+            for (int i = 0; i < 4; ++i) {
+                const int key = tile * 64 + h0 + i * 8 + t4 * 2;
 #pragma unroll
                 for (int j = 0; j < 2; ++j) {
                     s[i][j] = edge && key + j > pos0 ? -INFINITY : s[i][j] * sc;
@@ -106,13 +108,15 @@ __global__ void __launch_bounds__(256) k_flash_rows(FkState *st, FlashArgs a) {
             }
             x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
             x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
-            const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);         // tile 0 shows every row key 0, so these are finite
-            const float c0 = exp2f(m0 - n0), c1 = exp2f(m1 - n1);
-            m0 = n0; m1 = n1; l0 *= c0; l1 *= c1;
+            const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);         // the first 32 keys show every row key 0, so these are finite
+            if (__any_sync(0xffffffffu, n0 > m0 || n1 > m1)) {          // a new maximum somewhere in the warp
+                const float c0 = exp2f(m0 - n0), c1 = exp2f(m1 - n1);
+                m0 = n0; m1 = n1; l0 *= c0; l1 *= c1;
 #pragma unroll
-            for (int i = 0; i < VD / 8; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
+                for (int i = 0; i < VD / 8; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
+            }
 #pragma unroll
-            for (int k = 0; k < 4; ++k) {               // 16 keys at a time: weights as hi + lo, times the values
+            for (int k = 0; k < 2; ++k) {               // 16 keys at a time: weights as hi + lo, times the values
                 uint32_t ph[4], pl[4];
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
@@ -125,9 +129,9 @@ __global__ void __launch_bounds__(256) k_flash_rows(FkState *st, FlashArgs a) {
 #pragma unroll
                 for (int n = 0; n < VD / 16; ++n) {     // 16 value columns: matrices (keys 0-7 / 8-15) x (columns 0-7 / 8-15), transposed
                     uint32_t b[4];
-                    fl_ldsm_t(b, vb + (uint32_t)(((k * 16 + (lane & 15)) * VS + n * 16 + (lane >> 4) * 8) * 2));
-                    fl_mma(o[2 * n], ph, b[0], b[1]); fl_mma(o[2 * n], pl, b[0], b[1]);
-                    fl_mma(o[2 * n + 1], ph, b[2], b[3]); fl_mma(o[2 * n + 1], pl, b[2], b[3]);
+                    fl_ldsm_t(b, vb + (uint32_t)(((h0 + k * 16 + (lane & 15)) * VS + n * 16 + (lane >> 4) * 8) * 2));
+                    fl_mma(o[2 * n], ph, b[0], b[1]); fl_mma(o[2 * n + 1], ph, b[2], b[3]);
+                    fl_mma(o[2 * n], pl, b[0], b[1]); fl_mma(o[2 * n + 1], pl, b[2], b[3]);
                 }
             }
         }

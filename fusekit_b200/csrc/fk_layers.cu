@@ -63,11 +63,16 @@ static fk_status bad(char *err, size_t cap, const char *fmt, ...) {
 }
 static int round_up(int v, int m) { return (v + m - 1) / m * m; }
 
-// Blocks and K split of a matrix-vector product: one block per SM, and as few warps per row group as give every warp one.
+// Blocks and K split of a matrix-vector product: one block per SM; of the possible splits the one with the shortest critical
+// path, row groups of the busiest block x batches of a warp per group (plus a quarter of a batch to finish a group).
 static cudaError_t launch_gemv(FklEnv &c, int mode, GemvArgs &a) {
     const int groups = (a.n + FKL_GV_R - 1) / FKL_GV_R, slots = c.sm_count;
-    int ks = 1;
-    while (ks < FKL_GV_WARPS && ks * 2 <= a.nchunks && (long long)groups * ks < (long long)slots * FKL_GV_WARPS) ks *= 2;
+    int ks = 1; double best = 1e30;
+    for (int k = 1; k <= FKL_GV_WARPS && k <= a.nchunks; k *= 2) {
+        const int per = FKL_GV_WARPS / k, nblk = (groups + per - 1) / per, rounds = (nblk + slots - 1) / slots, chunks = (a.nchunks + k - 1) / k;
+        const double cost = rounds * ((chunks + FKL_GV_U - 1) / FKL_GV_U + 0.25);
+        if (cost < best - 1e-9) { best = cost; ks = k; }
+    }
     a.kslices = ks;
     const int spb = FKL_GV_WARPS / ks, blocks = (groups + spb - 1) / spb, grid = blocks < slots ? blocks : slots;
     const size_t smem = gv_smem_bytes(a.nchunks);
@@ -130,6 +135,14 @@ fk_status fkl_run(FklEnv &c, const fk_task &t, char *err, size_t ecap) {
         if ((size_t)i[0] * 4 > 200 * 1024) return bad(err, ecap, "residual_norm_rows: width above 51200");
         ResNormArgs a{(const float *)b[0], (const void *)b[1], (const uint16_t *)b[2], (const float *)b[3], (float *)b[4], (const uint16_t *)b[5], (void *)b[6],
                       (const uint32_t *)b[7], (const void *)b[8], (const int *)b[9], (const float *)b[10], i[0], i[3], i[4], i[5], f[0]};
+        if (i[0] % 4 == 0 && i[0] <= 8192 && i[3] % 4 == 0 && i[5] % 4 == 0) {
+            const dim3 g4(i[1]), b4(i[0] <= 512 ? 128 : 256);
+#define RN(T, NV) launch(c, k_residual_norm_rows4<T, NV>, g4, b4, 0, (const FkState *)c.state, a)
+            if (i[2]) e = i[0] <= 1024 ? RN(float, 1) : i[0] <= 2048 ? RN(float, 2) : i[0] <= 4096 ? RN(float, 4) : RN(float, 8);
+            else e = i[0] <= 1024 ? RN(uint16_t, 1) : i[0] <= 2048 ? RN(uint16_t, 2) : i[0] <= 4096 ? RN(uint16_t, 4) : RN(uint16_t, 8);
+#undef RN
+            break;
+        }
         const dim3 g(i[1]), blk(i[0] >= 2048 ? 512 : 256);
         e = i[2] ? launch(c, k_residual_norm_rows<float>, g, blk, (size_t)i[0] * 4, (const FkState *)c.state, a)
                  : launch(c, k_residual_norm_rows<uint16_t>, g, blk, (size_t)i[0] * 4, (const FkState *)c.state, a);

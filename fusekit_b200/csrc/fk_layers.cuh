@@ -53,6 +53,67 @@ struct ResNormArgs {
     const float *x; const void *y; const uint16_t *post_w; const float *add; float *x_out; const uint16_t *norm_w; void *h; const uint32_t *index;
     const void *moe_y; const int *slot; const float *weight; int d, ldh, top, ldy; float eps;
 };
+__device__ __forceinline__ float4 ld4(const uint16_t *p) { const uint2 v = __ldcg(reinterpret_cast<const uint2 *>(p)); return make_float4(bf_lo(v.x), bf_hi(v.x), bf_lo(v.y), bf_hi(v.y)); }
+__device__ __forceinline__ float4 ld4(const float *p) { return __ldcg(reinterpret_cast<const float4 *>(p)); }
+__device__ __forceinline__ void st4(uint16_t *p, float4 v) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
+}
+__device__ __forceinline__ void st4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
+// rows of a multiple of 4 and at most NV * 4 * blockDim.x values: everything in registers, one round of loads
+template <typename T, int NV>
+__global__ void __launch_bounds__(256) k_residual_norm_rows4(const FkState *st, ResNormArgs a) {
+    __shared__ float red[40];
+    const int tid = threadIdx.x, nt = blockDim.x;
+    pdl_wait(); pdl_launch_dependents();
+    const size_t row = a.index ? a.index[blockIdx.x] : blockIdx.x;
+    const bool pend = a.y || a.moe_y;
+    float4 x[NV], y[NV];
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+        const int i = (v * nt + tid) * 4;
+        x[v] = y[v] = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        if (i < a.d) {
+            x[v] = ld4(a.x + row * a.d + i);
+            if (a.y) y[v] = ld4((const T *)a.y + row * a.ldy + i);
+            if (a.add) { const float4 e = ld4(a.add + row * a.d + i); x[v].x += e.x; x[v].y += e.y; x[v].z += e.z; x[v].w += e.w; }
+        }
+    }
+    if (a.moe_y) for (int j = 0; j < a.top; ++j) {
+        const float w = a.weight[row * a.top + j]; const T *src = (const T *)a.moe_y + (size_t)a.slot[row * a.top + j] * a.ldy;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const int i = (v * nt + tid) * 4;
+            if (i < a.d) { const float4 e = ld4(src + i); y[v].x = fmaf(w, e.x, y[v].x); y[v].y = fmaf(w, e.y, y[v].y); y[v].z = fmaf(w, e.z, y[v].z); y[v].w = fmaf(w, e.w, y[v].w); }
+        }
+    }
+    if (pend) {
+        float ss = 0.0f;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) ss = fmaf(y[v].x, y[v].x, fmaf(y[v].y, y[v].y, fmaf(y[v].z, y[v].z, fmaf(y[v].w, y[v].w, ss))));
+        const float ry = inv_rms(block_sum(ss, red), a.d, a.eps);
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const int i = (v * nt + tid) * 4;
+            if (i < a.d) {
+                const float4 p = ld4(a.post_w + i);
+                x[v].x = fmaf(y[v].x * ry, p.x, x[v].x); x[v].y = fmaf(y[v].y * ry, p.y, x[v].y); x[v].z = fmaf(y[v].z * ry, p.z, x[v].z); x[v].w = fmaf(y[v].w * ry, p.w, x[v].w);
+            }
+        }
+    }
+    float ss = 0.0f;
+#pragma unroll
+    for (int v = 0; v < NV; ++v) ss = fmaf(x[v].x, x[v].x, fmaf(x[v].y, x[v].y, fmaf(x[v].z, x[v].z, fmaf(x[v].w, x[v].w, ss))));
+    const float r = inv_rms(block_sum(ss, red), a.d, a.eps);
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+        const int i = (v * nt + tid) * 4;
+        if (i >= a.d) continue;
+        if (a.x_out) st4(a.x_out + row * a.d + i, x[v]);
+        const float4 w = ld4(a.norm_w + i);
+        st4((T *)a.h + (size_t)blockIdx.x * a.ldh + i, make_float4(x[v].x * r * w.x, x[v].y * r * w.y, x[v].z * r * w.z, x[v].w * r * w.w));
+    }
+}
 template <typename T>
 __global__ void __launch_bounds__(512) k_residual_norm_rows(const FkState *st, ResNormArgs a) {
     extern __shared__ float xs[];                       // [d]
@@ -409,11 +470,20 @@ __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st
         const bool is_q = it < RT;
         const float *src = a.qkv + (is_q ? (g * nrow_kv + r0 + it) : (a.H * a.maps + g * a.maps + (it - RT))) * a.dim;
         const uint16_t *w = is_q ? a.qn : a.kn;
-        float ss = 0.0f;
-        for (int i = lane; i < a.dim; i += 32) { const float v = __ldcg(src + i); ss = fmaf(v, v, ss); }
+        float ss = 0.0f, xv[4], wv[4];                  // the first 128 values stay in registers
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const int i = lane + j * 32;
+            xv[j] = i < a.dim ? __ldcg(src + i) : 0.0f; wv[j] = i < a.dim ? bf2f(w[i]) : 0.0f;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; ++j) ss = fmaf(xv[j], xv[j], ss);
+        for (int i = lane + 128; i < a.dim; i += 32) { const float v = __ldcg(src + i); ss = fmaf(v, v, ss); }
         const float r = inv_rms(warp_sum(ss), a.dim, a.eps);
-        for (int i = lane; i < a.dpad; i += 32) {
-            const float v = i < a.dim ? __ldcg(src + i) * r * bf2f(w[i]) : 0.0f;
+#pragma unroll 4
+        for (int j = 0; j * 32 + lane < a.dpad; ++j) {
+            const int i = lane + j * 32;
+            const float v = j < 4 ? xv[j & 3] * r * wv[j & 3] : i < a.dim ? __ldcg(src + i) * r * bf2f(w[i]) : 0.0f;
             if (is_q) qs[it * a.dpad + i] = v * a.scale;
             else { nk[(it - RT) * a.dpad + i] = f2bf(v); if (i < a.dim) ck[((size_t)(it - RT) * a.cap + pos) * a.dpad + i] = f2bf(v); }
         }
@@ -505,25 +575,43 @@ __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st
         __syncthreads();
         if (!s_last) return;
         __threadfence();
-        // factors exp(m - max) / sum of every (split, row), one warp per row
-        for (int r = wid; r < nr; r += NT / 32) {
-            float mx = -INFINITY, ls = 0.0f;
-            for (int p = lane; p < active; p += 32) mx = fmaxf(mx, __ldcg(base + (size_t)p * stride + RT * a.vpad + r * 2));
+        // a thread folds four values; what the first splits left of them is requested before the factors are known
+        constexpr int PRE = 8;
+        float4 pre[PRE];
+        const bool own = tid < nr * a.vpad / 4;
+#pragma unroll
+        for (int p = 0; p < PRE; ++p) pre[p] = own && p < active ? __ldcg(reinterpret_cast<const float4 *>(base + (size_t)p * stride) + tid) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        // factors exp(m - max) / sum of every (split, row): warp r takes row r (there are as many warps as rows of a tile)
+        if (wid < nr) {
+            const int r = wid;
+            float2 ml[2];
+#pragma unroll
+            for (int j = 0; j < 2; ++j) ml[j] = lane + j * 32 < active ? __ldcg(reinterpret_cast<const float2 *>(base + (size_t)(lane + j * 32) * stride + RT * a.vpad) + r) : make_float2(-INFINITY, 0.0f);
+            float mx = fmaxf(ml[0].x, ml[1].x);
+            for (int p = lane + 64; p < active; p += 32) mx = fmaxf(mx, __ldcg(base + (size_t)p * stride + RT * a.vpad + r * 2));
             mx = warp_max(mx);
-            for (int p = lane; p < active; p += 32) {
-                const float f = expf(__ldcg(base + (size_t)p * stride + RT * a.vpad + r * 2) - mx);
-                s_fac[p * RT + r] = f; ls = fmaf(f, __ldcg(base + (size_t)p * stride + RT * a.vpad + r * 2 + 1), ls);
-            }
-            ls = warp_sum(ls);
-            __syncwarp();
-            for (int p = lane; p < active; p += 32) s_fac[p * RT + r] /= ls;
+            float f0 = expf(ml[0].x - mx), f1 = expf(ml[1].x - mx), ls = fmaf(f0, ml[0].y, f1 * ml[1].y);
+            for (int p = lane + 64; p < active; p += 32) ls = fmaf(expf(__ldcg(base + (size_t)p * stride + RT * a.vpad + r * 2) - mx), __ldcg(base + (size_t)p * stride + RT * a.vpad + r * 2 + 1), ls);
+            const float inv = 1.0f / warp_sum(ls);
+            if (lane < active) s_fac[lane * RT + r] = f0 * inv;
+            if (lane + 32 < active) s_fac[(lane + 32) * RT + r] = f1 * inv;
+            for (int p = lane + 64; p < active; p += 32) s_fac[p * RT + r] = expf(__ldcg(base + (size_t)p * stride + RT * a.vpad + r * 2) - mx) * inv;
         }
         __syncthreads();
         for (int i = tid; i < nr * a.vpad / 4; i += NT) {
             const int r = i * 4 / a.vpad;
             float4 s = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+            int p = 0;
+            if (i == tid) {
+#pragma unroll
+                for (int q = 0; q < PRE; ++q) if (q < active) {
+                    const float f = s_fac[q * RT + r];
+                    s.x = fmaf(f, pre[q].x, s.x); s.y = fmaf(f, pre[q].y, s.y); s.z = fmaf(f, pre[q].z, s.z); s.w = fmaf(f, pre[q].w, s.w);
+                }
+                p = PRE;
+            }
 #pragma unroll 8
-            for (int p = 0; p < active; ++p) {
+            for (; p < active; ++p) {
                 const float4 v = __ldcg(reinterpret_cast<const float4 *>(base + (size_t)p * stride) + i); const float f = s_fac[p * RT + r];
                 s.x = fmaf(f, v.x, s.x); s.y = fmaf(f, v.y, s.y); s.z = fmaf(f, v.z, s.z); s.w = fmaf(f, v.w, s.w);
             }
@@ -629,7 +717,7 @@ __global__ void __launch_bounds__(256) k_moe_gather(const FkState *st, RouteArgs
 
 // ---------------------------------------------------------------- one row: matrix-vector products over bf16 rows
 // A warp owns R = 2 weight rows at a time and streams them in chunks of 256 weights (16 bytes per lane and row), two batches
-// of U = 4 chunks in registers: one being multiplied, one in flight.  The activations sit in shared memory as fp32, in the
+// of U = 4 chunks in two register buffers: one being multiplied, one in flight.  The activations sit in shared memory as fp32, in the
 // order the lanes read them without bank conflicts.  With few rows, 2 .. 16 warps of a block share a row group and split K.
 // A chunk is described by (base of row 0, row stride, weights in it), which also expresses the concatenated K ranges of a
 // mixture's down projection.  The first batch is fetched before the dependency wait where the rows do not depend on it.
@@ -660,7 +748,7 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
     extern __shared__ __align__(16) unsigned char gv_smem[];
     constexpr int R = FKL_GV_R, U = FKL_GV_U, NT = FKL_GV_WARPS * 32;
     float *xs = reinterpret_cast<float *>(gv_smem); GvChunk *tab = reinterpret_cast<GvChunk *>(gv_smem + (size_t)a.nchunks * 1024);
-    __shared__ float red[40], part[FKL_GV_WARPS][R], tval[FKL_MAX_TOP]; __shared__ int tsel[FKL_MAX_TOP];
+    __shared__ float red[40], part[2][FKL_GV_WARPS][R], tval[FKL_MAX_TOP]; __shared__ int tsel[FKL_MAX_TOP];
     __shared__ unsigned long long wbest[FKL_GV_WARPS]; __shared__ int is_last;
     __shared__ float slog[MODE == FKL_GV_MOE_UP ? FKL_MAX_EXPERTS : 1];
     const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, KS = a.kslices, spb = FKL_GV_WARPS / KS, ksl = wid % KS, slot = wid / KS;
@@ -676,17 +764,17 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
             roff[r] = (size_t)row;
         }
     };
-    uint4 nxt[U][R];
-    auto fetch = [&](int c) {
+    uint4 buf0[U][R], buf1[U][R];
+    auto fetch = [&](uint4 (&dst)[U][R], int c) {
 #pragma unroll
         for (int u = 0; u < U; ++u) {
             if (c + u < c1) {
                 const GvChunk ch = tab[c + u];
 #pragma unroll
-                for (int r = 0; r < R; ++r) nxt[u][r] = lane * 8 < ch.len ? ldg_stream(ch.base + roff[r] * ch.stride + lane * 8) : make_uint4(0, 0, 0, 0);
+                for (int r = 0; r < R; ++r) dst[u][r] = lane * 8 < ch.len ? ldg_stream(ch.base + roff[r] * ch.stride + lane * 8) : make_uint4(0, 0, 0, 0);
             } else {
 #pragma unroll
-                for (int r = 0; r < R; ++r) nxt[u][r] = make_uint4(0, 0, 0, 0);
+                for (int r = 0; r < R; ++r) dst[u][r] = make_uint4(0, 0, 0, 0);
             }
         }
     };
@@ -694,7 +782,7 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
     if (MODE != FKL_GV_MOE_DOWN) {
         for (int c = tid; c < a.nchunks; c += NT) tab[c] = GvChunk{a.w + c * 256, a.ldk, min(256, a.ldk - c * 256)};
         __syncthreads();
-        if (MODE == FKL_GV_LINEAR && g < groups && nb > 0) { set_rows(g); fetch(c0); }
+        if (MODE == FKL_GV_LINEAR && g < groups && nb > 0) { set_rows(g); fetch(buf0, c0); }
     }
     uint2 pw[NV > 0 ? NV : 1], nw[NV > 0 ? NV : 1];
     if (NV > 0 && a.norm_w) {
@@ -718,7 +806,7 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
         }
         (void)nshared;
         __syncthreads();
-        if (g < groups && nb > 0) { set_rows(g); fetch(c0); }
+        if (g < groups && nb > 0) { set_rows(g); fetch(buf0, c0); }
         for (int j = 0; j < a.top; ++j) for (int i = tid; i < a.ff; i += NT) xs[gv_place(j * nce * 256 + i)] = tval[j] * __ldcg(a.x + j * a.ff + i);
         for (int i = tid; i < a.ffs; i += NT) xs[gv_place(a.top * nce * 256 + i)] = __ldcg(a.sact + i);
         __syncthreads();
@@ -734,7 +822,7 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
             }
         }
         __syncthreads();
-        if (g < groups && nb > 0) { set_rows(g); fetch(c0); }
+        if (g < groups && nb > 0) { set_rows(g); fetch(buf0, c0); }
     } else if (NV > 0 && a.norm_w) {
         float4 x[NV > 0 ? NV : 1], y[NV > 0 ? NV : 1];
 #pragma unroll
@@ -802,42 +890,37 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
     }
     // ---- rows
     unsigned long long best = 0ull;
-    const int rounds = (groups + gstride - 1) / gstride;          // the same for all blocks and warps (K split: barriers inside)
-    for (int rd = 0; rd < rounds; ++rd, g += gstride) {
-        if (KS == 1 && g >= groups) break;
-        const bool live = g < groups;
-        float acc[R] = {};
-        if (live) for (int b = 0; b < nb; ++b) {
-            uint4 cur[U][R];
+    float acc[R] = {};
+    int bi = 0, parity = 0;
+    // one batch: request the next one (of this row group or the following) into the other buffer, multiply this one; after a
+    // group's last batch, fold the lanes (and the warps that share the group, behind a barrier of their own) and store
+    auto step = [&](uint4 (&cur)[U][R], uint4 (&next)[U][R]) {
+        const bool last = bi + 1 == nb;
+        if (!last) fetch(next, c0 + (bi + 1) * U);
+        else if (g + gstride < groups) { set_rows(g + gstride); fetch(next, c0); }
 #pragma unroll
-            for (int u = 0; u < U; ++u)
+        for (int u = 0; u < U; ++u) {
+            const int c = c0 + bi * U + u;
+            if (c < c1) {
+                const float4 x0 = *reinterpret_cast<const float4 *>(xs + c * 256 + lane * 4), x1 = *reinterpret_cast<const float4 *>(xs + c * 256 + 128 + lane * 4);
 #pragma unroll
-                for (int r = 0; r < R; ++r) cur[u][r] = nxt[u][r];
-            if (b + 1 < nb) fetch(c0 + (b + 1) * U);
-            else if (g + gstride < groups) { set_rows(g + gstride); fetch(c0); }
-#pragma unroll
-            for (int u = 0; u < U; ++u) {
-                const int c = c0 + b * U + u;
-                if (c < c1) {
-                    const float4 x0 = *reinterpret_cast<const float4 *>(xs + c * 256 + lane * 4), x1 = *reinterpret_cast<const float4 *>(xs + c * 256 + 128 + lane * 4);
-#pragma unroll
-                    for (int r = 0; r < R; ++r) {
-                        float f[8]; unpack8f(cur[u][r], f);
-                        acc[r] = fmaf(f[0], x0.x, fmaf(f[1], x0.y, fmaf(f[2], x0.z, fmaf(f[3], x0.w, acc[r]))));
-                        acc[r] = fmaf(f[4], x1.x, fmaf(f[5], x1.y, fmaf(f[6], x1.z, fmaf(f[7], x1.w, acc[r]))));
-                    }
+                for (int r = 0; r < R; ++r) {
+                    float f[8]; unpack8f(cur[u][r], f);
+                    acc[r] = fmaf(f[0], x0.x, fmaf(f[1], x0.y, fmaf(f[2], x0.z, fmaf(f[3], x0.w, acc[r]))));
+                    acc[r] = fmaf(f[4], x1.x, fmaf(f[5], x1.y, fmaf(f[6], x1.z, fmaf(f[7], x1.w, acc[r]))));
                 }
             }
         }
+        if (!last) { ++bi; return; }
 #pragma unroll
         for (int r = 0; r < R; ++r) acc[r] = warp_sum(acc[r]);
         if (KS > 1) {
-            if (lane == 0) for (int r = 0; r < R; ++r) part[wid][r] = acc[r];
-            __syncthreads();
-            if (ksl == 0) for (int r = 0; r < R; ++r) for (int q = 1; q < KS; ++q) acc[r] += part[wid + q][r];
-            __syncthreads();
+            if (lane == 0) for (int r = 0; r < R; ++r) part[parity][wid][r] = acc[r];
+            asm volatile("bar.sync %0, %1;" ::"r"(1 + slot), "r"(KS * 32) : "memory");
+            if (ksl == 0) for (int r = 0; r < R; ++r) for (int q = 1; q < KS; ++q) acc[r] += part[parity][wid + q][r];
+            parity ^= 1;                               // the next group writes the other half while this one is still being read
         }
-        if (live && ksl == 0) {
+        if (ksl == 0) {
 #pragma unroll
             for (int r = 0; r < R; ++r) {
                 const int row = g * R + r;
@@ -852,6 +935,14 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
                 }
             }
         }
+#pragma unroll
+        for (int r = 0; r < R; ++r) acc[r] = 0.0f;
+        bi = 0; g += gstride;
+    };
+    while (g < groups) {
+        step(buf0, buf1);
+        if (g >= groups) break;
+        step(buf1, buf0);
     }
     if (MODE != FKL_GV_LINEAR || !a.amax) return;
     if (lane == 0) wbest[wid] = best;

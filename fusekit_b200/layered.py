@@ -11,7 +11,6 @@ router), "float32" keeps everything in fp32.  Weights are bf16 as stored in eith
 """
 from __future__ import annotations
 
-import ctypes as C
 import math
 
 import numpy as np
@@ -19,7 +18,7 @@ import numpy as np
 from . import _native as N
 from . import task_graph as TG
 from .model_spec import LayeredSpec, stream_id
-from .runtime import EngineBase, Runtime, sample_logits
+from .runtime import EngineBase, Runtime
 
 MAX_ROWS = 2048          # positions per portion of a prompt
 
@@ -85,7 +84,7 @@ class Sequence:
 
 class LayeredEngine(EngineBase):
     def __init__(self, spec: LayeredSpec, capacity: int, device: int = 0, dtype: str = "bfloat16", max_rows: int = MAX_ROWS,
-                 runtime: Runtime | None = None, want_logits: bool = True):
+                 runtime: Runtime | None = None, want_logits: bool = True):          # fp32 logits are always kept
         if dtype not in ("bfloat16", "float32"):
             raise ValueError(f"dtype {dtype!r}: bfloat16 or float32")
         if capacity < 1 or max_rows < 1:
@@ -339,22 +338,11 @@ class LayeredEngine(EngineBase):
         with the embedding output added)."""
         return self.rt.download(self.X, (len(self.spec.runs()) + 1, self.spec.hidden), np.float32)
 
-    def complete(self, prompt, max_tokens: int, temperature: float = 0.0, top_k: int = 0, top_p: float = 1.0, seed: int = 0) -> np.ndarray:
-        """Generate ``max_tokens`` tokens after ``prompt`` in a slot of its own: greedy on the device, or sampled on the host from the
-        logits of every step."""
+    def complete(self, prompt, max_tokens: int, *args, **kw) -> np.ndarray:
+        """A completion in a slot of its own (see EngineBase.complete)."""
         seq = self.open_sequence()
         try:
             self.select(seq.slot)
-            if temperature <= 0.0 or top_k == 1:
-                first = self.prefill(prompt)
-                rest = self.generate(first, len(prompt), max_tokens - 1)[0] if max_tokens > 1 else np.empty(0, np.uint32)
-                return np.concatenate([[first], rest]).astype(np.uint32)[:max_tokens]
-            rng = np.random.default_rng(seed)
-            out, logits = [], seq.append(prompt, [len(prompt) - 1])[0]
-            while True:
-                out.append(sample_logits(logits, temperature, top_k, top_p, rng))
-                if len(out) == max_tokens:
-                    return np.array(out, np.uint32)
-                logits = seq.append(out[-1:], [0])[0]
+            return super().complete(prompt, max_tokens, *args, **kw)
         finally:
             seq.close()

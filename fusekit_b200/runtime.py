@@ -300,6 +300,27 @@ class EngineBase:
             toks.append(tok)
         return np.array(toks, np.uint32)
 
+    def prefill(self, tokens, base_offset: int = 0) -> int:
+        """Run a prompt position by position; the greedy token after its last position."""
+        out = None
+        for i, t in enumerate(tokens):
+            out, _ = self.decode_chunk(base_offset + i, int(t), 1)
+        return int(out[0])
+
+    def complete(self, prompt, max_tokens: int, temperature: float = 0.0, top_k: int = 0, top_p: float = 1.0, seed: int = 0) -> np.ndarray:
+        """``max_tokens`` tokens after ``prompt`` from an empty cache: greedy with on-device feedback, or sampled on the host from
+        the logits of every step."""
+        prompt = [int(t) for t in prompt]
+        if not prompt or max_tokens < 1:
+            raise ValueError("a completion needs a prompt and at least one token to generate")
+        if temperature <= 0.0 or top_k == 1:
+            first = self.prefill(prompt)
+            rest = self.generate(first, len(prompt), max_tokens - 1)[0] if max_tokens > 1 else []
+            return np.array([first, *rest], np.uint32)
+        if len(prompt) > 1:
+            self.prefill(prompt[:-1])
+        return self.generate_sampled(prompt[-1], len(prompt) - 1, max_tokens, temperature, top_k, top_p, seed)
+
     def profile_nodes(self, repeats: int = 3):
         if not self.graph:
             self.capture()

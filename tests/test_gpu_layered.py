@@ -418,10 +418,29 @@ def test_greedy_and_sampled_generation(runtime, tmp_path, name):
                 toks = [int(np.argmax(z))]; want += toks
             assert e.complete(prompt, 30).tolist() == want
             assert e.complete(prompt, 5, temperature=0.7, top_k=1).tolist() == want[:5]
-            a, b = (e.complete(prompt, 6, temperature=1.2, top_k=8, seed=3).tolist() for _ in range(2))
+            a, b = (e.complete(prompt, 6, 1.2, top_k=8, seed=3).tolist() for _ in range(2))
             assert a == b and max(a) < s.vocab
     finally:
         ck.close()
+
+
+@pytest.mark.parametrize("which", ["model", "layered", "older"])
+def test_command_line(tmp_path, capsys, which):
+    from fusekit_b200.generate import main
+    if which == "model":
+        s = LM.SPECS["mixed"]
+        t = LM.random_tensors(s, 8)
+        LM.write_model(tmp_path / "m", s, t)
+        o, want, toks = LM.oracle(s, t), [], [3, 1, 4]
+        for _ in range(6):
+            toks = [int(np.argmax(o.forward(toks)[-1]))]; want += toks
+        assert main(["--model", str(tmp_path / "m"), "--dtype", "float32", "--prompt", "3,1,4", "--max-tokens", "6"]) == 0
+        assert [int(v) for v in capsys.readouterr().out.split(",")] == want
+        return
+    args = ["--config", "tiny-fatulix" if which == "layered" else "tiny-qwen", "--prompt", "3,1,4", "--max-tokens", "6"]
+    assert main(args) == 0 and main(args + ["--temperature", "0.8", "--top-k", "1"]) == 0
+    a, b = capsys.readouterr().out.split()
+    assert a == b and len(a.split(",")) == 6
 
 
 def test_registered_shape_through_attach(runtime):
