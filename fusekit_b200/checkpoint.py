@@ -341,6 +341,8 @@ def load_engine(path: str, capacity: int, device: int = 0, tp_rank: int = 0, tp_
         leng.load_from(lck.provider())
         return leng, lck
     from .runtime import DecodeEngine
+    if kw.pop("dtype", None) == "float32":
+        raise ValueError("only layered decoders run in 32-bit")
     ck = Checkpoint(path)
     eng = DecodeEngine(ck.spec, capacity, device=device, tp_rank=tp_rank, tp_size=tp_size, **kw)
     eng.load_from(ck.weight_provider(), ck.vector_provider(), ck.embed_provider())

@@ -47,6 +47,8 @@ def main(argv=None) -> int:
     args = ap.parse_args(argv)
     engine, ck = load_engine(args.model, max(args.max_tokens, 1), dtype=args.dtype)
     try:
+        if not hasattr(engine, "open_sequence"):
+            raise ValueError(f"trace replay runs layered decoders; {args.model} holds a {ck.spec.arch} model")
         runner = TraceRunner(engine, args.out)
         for line in sys.stdin:
             if line.strip():
