@@ -16,9 +16,11 @@ LIB_PATH = os.environ.get("FUSEKIT_CUDA_LIB") or os.path.join(_HERE, "libfusekit
  TASK_LINEAR_RESIDUAL, TASK_RMSNORM_GATEUP_ACT, TASK_FINAL_RMSNORM_LM_HEAD, TASK_ARGMAX_FINALIZE,
  TASK_ALLREDUCE, TASK_RESIDUAL_ADD, TASK_RMSNORM_ROWS, TASK_ROPE_STORE_ROWS, TASK_ARGMAX_ROWS, TASK_KV_STORE_QUANT,
  TASK_SDPA_DECODE_QUANT, TASK_EMBED_ROWS, TASK_RESIDUAL_NORM_ROWS, TASK_LINEAR_ROWS, TASK_QK_NORM_STORE_ROWS, TASK_ATTENTION_ROWS,
- TASK_MOE_ROUTE_ROWS, TASK_NORM_LINEAR, TASK_ATTENTION_DECODE, TASK_MOE_UP, TASK_MOE_DOWN, TASK_ARGMAX_ROW) = range(27)
+ TASK_MOE_ROUTE_ROWS, TASK_NORM_LINEAR, TASK_ATTENTION_DECODE, TASK_MOE_UP, TASK_MOE_DOWN, TASK_ARGMAX_ROW, TASK_BLOCK_NORM_ROWS,
+ TASK_BLOCK_LINEAR_ROWS, TASK_ROTARY_STORE_ROWS, TASK_WINDOW_ATTENTION_ROWS, TASK_WINDOW_ATTENTION_DECODE, TASK_RECURRENCE_ROWS,
+ TASK_RECURRENCE_DECODE, TASK_NORM_GATE_ROWS, TASK_SEGMENT_LINEAR) = range(36)
 ACT_SWIGLU, ACT_GEGLU_TANH = 0, 1
-ACT_NONE, ACT_RELU_SQUARED = 0, 2
+ACT_NONE, ACT_RELU_SQUARED, ACT_SILU = 0, 2, 3
 
 
 class RoleBinding(C.Structure):

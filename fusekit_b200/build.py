@@ -8,7 +8,7 @@ import sys
 HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OUT = os.path.join(HERE, "libfusekit_cuda.so")
-SOURCES = ["fk_runtime.cu", "fk_layers.cu"]        # compiled side by side, linked into one library
+SOURCES = ["fk_runtime.cu", "fk_layers.cu", "fk_blocks.cu"]        # compiled side by side, linked into one library
 FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-O3", "-lineinfo", "-std=c++17",
          "-Xcompiler", "-fPIC", "-ccbin", "/usr/bin/g++"]
 

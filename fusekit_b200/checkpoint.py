@@ -26,7 +26,8 @@ import struct
 
 import numpy as np
 
-from .model_spec import AttentionSpec, LayeredSpec, LayerSpec, LoopSpec, ModelSpec, MoeSpec
+from .model_spec import (AttentionSpec, ClampedGluSpec, FrequencyScaling, LayeredSpec, LayerSpec, LightningSpec, LoopSpec, MatrixMemorySpec, ModelSpec,
+                         MoeSpec, ParallelMixerSpec, RotarySpec)
 
 _DT = {"U32": (np.uint32, 4), "I32": (np.int32, 4), "BF16": (np.uint16, 2), "F16": (np.float16, 2), "F32": (np.float32, 4),
        "U8": (np.uint8, 1), "I64": (np.int64, 8), "U16": (np.uint16, 2)}
@@ -152,15 +153,42 @@ def spec_from_config(cfg: dict, name: str = "checkpoint") -> ModelSpec:
                      window=window, global_every=every)
 
 
-LAYERED_ARCHITECTURES = ("Fatulix",)
+LAYERED_ARCHITECTURES = ("Fatulix", "Kakunex")
+
+
+def _rotary(rot: dict | None) -> RotarySpec | None:
+    if not rot:
+        return None
+    s = rot.get("scaling")
+    return RotarySpec(int(rot["dims"]), float(rot["base"]), FrequencyScaling(*(float(s[k]) for k in ("factor", "low", "high", "original"))) if s else None)
+
+
+def _parallel_layer(i: int, e: dict) -> LayerSpec:
+    """A layer of a parallel block: mixer type "parallel" (attention left, linear attention right) or "mlstm"; dense feed-forward or none."""
+    m, f = e["mixer"], e.get("mlp")
+    if e["type"] == "parallel":
+        l, r, mask = m["left"], m["right"], m["left"].get("mask") or {}
+        left = AttentionSpec(int(l["heads"]), int(l["kv_heads"]), int(l["dim"]), int(l["vdim"]), float(l["scale"]), norm="projection", gate=False, rotary=_rotary(l.get("rot")),
+                             window=int(mask["size"]) if mask.get("size") is not None else None, keep_first=int(mask.get("keep_first") or 0))
+        mixer = ParallelMixerSpec(left, LightningSpec(int(r["heads"]), int(r["dim"]), int(r["vdim"]), tuple(float(d) for d in r["decay"])))
+    elif e["type"] == "mlstm":
+        mixer = MatrixMemorySpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
+    else:
+        raise ValueError(f"layer {i}: mixer type {e['type']!r} is not supported (parallel, mlstm)")
+    if f is not None and f["kind"] != "dense":
+        raise ValueError(f"layer {i}: feed-forward kind {f['kind']!r} is not supported (dense)")
+    return LayerSpec(mixer, ClampedGluSpec(int(f["ff"]), float(f["limit"])) if f is not None else None)
 
 
 def layered_spec_from_config(cfg: dict, name: str = "checkpoint") -> LayeredSpec:
     """config.json of a layered decoder: ``architecture``, ``width``, ``vocab``, ``norm.eps``, ``layers`` (each ``type``, ``mixer``,
-    ``mlp`` or null) and an optional ``loop``.  Anything this build has no mechanism for is refused by name."""
+    ``mlp`` or null), an optional ``loop`` (Fatulix), ``logit_scale`` (Kakunex).  Anything this build has no mechanism for is refused by name."""
     arch = cfg.get("architecture")
     if arch not in LAYERED_ARCHITECTURES:
         raise ValueError(f"architecture {arch!r} has no decode path here ({', '.join(LAYERED_ARCHITECTURES)})")
+    if arch == "Kakunex":
+        return LayeredSpec(name=name, arch=arch, hidden=int(cfg["width"]), vocab=int(cfg["vocab"]), layers=tuple(_parallel_layer(i, e) for i, e in enumerate(cfg["layers"])),
+                           eps=float(cfg["norm"]["eps"]), block="parallel", logit_scale=float(cfg["logit_scale"]))
     layers = []
     for i, e in enumerate(cfg["layers"]):
         if e["type"] != "attention":
@@ -312,7 +340,7 @@ class Checkpoint(TensorFiles):
 
 
 class LayeredCheckpoint(TensorFiles):
-    """A model directory of a layered decoder: tensors ``embed``, ``head``, ``final.norm`` and ``l<i>.<name>``, bf16."""
+    """A model directory of a layered decoder: tensors ``embed``, ``head`` (unless tied), ``final.norm`` and ``l<i>.<name>``, bf16."""
 
     def __init__(self, path: str):
         super().__init__(path)

@@ -5,11 +5,12 @@
 // time, through a double-buffered shared-memory tile (cp.async) of the maps' keys and the one set of values.  Scores and the
 // online softmax are fp32; a weight enters the value product as two bf16 terms (hi + lo), which keeps it at fp32 grade.  At the
 // end the second map's warps hand their result over in shared memory and the first map's apply a1 - lambda a2, the unit rms, the
-// factor 1 - diff and the output gate.  KD / VD: head sizes padded to the instance (zero columns).
+// factor 1 - diff and the output gate.  KD / VD: head sizes padded to the instance (zero columns).  With a window the block walks the
+// tiles of the kept first keys and those from the oldest key its first position sees; a tile may hide all of a row's keys.
 #pragma once
 #include "fk_layers.cuh"
 
-struct FlashArgs { const uint16_t *q, *ck, *cv, *gate; uint16_t *out; int H, G, maps, vdim, dpad, vpad, cap, ldo, ldg, rows; float scale, lambda, diff, eps; };
+struct FlashArgs { const uint16_t *q, *ck, *cv, *gate; uint16_t *out; int H, G, maps, vdim, dpad, vpad, cap, ldo, ldg, rows; float scale, lambda, diff, eps; int window, keep; };
 template <int KD, int VD> __host__ __device__ constexpr size_t flash_stage_bytes(int maps) { return (size_t)64 * 2 * ((size_t)maps * (KD + 8) + (VD + 8)); }
 template <int KD, int VD> __host__ __device__ constexpr size_t flash_smem_bytes(int maps) {
     return 2 * flash_stage_bytes<KD, VD>(maps) > (size_t)64 * (VD + 2) * 4 ? 2 * flash_stage_bytes<KD, VD>(maps) : (size_t)64 * (VD + 2) * 4;
@@ -29,7 +30,7 @@ __device__ __forceinline__ void fl_copy16(uint32_t dst, const void *src, bool va
 }
 __device__ __forceinline__ uint32_t fl_pack(float lo, float hi) { const __nv_bfloat162 h = __floats2bfloat162_rn(lo, hi); return *reinterpret_cast<const uint32_t *>(&h); }
 
-template <int KD, int VD>
+template <int KD, int VD, bool WIN>
 __global__ void __launch_bounds__(256, VD <= 128 && KD <= 64 ? 2 : 1) k_flash_rows(FkState *st, FlashArgs a) {
     extern __shared__ __align__(128) unsigned char fl_smem[];
     constexpr int KS = KD + 8, VS = VD + 8;             // row strides in elements: odd multiples of 16 bytes, so ldmatrix has no conflicts
@@ -39,7 +40,8 @@ __global__ void __launch_bounds__(256, VD <= 128 && KD <= 64 ? 2 : 1) k_flash_ro
     const int off = (int)st->offset;
     const int last = off + min(row0 + 63, a.rows - 1);  // newest position of the block
     if (off + a.rows > a.cap) return;                   // reported by the cache store that came before
-    const int ntiles = last / 64 + 1;
+    const int wtile = WIN ? max(0, off + row0 - a.window + 1) / 64 : 0, kept = WIN ? min((a.keep + 63) / 64, wtile) : 0, ntiles = kept + last / 64 - wtile + 1;
+    auto place = [&](int i) { return i < kept ? i : wtile + i - kept; };
     const uint32_t sbase = (uint32_t)__cvta_generic_to_shared(fl_smem), stage = (uint32_t)flash_stage_bytes<KD, VD>(a.maps);
     const uint16_t *ck = a.ck + (size_t)g * a.maps * a.cap * a.dpad, *cv = a.cv + (size_t)g * a.cap * a.vpad;
     auto fetch = [&](int tile, int s) {
@@ -56,7 +58,7 @@ __global__ void __launch_bounds__(256, VD <= 128 && KD <= 64 ? 2 : 1) k_flash_ro
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(0, 0);
+    fetch(place(0), 0);
     // the warp's query rows as A fragments
     uint32_t qf[KD / 16][4];
     {
@@ -75,14 +77,16 @@ __global__ void __launch_bounds__(256, VD <= 128 && KD <= 64 ? 2 : 1) k_flash_ro
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.0f, l1 = 0.0f;
     const float sc = a.scale * 1.44269504088896341f;     // scores in base-2 exponents
     const int pos0 = off + wrow + g8, pos1 = pos0 + 8;
-    for (int tile = 0; tile < ntiles; ++tile) {
-        if (tile + 1 < ntiles) { fetch(tile + 1, (tile + 1) & 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
+    for (int it = 0; it < ntiles; ++it) {
+        const int tile = place(it);
+        if (it + 1 < ntiles) { fetch(place(it + 1), (it + 1) & 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
         else asm volatile("cp.async.wait_group 0;" ::: "memory");
         __syncthreads();
-        const uint32_t kb = sbase + (tile & 1) * stage + (uint32_t)(map * 64 * KS * 2), vb = sbase + (tile & 1) * stage + (uint32_t)(a.maps * 64 * KS * 2);
+        const uint32_t kb = sbase + (it & 1) * stage + (uint32_t)(map * 64 * KS * 2), vb = sbase + (it & 1) * stage + (uint32_t)(a.maps * 64 * KS * 2);
         // 32 keys at a time, as far as some key is visible to some row of the warp
 #pragma unroll 1
         for (int h0 = 0; h0 < 64 && tile * 64 + h0 <= off + wrow + 15; h0 += 32) {
+            if (WIN && tile * 64 + h0 >= a.keep && tile * 64 + h0 + 31 <= off + wrow - a.window) continue;
             float s[4][4];
 #pragma unroll
             for (int i = 0; i < 4; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
@@ -94,23 +98,25 @@ __global__ void __launch_bounds__(256, VD <= 128 && KD <= 64 ? 2 : 1) k_flash_ro
                     fl_ldsm(b, kb + (uint32_t)(((h0 + n * 16 + (lane & 7) + ((lane >> 4) << 3)) * KS + k * 16 + ((lane >> 3) & 1) * 8) * 2));
                     fl_mma(s[2 * n], qf[k], b[0], b[1]); fl_mma(s[2 * n + 1], qf[k], b[2], b[3]);
                 }
-            const bool edge = tile * 64 + h0 + 31 > off + wrow;
+            const bool edge = tile * 64 + h0 + 31 > off + wrow || (WIN && tile * 64 + h0 <= off + wrow + 15 - a.window);
+            auto hidden = [&](int k, int p) { return k > p || (WIN && p - k >= a.window && k >= a.keep); };
             float x0 = -INFINITY, x1 = -INFINITY;
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
                 const int key = tile * 64 + h0 + i * 8 + t4 * 2;
 #pragma unroll
                 for (int j = 0; j < 2; ++j) {
-                    s[i][j] = edge && key + j > pos0 ? -INFINITY : s[i][j] * sc;
-                    s[i][2 + j] = edge && key + j > pos1 ? -INFINITY : s[i][2 + j] * sc;
+                    s[i][j] = edge && hidden(key + j, pos0) ? -INFINITY : s[i][j] * sc;
+                    s[i][2 + j] = edge && hidden(key + j, pos1) ? -INFINITY : s[i][2 + j] * sc;
                     x0 = fmaxf(x0, s[i][j]); x1 = fmaxf(x1, s[i][2 + j]);
                 }
             }
             x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 1)); x0 = fmaxf(x0, __shfl_xor_sync(0xffffffffu, x0, 2));
             x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 1)); x1 = fmaxf(x1, __shfl_xor_sync(0xffffffffu, x1, 2));
-            const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);         // the first 32 keys show every row key 0, so these are finite
+            const float n0 = fmaxf(m0, x0), n1 = fmaxf(m1, x1);
+            const float e0 = WIN && n0 == -INFINITY ? 0.0f : n0, e1 = WIN && n1 == -INFINITY ? 0.0f : n1;       // no key seen yet: every factor is 0
             if (__any_sync(0xffffffffu, n0 > m0 || n1 > m1)) {          // a new maximum somewhere in the warp
-                const float c0 = exp2f(m0 - n0), c1 = exp2f(m1 - n1);
+                const float c0 = exp2f(m0 - e0), c1 = exp2f(m1 - e1);
                 m0 = n0; m1 = n1; l0 *= c0; l1 *= c1;
 #pragma unroll
                 for (int i = 0; i < VD / 8; ++i) { o[i][0] *= c0; o[i][1] *= c0; o[i][2] *= c1; o[i][3] *= c1; }
@@ -121,7 +127,7 @@ __global__ void __launch_bounds__(256, VD <= 128 && KD <= 64 ? 2 : 1) k_flash_ro
 #pragma unroll
                 for (int h = 0; h < 2; ++h) {
                     const int i = 2 * k + h;
-                    const float p0 = exp2f(s[i][0] - m0), p1 = exp2f(s[i][1] - m0), p2 = exp2f(s[i][2] - m1), p3 = exp2f(s[i][3] - m1);
+                    const float p0 = exp2f(s[i][0] - e0), p1 = exp2f(s[i][1] - e0), p2 = exp2f(s[i][2] - e1), p3 = exp2f(s[i][3] - e1);
                     l0 += p0 + p1; l1 += p2 + p3;
                     ph[2 * h] = fl_pack(p0, p1); ph[2 * h + 1] = fl_pack(p2, p3);
                     pl[2 * h] = fl_pack(p0 - bf_lo(ph[2 * h]), p1 - bf_hi(ph[2 * h])); pl[2 * h + 1] = fl_pack(p2 - bf_lo(ph[2 * h + 1]), p3 - bf_hi(ph[2 * h + 1]));

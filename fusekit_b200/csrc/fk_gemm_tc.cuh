@@ -19,7 +19,7 @@ template <int BN> struct TcTile {
     static constexpr int A_BYTES = 128 * FKL_TC_BK * 2, B_BYTES = BN * FKL_TC_BK * 2, STAGE = A_BYTES + B_BYTES, COLS = 2 * BN;
     static constexpr size_t SMEM = (size_t)STAGES * STAGE + 1024;
 };
-struct TcGemmArgs { void *y; const int *offsets; int m, n, kblocks, row0, ldy, act, out_f32, experts; };
+struct TcGemmArgs { void *y; const int *offsets; int m, n, kblocks, row0, ldy, act, out_f32, experts; float scale; BlockCols b; };       // b: BLOCK form
 
 __device__ __forceinline__ uint32_t tcg_smem(const void *p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void tcg_init(uint32_t bar, uint32_t count) { asm volatile("mbarrier.init.shared::cta.b64 [%0], %1;" ::"r"(bar), "r"(count) : "memory"); }
@@ -40,7 +40,7 @@ __device__ __forceinline__ void tcg_load(uint32_t dst, const CUtensorMap *map, i
 __device__ __forceinline__ uint64_t tcg_desc(uint32_t addr) {
     return (uint64_t)((addr >> 4) & 0x3FFFu) | (1ull << 16) | ((uint64_t)(1024 >> 4) << 32) | (1ull << 46) | (2ull << 61);
 }
-template <int BN>
+template <int BN, bool BLOCK>
 __global__ void __launch_bounds__(FKL_TC_THREADS, 1) k_gemm_tc(FkState *st, const __grid_constant__ CUtensorMap mx, const __grid_constant__ CUtensorMap mw, TcGemmArgs a) {
     using T = TcTile<BN>;
     constexpr int S = T::STAGES;
@@ -158,12 +158,34 @@ __global__ void __launch_bounds__(FKL_TC_THREADS, 1) k_gemm_tc(FkState *st, cons
                 asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
                 const int col = n0 + c;
                 if (row >= mend || col >= a.n) continue;
+                if (BLOCK && col >= a.b.exact) {            // 16 (gate, up) pairs
+                    uint16_t *y = (uint16_t *)a.b.y3 + (size_t)row * a.b.ld3 + (col - a.b.exact) / 2;
+                    float v[16];
 #pragma unroll
-                for (int i = 0; i < 32; ++i) d[i] = __float_as_uint(act_apply(__uint_as_float(d[i]), a.act));
-                const bool whole = col + 32 <= a.n;
-                if (a.out_f32) {
-                    float *y = (float *)a.y + (size_t)row * a.ldy + col;
-                    if (whole && (a.ldy & 3) == 0) {
+                    for (int i = 0; i < 16; ++i) v[i] = clamped_glu(__uint_as_float(d[2 * i]), __uint_as_float(d[2 * i + 1]), a.b.limit);
+                    if (col + 32 <= a.n) {
+#pragma unroll
+                        for (int i = 0; i < 4; ++i) st4(y + 4 * i, make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]));
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) if (col + 2 * i < a.n) y[i] = f2bf(v[i]);
+                    }
+                    continue;
+                }
+                if (BLOCK) {
+                    if (col < a.b.silu) {
+#pragma unroll
+                        for (int i = 0; i < 32; ++i) if (col + i < a.b.silu) d[i] = __float_as_uint(act_apply(__uint_as_float(d[i]), FKL_ACT_SILU));
+                    }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) d[i] = __float_as_uint(act_apply(__uint_as_float(d[i]), a.act) * a.scale);
+                }
+                const bool whole = col + 32 <= a.n, exact = BLOCK && col >= a.b.plain;
+                if (a.out_f32 || exact) {
+                    const int ld = exact ? a.b.exact - a.b.plain : a.ldy;
+                    float *y = exact ? a.b.y2 + (size_t)row * ld + col - a.b.plain : (float *)a.y + (size_t)row * ld + col;
+                    if (whole && (ld & 3) == 0) {
 #pragma unroll
                         for (int i = 0; i < 8; ++i) reinterpret_cast<uint4 *>(y)[i] = make_uint4(d[4 * i], d[4 * i + 1], d[4 * i + 2], d[4 * i + 3]);
                     } else {

@@ -1,5 +1,6 @@
-// Kernels of the layered decoders: a residual stream in fp32, norms before and after every sublayer, (differential)
-// attention with per-head q/k norm and an output gate, mixture-of-experts feed-forward with a shared expert.
+// Kernels of the layered decoders: a residual stream in fp32, norms before and after every sublayer or one layer norm in front
+// of a parallel block, (differential, rotary, windowed) attention with normed queries and keys and an output gate, mixture-of-experts
+// feed-forward with a shared expert, clamped gated feed-forward.
 //
 // Two families.  The *row* kernels work on M consecutive positions (prompt portions); activations between the matrix
 // products are T = bf16 or float, everything a norm, a router, a softmax or the residual touches is fp32.  The *decode*
@@ -7,41 +8,16 @@
 // activations cost nothing.  Weights are bf16 rows [n, k] with k padded by zeros to a multiple of 64, so no product has a
 // ragged K; activation buffers carry the same zero padding.
 #pragma once
-#include "fk_common.cuh"
-#include <math.h>
-
-#define FKL_MAX_EXPERTS 1024
-#define FKL_MAX_TOP 64
-#define FKL_ERR_TOKEN 0x20000u
-#define FKL_ERR_CAPACITY 0x100000u
-#define FKL_ERR_TC_WAIT 0x200000u
-
-enum { FKL_ACT_NONE = 0, FKL_ACT_RELU2 = 2 };
-
-__device__ __forceinline__ float ldT(const uint16_t *p) { return bf2f(*p); }
-__device__ __forceinline__ float ldT(const float *p) { return *p; }
-__device__ __forceinline__ void stT(uint16_t *p, float v) { *p = f2bf(v); }
-__device__ __forceinline__ void stT(float *p, float v) { *p = v; }
-__device__ __forceinline__ float act_apply(float v, int act) { if (act == FKL_ACT_RELU2) { v = fmaxf(v, 0.0f); v *= v; } return v; }
-__device__ __forceinline__ float inv_rms(float ss, int n, float eps) { return __fdiv_rn(1.0f, __fsqrt_rn(ss / (float)n + eps)); }
-__device__ __forceinline__ float sigmoid_f(float z) { return __fdiv_rn(1.0f, 1.0f + expf(-z)); }
-__device__ __forceinline__ void unpack8f(uint4 v, float (&f)[8]) {
-    f[0] = bf_lo(v.x); f[1] = bf_hi(v.x); f[2] = bf_lo(v.y); f[3] = bf_hi(v.y); f[4] = bf_lo(v.z); f[5] = bf_hi(v.z); f[6] = bf_lo(v.w); f[7] = bf_hi(v.w);
-}
-__device__ __forceinline__ void load8(const uint16_t *p, float (&f)[8]) { unpack8f(__ldcg(reinterpret_cast<const uint4 *>(p)), f); }
-__device__ __forceinline__ void load8(const float *p, float (&f)[8]) {
-    const float4 a = __ldcg(reinterpret_cast<const float4 *>(p)), b = __ldcg(reinterpret_cast<const float4 *>(p) + 1);
-    f[0] = a.x; f[1] = a.y; f[2] = a.z; f[3] = a.w; f[4] = b.x; f[5] = b.y; f[6] = b.z; f[7] = b.w;
-}
+#include "fk_layer_ops.cuh"
 
 // ---------------------------------------------------------------- embedding rows, fp32
-struct EmbedRowsArgs { const uint16_t *table; float *x; const uint32_t *tokens; int d, vocab; };
+struct EmbedRowsArgs { const uint16_t *table; float *x; const uint32_t *tokens; int d, vocab, ld; };
 __global__ void k_embed_rows(FkState *st, EmbedRowsArgs a) {
     pdl_wait(); pdl_launch_dependents();
     const int m = blockIdx.x;
     uint32_t tok = a.tokens ? __ldcg(a.tokens + m) : st->token[m];
     if (tok >= (uint32_t)a.vocab) { if (threadIdx.x == 0) atomicOr(&st->error, FKL_ERR_TOKEN); tok = 0; }
-    const uint16_t *src = a.table + (size_t)tok * a.d; float *dst = a.x + (size_t)m * a.d;
+    const uint16_t *src = a.table + (size_t)tok * a.ld; float *dst = a.x + (size_t)m * a.d;
     for (int i = threadIdx.x; i < a.d; i += blockDim.x) dst[i] = bf2f(src[i]);
 }
 
@@ -53,13 +29,6 @@ struct ResNormArgs {
     const float *x; const void *y; const uint16_t *post_w; const float *add; float *x_out; const uint16_t *norm_w; void *h; const uint32_t *index;
     const void *moe_y; const int *slot; const float *weight; int d, ldh, top, ldy; float eps;
 };
-__device__ __forceinline__ float4 ld4(const uint16_t *p) { const uint2 v = __ldcg(reinterpret_cast<const uint2 *>(p)); return make_float4(bf_lo(v.x), bf_hi(v.x), bf_lo(v.y), bf_hi(v.y)); }
-__device__ __forceinline__ float4 ld4(const float *p) { return __ldcg(reinterpret_cast<const float4 *>(p)); }
-__device__ __forceinline__ void st4(uint16_t *p, float4 v) {
-    const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
-    *reinterpret_cast<uint2 *>(p) = make_uint2(*reinterpret_cast<const uint32_t *>(&a), *reinterpret_cast<const uint32_t *>(&b));
-}
-__device__ __forceinline__ void st4(float *p, float4 v) { *reinterpret_cast<float4 *>(p) = v; }
 // rows of a multiple of 4 and at most NV * 4 * blockDim.x values: everything in registers, one round of loads
 template <typename T, int NV>
 __global__ void __launch_bounds__(256) k_residual_norm_rows4(const FkState *st, ResNormArgs a) {
@@ -148,7 +117,11 @@ __global__ void __launch_bounds__(512) k_residual_norm_rows(const FkState *st, R
 // ---------------------------------------------------------------- matrix product on rows, CUDA cores
 // Y[m, n] = act(sum_k X[m, k] W[row0 + n, k]); with `offsets` the rows of X are grouped by expert (expert e owns rows
 // offsets[e] .. offsets[e + 1] - 1 and the weight rows e * N ..).  fp32 arithmetic: the product of the 32-bit mode.
-struct LinRowsArgs { const float *x; const uint16_t *w; float *y; const int *offsets; int m, n, k, ldx, ldw, ldy, act; };
+// The joint projection of a parallel block stores its columns in three ways: [0, plain) as activations (a silu on the first `silu`),
+// [plain, exact) as fp32, from `exact` on (gate, up) neighbours folded by the clamped gated unit.  All borders are multiples of 32.
+struct BlockCols { float *y2; void *y3; int silu, plain, exact, ld3; float limit; };
+struct LinRowsArgs { const float *x; const uint16_t *w; float *y; const int *offsets; int m, n, k, ldx, ldw, ldy, act; float scale; BlockCols b; };
+template <bool BLOCK>
 __global__ void __launch_bounds__(256) k_linear_rows(const FkState *st, LinRowsArgs a) {
     __shared__ float As[16][68], Bs[16][68];
     pdl_wait(); pdl_launch_dependents();
@@ -183,7 +156,10 @@ __global__ void __launch_bounds__(256) k_linear_rows(const FkState *st, LinRowsA
     for (int i = 0; i < 4; ++i) for (int j = 0; j < 4; ++j) {
         const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
         if (m >= mend || n >= a.n) continue;
-        a.y[(size_t)m * a.ldy + n] = act_apply(acc[i][j], a.act);
+        if (!BLOCK) { a.y[(size_t)m * a.ldy + n] = act_apply(acc[i][j], a.act) * a.scale; continue; }
+        if (n < a.b.plain) a.y[(size_t)m * a.ldy + n] = n < a.b.silu ? act_apply(acc[i][j], FKL_ACT_SILU) : acc[i][j];
+        else if (n < a.b.exact) a.b.y2[(size_t)m * (a.b.exact - a.b.plain) + n - a.b.plain] = acc[i][j];
+        else if (!(j & 1)) ((float *)a.b.y3)[(size_t)m * a.b.ld3 + (n - a.b.exact) / 2] = clamped_glu(acc[i][j], acc[i][j | 1], a.b.limit);
     }
 }
 
@@ -229,6 +205,8 @@ __global__ void __launch_bounds__(128) k_qk_norm_store_rows(FkState *st, QkStore
 struct AttnArgs {
     const float *qkv; const uint16_t *qn, *kn; const void *q; void *ck, *cv, *out; const void *gate; float *part; uint32_t *counter;
     int H, G, maps, dim, vdim, dpad, vpad, cap, ldo, ldg, splits, tiles; float scale, lambda, diff, eps;
+    const float *rot;           // cos / sin of every position's pairs, [capacity][rot_dims], or null
+    int rot_dims, joint, window, keep;          // joint: q (and k) rows are normed all together, a weight for each
 };
 __host__ __device__ inline size_t attn_smem_floats(int dpad, int vpad) {
     return (size_t)FKL_ATT_ROWS * dpad + FKL_ATT_WARPS * 32 * FKL_ATT_ROWS + FKL_ATT_WARPS * FKL_ATT_ROWS * ((size_t)vpad + 2) + FKL_ATT_ROWS * ((size_t)vpad + 2);
@@ -245,14 +223,25 @@ __global__ void __launch_bounds__(FKL_ATT_WARPS * 32) k_attention(FkState *st, A
     const int r0 = tile * RT, nr = min(RT, nrow_kv - r0);
     const uint32_t pos = st->offset + (uint32_t)row;
     if (pos >= (uint32_t)a.cap) { if (tid == 0) atomicOr(&st->error, FKL_ERR_CAPACITY); return; }
-    const int n = (int)pos + 1, per = ((n + a.splits - 1) / a.splits + 31) / 32 * 32;
+    const Visible vis = visible_keys((int)pos, a.window, a.keep);
+    const int n = vis.n, per = ((n + a.splits - 1) / a.splits + 31) / 32 * 32;
     const int k0 = blockIdx.x * per, k1 = min(n, k0 + per);
     T *ck = (T *)a.ck + (size_t)g * a.maps * a.cap * a.dpad, *cv = (T *)a.cv + (size_t)g * a.cap * a.vpad;
     // ---- the query rows (normalised), and in decode the new key and value
     for (int i = tid; i < RT * a.dpad; i += NW * 32) qs[i] = 0.0f;
     __syncthreads();
     if (DECODE) {
-        const bool mine = (int)pos >= k0 && (int)pos < k1;
+        const bool mine = n - 1 >= k0 && n - 1 < k1;
+        __shared__ float red[66];
+        float2 joint = make_float2(0.0f, 0.0f);
+        if (a.joint) {
+            float sq = 0.0f, sk = 0.0f;
+            for (int i = tid; i < a.H * a.dim; i += NW * 32) { const float v = a.qkv[i]; sq = fmaf(v, v, sq); }
+            for (int i = tid; i < a.G * a.dim; i += NW * 32) { const float v = a.qkv[a.H * a.dim + i]; sk = fmaf(v, v, sk); }
+            joint = block_sum2(sq, sk, red);
+            joint = make_float2(inv_rms(joint.x, a.H * a.dim, a.eps), inv_rms(joint.y, a.G * a.dim, a.eps));
+        }
+        const float *rot = a.rot ? a.rot + (size_t)pos * a.rot_dims : nullptr;
         const int items = nr + (mine ? a.maps + 1 : 0);
         for (int it = wid; it < items; it += NW) {
             if (it == nr + a.maps) {
@@ -262,12 +251,16 @@ __global__ void __launch_bounds__(FKL_ATT_WARPS * 32) k_attention(FkState *st, A
             }
             const bool is_q = it < nr;
             const float *src = a.qkv + (is_q ? (g * nrow_kv + r0 + it) : (a.H * a.maps + g * a.maps + (it - nr))) * a.dim;
-            const uint16_t *w = is_q ? a.qn : a.kn;
-            float ss = 0.0f;
-            for (int i = lane; i < a.dim; i += 32) ss = fmaf(src[i], src[i], ss);
-            const float r = inv_rms(warp_sum(ss), a.dim, a.eps);
+            const uint16_t *w = (is_q ? a.qn : a.kn) + (a.joint ? (is_q ? g * nrow_kv + r0 + it : g) * a.dim : 0);
+            float r = is_q ? joint.x : joint.y;
+            if (!a.joint) {
+                float ss = 0.0f;
+                for (int i = lane; i < a.dim; i += 32) ss = fmaf(src[i], src[i], ss);
+                r = inv_rms(warp_sum(ss), a.dim, a.eps);
+            }
             for (int i = lane; i < a.dim; i += 32) {
-                const float v = src[i] * r * bf2f(w[i]);
+                float v = src[i] * r * bf2f(w[i]);
+                if (rot && i < a.rot_dims) v = rotate_dim(v, src[i ^ 1] * r * bf2f(w[i ^ 1]), i, a.rot_dims, rot);
                 if (is_q) qs[it * a.dpad + i] = v; else stT(ck + ((size_t)(it - nr) * a.cap + pos) * a.dpad + i, v);
             }
         }
@@ -288,7 +281,7 @@ __global__ void __launch_bounds__(FKL_ATT_WARPS * 32) k_attention(FkState *st, A
         for (int p0 = 0; p0 < nk; p0 += kpp) {
             const int kk = p0 + kin; const bool kv = kk < nk;
             for (int m = 0; m < a.maps; ++m) {
-                const T *krow = ck + ((size_t)m * a.cap + kb + (kv ? kk : 0)) * a.dpad;
+                const T *krow = ck + ((size_t)m * a.cap + vis.key(kb + (kv ? kk : 0))) * a.dpad;
                 float dot[RT] = {};
                 for (int d = sub * 8; d < a.dpad; d += lpk * 8) {
                     float kf[8]; load8(krow + d, kf);
@@ -320,7 +313,7 @@ __global__ void __launch_bounds__(FKL_ATT_WARPS * 32) k_attention(FkState *st, A
         __syncwarp();
         for (int k = 0; k < nk; ++k) {
             float v[VPL];
-            const T *vrow = cv + (size_t)(kb + k) * a.vpad;
+            const T *vrow = cv + (size_t)vis.key(kb + k) * a.vpad;
 #pragma unroll
             for (int i = 0; i < VPL; ++i) { const int d = lane * VPL + i; v[i] = d < a.vpad ? ldT(vrow + d) : 0.0f; }
 #pragma unroll
@@ -423,9 +416,6 @@ __host__ __device__ inline AdLayout ad_layout(int maps, int dpad, int vpad) {
     l.total = l.of + FKL_ATT_ROWS * vpad * 4;
     return l;
 }
-__device__ __forceinline__ void cp16_zfill(uint32_t dst, const void *src, bool valid) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(valid ? 16 : 0) : "memory");
-}
 __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st, AttnArgs a) {
     extern __shared__ __align__(128) unsigned char ad_smem[];
     constexpr int RT = FKL_ATT_ROWS, KC = FKL_AD_KEYS, NT = FKL_AD_THREADS;
@@ -433,11 +423,13 @@ __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st
     float *qs = reinterpret_cast<float *>(ad_smem + L.q), *sc = reinterpret_cast<float *>(ad_smem + L.sc), *pr = reinterpret_cast<float *>(ad_smem + L.pr);
     uint16_t *nk = reinterpret_cast<uint16_t *>(ad_smem + L.nk), *nv = reinterpret_cast<uint16_t *>(ad_smem + L.nv);
     float *of = reinterpret_cast<float *>(ad_smem + L.of);
-    __shared__ float s_corr[RT], s_m[RT], s_l[RT], s_fac[256 * RT]; __shared__ int s_last;
+    __shared__ float s_corr[RT], s_m[RT], s_l[RT], s_fac[256 * RT], s_red[66]; __shared__ int s_last;
     const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
     const int g = blockIdx.y / a.tiles, tile = blockIdx.y - g * a.tiles, group = a.H / a.G, nrow_kv = group * a.maps, r0 = tile * RT, nr = min(RT, nrow_kv - r0);
     const uint32_t upos = st->offset;                   // advanced by the head of the token before, long since finished
-    const int pos = (int)upos, n = pos + 1, per = ((n + a.splits - 1) / a.splits + KC - 1) / KC * KC, active = (n + per - 1) / per;
+    const int pos = (int)upos;
+    const Visible vis = visible_keys(pos, a.window, a.keep);
+    const int n = vis.n, newest = n - 1, per = ((n + a.splits - 1) / a.splits + KC - 1) / KC * KC, active = (n + per - 1) / per;
     const int k0 = blockIdx.x * per, k1 = min(n, k0 + per), nchunk = k1 > k0 ? (k1 - k0 + KC - 1) / KC : 0;
     const bool fits = upos < (uint32_t)a.cap;
     uint16_t *ck = (uint16_t *)a.ck + (size_t)g * a.maps * a.cap * a.dpad, *cv = (uint16_t *)a.cv + (size_t)g * a.cap * a.vpad;
@@ -446,12 +438,12 @@ __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st
         const uint32_t kb = sbase + (uint32_t)((c & 1) * L.stage), vb = kb + (uint32_t)(a.maps * KC * L.ks * 2);
         const int kn = a.dpad / 8, vn = a.vpad / 8, key0 = k0 + c * KC;
         for (int i = tid; i < a.maps * KC * kn; i += NT) {
-            const int r = i / kn, cc = (i - r * kn) * 8, key = key0 + (r & (KC - 1)); const bool v = key < pos;
-            if (key != pos) cp16_zfill(kb + (uint32_t)((r * L.ks + cc) * 2), v ? ck + ((size_t)(r / KC) * a.cap + key) * a.dpad + cc : ck, v);
+            const int r = i / kn, cc = (i - r * kn) * 8, key = key0 + (r & (KC - 1)); const bool v = key < newest;
+            if (key != newest) cp16_zfill(kb + (uint32_t)((r * L.ks + cc) * 2), v ? ck + ((size_t)(r / KC) * a.cap + vis.key(key)) * a.dpad + cc : ck, v);
         }
         for (int i = tid; i < KC * vn; i += NT) {
-            const int r = i / vn, cc = (i - r * vn) * 8, key = key0 + r; const bool v = key < pos;
-            if (key != pos) cp16_zfill(vb + (uint32_t)((r * L.vs + cc) * 2), v ? cv + (size_t)key * a.vpad + cc : cv, v);
+            const int r = i / vn, cc = (i - r * vn) * 8, key = key0 + r; const bool v = key < newest;
+            if (key != newest) cp16_zfill(vb + (uint32_t)((r * L.vs + cc) * 2), v ? cv + (size_t)vis.key(key) * a.vpad + cc : cv, v);
         }
     };
     if (fits) for (int c = 0; c < 2; ++c) { if (c < nchunk) request(c); asm volatile("cp.async.commit_group;" ::: "memory"); }
@@ -459,7 +451,16 @@ __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st
     if (!fits) { if (tid == 0) atomicOr(&st->error, FKL_ERR_CAPACITY); return; }
     if (nchunk == 0) return;                            // more splits than this many keys need
     // ---- query rows, and where the position falls here the new key and value
-    const bool mine = pos >= k0 && pos < k1;
+    const bool mine = newest >= k0 && newest < k1;
+    float2 joint = make_float2(0.0f, 0.0f);
+    if (a.joint) {
+        float sq = 0.0f, sk = 0.0f;
+        for (int i = tid; i < a.H * a.dim; i += NT) { const float v = __ldcg(a.qkv + i); sq = fmaf(v, v, sq); }
+        for (int i = tid; i < a.G * a.dim; i += NT) { const float v = __ldcg(a.qkv + a.H * a.dim + i); sk = fmaf(v, v, sk); }
+        joint = block_sum2(sq, sk, s_red);
+        joint = make_float2(inv_rms(joint.x, a.H * a.dim, a.eps), inv_rms(joint.y, a.G * a.dim, a.eps));
+    }
+    const float *rot = a.rot ? a.rot + (size_t)pos * a.rot_dims : nullptr;
     for (int it = wid; it < RT + (mine ? a.maps + 1 : 0); it += NT / 32) {
         if (it >= nr && it < RT) { for (int i = lane; i < a.dpad; i += 32) qs[it * a.dpad + i] = 0.0f; continue; }
         if (it == RT + a.maps) {
@@ -469,7 +470,7 @@ __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st
         }
         const bool is_q = it < RT;
         const float *src = a.qkv + (is_q ? (g * nrow_kv + r0 + it) : (a.H * a.maps + g * a.maps + (it - RT))) * a.dim;
-        const uint16_t *w = is_q ? a.qn : a.kn;
+        const uint16_t *w = (is_q ? a.qn : a.kn) + (a.joint ? (is_q ? g * nrow_kv + r0 + it : g) * a.dim : 0);
         float ss = 0.0f, xv[4], wv[4];                  // the first 128 values stay in registers
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
@@ -479,11 +480,13 @@ __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st
 #pragma unroll
         for (int j = 0; j < 4; ++j) ss = fmaf(xv[j], xv[j], ss);
         for (int i = lane + 128; i < a.dim; i += 32) { const float v = __ldcg(src + i); ss = fmaf(v, v, ss); }
-        const float r = inv_rms(warp_sum(ss), a.dim, a.eps);
+        const float r = a.joint ? (is_q ? joint.x : joint.y) : inv_rms(warp_sum(ss), a.dim, a.eps);
 #pragma unroll 4
-        for (int j = 0; j * 32 + lane < a.dpad; ++j) {
+        for (int j = 0; j * 32 < a.dpad; ++j) {
             const int i = lane + j * 32;
-            const float v = j < 4 ? xv[j & 3] * r * wv[j & 3] : i < a.dim ? __ldcg(src + i) * r * bf2f(w[i]) : 0.0f;
+            float v = j < 4 ? xv[j & 3] * r * wv[j & 3] : i < a.dim ? __ldcg(src + i) * r * bf2f(w[i]) : 0.0f;
+            if (rot) v = rotate_dim(v, __shfl_xor_sync(0xffffffffu, v, 1), i, a.rot_dims, rot);
+            if (i >= a.dpad) continue;
             if (is_q) qs[it * a.dpad + i] = v * a.scale;
             else { nk[(it - RT) * a.dpad + i] = f2bf(v); if (i < a.dim) ck[((size_t)(it - RT) * a.cap + pos) * a.dpad + i] = f2bf(v); }
         }
@@ -501,10 +504,10 @@ __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st
         const unsigned char *kb = ad_smem + (c & 1) * L.stage; unsigned char *kbw = ad_smem + (c & 1) * L.stage;
         const uint16_t *ks = reinterpret_cast<const uint16_t *>(kb), *vs = ks + a.maps * KC * L.ks;
         const int key0 = k0 + c * KC;
-        if (mine && pos >= key0 && pos < key0 + KC) {
+        if (mine && newest >= key0 && newest < key0 + KC) {
             uint16_t *kw = reinterpret_cast<uint16_t *>(kbw), *vw = kw + a.maps * KC * L.ks;
-            for (int i = tid; i < a.maps * a.dpad; i += NT) { const int mm = i / a.dpad; kw[(mm * KC + pos - key0) * L.ks + i - mm * a.dpad] = nk[i]; }
-            for (int i = tid; i < a.vpad; i += NT) vw[(pos - key0) * L.vs + i] = nv[i];
+            for (int i = tid; i < a.maps * a.dpad; i += NT) { const int mm = i / a.dpad; kw[(mm * KC + newest - key0) * L.ks + i - mm * a.dpad] = nk[i]; }
+            for (int i = tid; i < a.vpad; i += NT) vw[(newest - key0) * L.vs + i] = nv[i];
             __syncthreads();
         }
         {   // scores: key tid % 64, rows tid / 64 and 4 more (of the same map)
@@ -721,19 +724,25 @@ __global__ void __launch_bounds__(256) k_moe_gather(const FkState *st, RouteArgs
 // order the lanes read them without bank conflicts.  With few rows, 2 .. 16 warps of a block share a row group and split K.
 // A chunk is described by (base of row 0, row stride, weights in it), which also expresses the concatenated K ranges of a
 // mixture's down projection.  The first batch is fetched before the dependency wait where the rows do not depend on it.
+// SEGMENTS: up to three products W_s x_s of n rows each in one launch (outputs one after the other), each with a K range of its own;
+// one of the inputs may be a mixer's raw output that is RMS-normed in groups, scaled and gated while it is staged.
 #define FKL_GV_R 2
 #define FKL_GV_U 4
 #define FKL_GV_WARPS 16
-enum { FKL_GV_LINEAR = 0, FKL_GV_MOE_UP = 1, FKL_GV_MOE_DOWN = 2 };
+enum { FKL_GV_LINEAR = 0, FKL_GV_MOE_UP = 1, FKL_GV_MOE_DOWN = 2, FKL_GV_SEGMENTS = 3 };
 struct GvChunk { const uint16_t *base; int stride, len; };
 struct GemvArgs {
-    // input vector: x, or with norm_w set: x' = x + norm(pend) * post_w (+ add) -> x_out, then norm(x') * norm_w (-> h_out)
+    // input vector: x, or with norm_w set: x' = x + pscale * sum_p norm(pend_p) * post_w_p + the rest of the pending vectors as they are
+    // (+ add) -> x_out, then norm(x') * norm_w (-> h_out); with norm_b a layer norm.  npend vectors of k values, the first nnorm normed.
     const float *x, *pend; const uint16_t *post_w; const float *add; float *x_out; const uint16_t *norm_w; float *h_out;
     const uint16_t *w; float *y; int k, ldk, n, act, act_row0; float eps;
     unsigned long long *amax; uint32_t *counter, *history;             // greedy choice over y (the last block advances the state)
     // mixture of experts
     const float *logits; int *sel; float *wts; const float *sact; const uint16_t *w2; int E, top, ff, ldff, ffs, ldffs;
     int kslices, nchunks;
+    const uint16_t *norm_b; int npend, nnorm, act_end, pair0; float pscale, limit, oscale;      // rows from pair0 on: (gate, up) neighbours -> one value
+    const float *sx[3]; const uint16_t *sw[3]; int sk[3], sld[3], sc[4], nseg, gseg, group;     // SEGMENTS; sc: first chunk; gseg: the normed input or -1
+    const uint16_t *gw; const float *gate;
 };
 __host__ __device__ inline int gv_chunks(int ldk) { return (ldk + 255) / 256; }
 __host__ __device__ inline size_t gv_smem_bytes(int nchunks) { return (size_t)nchunks * (256 * 4 + sizeof(GvChunk)); }
@@ -748,15 +757,20 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
     extern __shared__ __align__(16) unsigned char gv_smem[];
     constexpr int R = FKL_GV_R, U = FKL_GV_U, NT = FKL_GV_WARPS * 32;
     float *xs = reinterpret_cast<float *>(gv_smem); GvChunk *tab = reinterpret_cast<GvChunk *>(gv_smem + (size_t)a.nchunks * 1024);
-    __shared__ float red[40], part[2][FKL_GV_WARPS][R], tval[FKL_MAX_TOP]; __shared__ int tsel[FKL_MAX_TOP];
+    __shared__ float red[66], part[2][FKL_GV_WARPS][R], tval[FKL_MAX_TOP]; __shared__ int tsel[FKL_MAX_TOP];
     __shared__ unsigned long long wbest[FKL_GV_WARPS]; __shared__ int is_last;
-    __shared__ float slog[MODE == FKL_GV_MOE_UP ? FKL_MAX_EXPERTS : 1];
+    __shared__ float slog[MODE == FKL_GV_MOE_UP ? FKL_MAX_EXPERTS : MODE == FKL_GV_SEGMENTS ? FKL_GV_MAX_GROUPS : 1];
     const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, KS = a.kslices, spb = FKL_GV_WARPS / KS, ksl = wid % KS, slot = wid / KS;
-    const int c0 = a.nchunks * ksl / KS, c1 = a.nchunks * (ksl + 1) / KS, nb = (c1 - c0 + U - 1) / U;
-    const int groups = (a.n + R - 1) / R, gstride = gridDim.x * spb;
+    int c0 = a.nchunks * ksl / KS, c1 = a.nchunks * (ksl + 1) / KS, nb = (c1 - c0 + U - 1) / U;       // of the group being fetched
+    const int sgroups = (a.n + R - 1) / R, groups = MODE == FKL_GV_SEGMENTS ? sgroups * a.nseg : sgroups, gstride = gridDim.x * spb;
     int g = blockIdx.x * spb + slot;
     size_t roff[R];                                    // rows of the current fetch group: index into the chunk's rows
     auto set_rows = [&](int gg) {
+        if (MODE == FKL_GV_SEGMENTS) {
+            const int s = gg / sgroups, nc = a.sc[s + 1] - a.sc[s];
+            gg -= s * sgroups;
+            c0 = a.sc[s] + nc * ksl / KS; c1 = a.sc[s] + nc * (ksl + 1) / KS; nb = (c1 - c0 + U - 1) / U;
+        }
 #pragma unroll
         for (int r = 0; r < R; ++r) {
             int row = gg * R + r; row = row < a.n ? row : a.n - 1;
@@ -780,12 +794,18 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
     };
     for (int i = tid; i < a.nchunks * 256; i += NT) xs[i] = 0.0f;
     if (MODE != FKL_GV_MOE_DOWN) {
-        for (int c = tid; c < a.nchunks; c += NT) tab[c] = GvChunk{a.w + c * 256, a.ldk, min(256, a.ldk - c * 256)};
+        if (MODE == FKL_GV_SEGMENTS) {
+            for (int s = 0; s < a.nseg; ++s) for (int c = a.sc[s] + tid; c < a.sc[s + 1]; c += NT) {
+                const int o = (c - a.sc[s]) * 256;
+                tab[c] = GvChunk{a.sw[s] + o, a.sld[s], min(256, a.sld[s] - o)};
+            }
+        } else for (int c = tid; c < a.nchunks; c += NT) tab[c] = GvChunk{a.w + c * 256, a.ldk, min(256, a.ldk - c * 256)};
         __syncthreads();
-        if (MODE == FKL_GV_LINEAR && g < groups && nb > 0) { set_rows(g); fetch(buf0, c0); }
+        if ((MODE == FKL_GV_LINEAR || MODE == FKL_GV_SEGMENTS) && g < groups && nb > 0) { set_rows(g); fetch(buf0, c0); }
     }
     uint2 pw[NV > 0 ? NV : 1], nw[NV > 0 ? NV : 1];
-    if (NV > 0 && a.norm_w) {
+    const bool block = a.norm_b || a.npend > 1 || a.nnorm < a.npend;       // several pending vectors, or a layer norm
+    if (NV > 0 && a.norm_w && !block) {
 #pragma unroll
         for (int v = 0; v < NV; ++v) {
             const int i = (v * NT + tid) * 4;
@@ -823,6 +843,86 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
         }
         __syncthreads();
         if (g < groups && nb > 0) { set_rows(g); fetch(buf0, c0); }
+    } else if (MODE == FKL_GV_SEGMENTS) {
+        for (int s = 0; s < a.nseg; ++s) {
+            const float *x = a.sx[s]; const int k = a.sk[s], o = a.sc[s] * 256;
+            if (s != a.gseg) {
+                if ((k & 3) == 0 && ((uintptr_t)x & 15) == 0) {
+                    for (int i = tid * 4; i < k; i += NT * 4) *reinterpret_cast<float4 *>(xs + gv_place(o + i)) = __ldcg(reinterpret_cast<const float4 *>(x + i));
+                } else for (int i = tid; i < k; i += NT) xs[gv_place(o + i)] = __ldcg(x + i);
+                continue;
+            }
+            const int ng = k / a.group;
+            if (ng == 1) {
+                float ss = 0.0f;
+                for (int i = tid; i < k; i += NT) { const float v = __ldcg(x + i); ss = fmaf(v, v, ss); }
+                ss = block_sum(ss, red);
+                if (tid == 0) slog[0] = inv_rms(ss, k, a.eps);
+            } else for (int q = wid; q < ng; q += FKL_GV_WARPS) {
+                float ss = 0.0f;
+                for (int i = lane; i < a.group; i += 32) { const float v = __ldcg(x + q * a.group + i); ss = fmaf(v, v, ss); }
+                ss = warp_sum(ss);
+                if (lane == 0) slog[q] = inv_rms(ss, a.group, a.eps);
+            }
+            __syncthreads();
+            for (int i = tid; i < k; i += NT) xs[gv_place(o + i)] = __ldcg(x + i) * slog[i / a.group] * bf2f(a.gw[i]) * sigmoid_f(__ldcg(a.gate + i));
+        }
+        __syncthreads();
+    } else if (NV > 0 && a.norm_w && block) {
+        // everything this needs is requested at once; two normed pending vectors share a reduction
+        float4 x[NV > 0 ? NV : 1], y[3][NV > 0 ? NV : 1];
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const int i = (v * NT + tid) * 4;
+            x[v] = i < a.k ? __ldcg(reinterpret_cast<const float4 *>(a.x + i)) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+            for (int p = 0; p < 3; ++p) y[p][v] = p < a.npend && i < a.k ? __ldcg(reinterpret_cast<const float4 *>(a.pend + (size_t)p * a.k + i)) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        }
+        float f[3] = {1.0f, 1.0f, 1.0f};
+        if (a.nnorm > 0) {
+            float ss[3] = {};
+#pragma unroll
+            for (int p = 0; p < 3; ++p)
+#pragma unroll
+                for (int v = 0; v < NV; ++v) ss[p] = fmaf(y[p][v].x, y[p][v].x, fmaf(y[p][v].y, y[p][v].y, fmaf(y[p][v].z, y[p][v].z, fmaf(y[p][v].w, y[p][v].w, ss[p]))));
+            const float2 s01 = block_sum2(ss[0], ss[1], red);
+            f[0] = a.pscale * inv_rms(s01.x, a.k, a.eps);
+            if (a.nnorm > 1) f[1] = a.pscale * inv_rms(s01.y, a.k, a.eps);
+            if (a.nnorm > 2) f[2] = a.pscale * inv_rms(block_sum(ss[2], red), a.k, a.eps);
+        }
+        float sum = 0.0f;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const int i = (v * NT + tid) * 4;
+#pragma unroll
+            for (int p = 0; p < 3; ++p) if (p < a.npend && i < a.k) {
+                float4 w = make_float4(1.0f, 1.0f, 1.0f, 1.0f);
+                if (p < a.nnorm) { const uint2 q = __ldg(reinterpret_cast<const uint2 *>(a.post_w + (size_t)p * a.k + i)); w = make_float4(bf_lo(q.x), bf_hi(q.x), bf_lo(q.y), bf_hi(q.y)); }
+                x[v].x = fmaf(y[p][v].x * f[p], w.x, x[v].x); x[v].y = fmaf(y[p][v].y * f[p], w.y, x[v].y);
+                x[v].z = fmaf(y[p][v].z * f[p], w.z, x[v].z); x[v].w = fmaf(y[p][v].w * f[p], w.w, x[v].w);
+            }
+            sum += (x[v].x + x[v].y) + (x[v].z + x[v].w);
+        }
+        const float mean = a.norm_b ? block_sum(sum, red) / (float)a.k : 0.0f;
+        float ss = 0.0f;
+#pragma unroll
+        for (int v = 0; v < NV; ++v) if ((v * NT + tid) * 4 < a.k) {
+            const float d0 = x[v].x - mean, d1 = x[v].y - mean, d2 = x[v].z - mean, d3 = x[v].w - mean;
+            ss = fmaf(d0, d0, fmaf(d1, d1, fmaf(d2, d2, fmaf(d3, d3, ss))));
+        }
+        const float r = inv_rms(block_sum(ss, red), a.k, a.eps);
+#pragma unroll
+        for (int v = 0; v < NV; ++v) {
+            const int i = (v * NT + tid) * 4;
+            if (i >= a.k) continue;
+            if (a.x_out && blockIdx.x == 0) *reinterpret_cast<float4 *>(a.x_out + i) = x[v];
+            const uint2 w = __ldg(reinterpret_cast<const uint2 *>(a.norm_w + i)), b = a.norm_b ? __ldg(reinterpret_cast<const uint2 *>(a.norm_b + i)) : make_uint2(0, 0);
+            const float4 h = make_float4(fmaf((x[v].x - mean) * r, bf_lo(w.x), bf_lo(b.x)), fmaf((x[v].y - mean) * r, bf_hi(w.x), bf_hi(b.x)),
+                                         fmaf((x[v].z - mean) * r, bf_lo(w.y), bf_lo(b.y)), fmaf((x[v].w - mean) * r, bf_hi(w.y), bf_hi(b.y)));
+            *reinterpret_cast<float4 *>(xs + gv_place(i)) = h;
+            if (a.h_out && blockIdx.x == 0) *reinterpret_cast<float4 *>(a.h_out + i) = h;
+        }
+        __syncthreads();
     } else if (NV > 0 && a.norm_w) {
         float4 x[NV > 0 ? NV : 1], y[NV > 0 ? NV : 1];
 #pragma unroll
@@ -862,23 +962,27 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
         __syncthreads();
     } else if (a.norm_w) {
         __syncthreads();
-        float ry = 0.0f;
-        if (a.pend) {
+        float ry[3] = {1.0f, 1.0f, 1.0f};
+        for (int p = 0; p < a.nnorm; ++p) {
             float ss = 0.0f;
-            for (int i = tid; i < a.k; i += NT) { const float v = __ldcg(a.pend + i); ss = fmaf(v, v, ss); }
-            ry = inv_rms(block_sum(ss, red), a.k, a.eps);
+            for (int i = tid; i < a.k; i += NT) { const float v = __ldcg(a.pend + (size_t)p * a.k + i); ss = fmaf(v, v, ss); }
+            ry[p] = a.pscale * inv_rms(block_sum(ss, red), a.k, a.eps);
         }
-        float ss = 0.0f;
+        float ss = 0.0f, sum = 0.0f, mean = 0.0f;
         for (int i = tid; i < a.k; i += NT) {
             float v = __ldcg(a.x + i);
-            if (a.pend) v = fmaf(__ldcg(a.pend + i) * ry, bf2f(a.post_w[i]), v);
+            for (int p = 0; p < a.npend; ++p) v = fmaf(__ldcg(a.pend + (size_t)p * a.k + i) * ry[p], p < a.nnorm ? bf2f(a.post_w[(size_t)p * a.k + i]) : 1.0f, v);
             if (a.add) v += __ldcg(a.add + i);
-            xs[gv_place(i)] = v; ss = fmaf(v, v, ss);
+            xs[gv_place(i)] = v; ss = fmaf(v, v, ss); sum += v;
             if (a.x_out && blockIdx.x == 0) a.x_out[i] = v;
+        }
+        if (a.norm_b) {
+            mean = block_sum(sum, red) / (float)a.k; ss = 0.0f;
+            for (int i = tid; i < a.k; i += NT) { const float v = xs[gv_place(i)] - mean; ss = fmaf(v, v, ss); }
         }
         const float r = inv_rms(block_sum(ss, red), a.k, a.eps);
         for (int i = tid; i < a.k; i += NT) {
-            const float v = xs[gv_place(i)] * r * bf2f(a.norm_w[i]);
+            const float v = fmaf((xs[gv_place(i)] - mean) * r, bf2f(a.norm_w[i]), a.norm_b ? bf2f(a.norm_b[i]) : 0.0f);
             xs[gv_place(i)] = v;
             if (a.h_out && blockIdx.x == 0) a.h_out[i] = v;
         }
@@ -891,17 +995,17 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
     // ---- rows
     unsigned long long best = 0ull;
     float acc[R] = {};
-    int bi = 0, parity = 0;
+    int bi = 0, parity = 0, mc0 = c0, mc1 = c1, mnb = nb;          // the group being multiplied
     // one batch: request the next one (of this row group or the following) into the other buffer, multiply this one; after a
     // group's last batch, fold the lanes (and the warps that share the group, behind a barrier of their own) and store
     auto step = [&](uint4 (&cur)[U][R], uint4 (&next)[U][R]) {
-        const bool last = bi + 1 == nb;
-        if (!last) fetch(next, c0 + (bi + 1) * U);
+        const bool last = bi + 1 == mnb;
+        if (!last) fetch(next, mc0 + (bi + 1) * U);
         else if (g + gstride < groups) { set_rows(g + gstride); fetch(next, c0); }
 #pragma unroll
         for (int u = 0; u < U; ++u) {
-            const int c = c0 + bi * U + u;
-            if (c < c1) {
+            const int c = mc0 + bi * U + u;
+            if (c < mc1) {
                 const float4 x0 = *reinterpret_cast<const float4 *>(xs + c * 256 + lane * 4), x1 = *reinterpret_cast<const float4 *>(xs + c * 256 + 128 + lane * 4);
 #pragma unroll
                 for (int r = 0; r < R; ++r) {
@@ -920,12 +1024,21 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
             if (ksl == 0) for (int r = 0; r < R; ++r) for (int q = 1; q < KS; ++q) acc[r] += part[parity][wid + q][r];
             parity ^= 1;                               // the next group writes the other half while this one is still being read
         }
-        if (ksl == 0) {
+        if (ksl == 0 && MODE == FKL_GV_LINEAR && g * R >= a.pair0) {
+            if (lane == 0) a.y[a.pair0 + (g * R - a.pair0) / 2] = clamped_glu(acc[0], acc[1], a.limit);
+        } else if (ksl == 0 && MODE == FKL_GV_SEGMENTS) {
+            const int s = g / sgroups;
+#pragma unroll
+            for (int r = 0; r < R; ++r) {
+                const int row = (g - s * sgroups) * R + r;
+                if (row < a.n && lane == 0) a.y[(size_t)s * a.n + row] = acc[r];
+            }
+        } else if (ksl == 0) {
 #pragma unroll
             for (int r = 0; r < R; ++r) {
                 const int row = g * R + r;
                 if (row < a.n) {
-                    const float v = row >= a.act_row0 ? act_apply(acc[r], a.act) : acc[r];
+                    const float v = (row >= a.act_row0 && row < a.act_end ? act_apply(acc[r], a.act) : acc[r]) * (MODE == FKL_GV_LINEAR ? a.oscale : 1.0f);
                     if (lane == 0) a.y[row] = v;
                     if (a.amax) {
                         const uint32_t u = __float_as_uint(v), key = (u & 0x80000000u) ? ~u : u | 0x80000000u;
@@ -937,7 +1050,7 @@ __global__ void __launch_bounds__(FKL_GV_WARPS * 32, 1) k_gemv(FkState *st, Gemv
         }
 #pragma unroll
         for (int r = 0; r < R; ++r) acc[r] = 0.0f;
-        bi = 0; g += gstride;
+        bi = 0; g += gstride; mc0 = c0; mc1 = c1; mnb = nb;
     };
     while (g < groups) {
         step(buf0, buf1);

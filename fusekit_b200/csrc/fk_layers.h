@@ -1,5 +1,5 @@
-// Boundary between the host runtime (fk_runtime.cu) and the kernels of the layered decoders (fk_layers.cu), which are a
-// translation unit of their own so that both compile side by side.
+// Boundary between the host runtime (fk_runtime.cu) and the kernels of the layered decoders (fk_layers.cu; fk_blocks.cu for those of the
+// parallel blocks), which are translation units of their own so that all compile side by side.
 #pragma once
 #include "../../include/fusekit_cuda.h"
 #include "fk_common.cuh"
@@ -13,3 +13,5 @@ struct FklEnv {
 bool fkl_owns(int kind);                                           // whether a task kind is handled here
 fk_status fkl_run(FklEnv &env, const fk_task &t, char *err, size_t cap);
 cudaError_t fkl_init();                                            // shared-memory limits of the kernels, once per context
+fk_status fkb_run(FklEnv &env, const fk_task &t, char *err, size_t cap);      // the kinds of fk_blocks.cu
+cudaError_t fkb_init();

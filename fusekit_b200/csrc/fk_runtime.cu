@@ -206,7 +206,9 @@ static const char *kKernelNames[FK_TASK_KIND_COUNT] = {
     "fusekit_argmax_finalize", "fusekit_allreduce", "fusekit_residual_add", "fusekit_rmsnorm_rows", "fusekit_rope_store_rows",
     "fusekit_argmax_rows", "fusekit_kv_store_quant", "fusekit_sdpa_decode_quant", "fusekit_embed_rows", "fusekit_residual_norm_rows",
     "fusekit_linear_rows", "fusekit_qk_norm_store_rows", "fusekit_attention_rows", "fusekit_moe_route_rows", "fusekit_norm_linear",
-    "fusekit_attention_decode", "fusekit_moe_up", "fusekit_moe_down", "fusekit_argmax_row"};
+    "fusekit_attention_decode", "fusekit_moe_up", "fusekit_moe_down", "fusekit_argmax_row", "fusekit_block_norm_rows",
+    "fusekit_block_linear_rows", "fusekit_rotary_store_rows", "fusekit_window_attention_rows", "fusekit_window_attention_decode", "fusekit_recurrence_rows",
+    "fusekit_recurrence_decode", "fusekit_norm_gate_rows", "fusekit_segment_linear"};
 extern "C" fk_status fk_kernel_names(char *buf, size_t cap) {
     if (!buf || cap == 0) return fail(FK_ERR_VALUE, "buf is null");
     std::string s;

@@ -12,17 +12,19 @@ from __future__ import annotations
 
 import math
 
-from .model_spec import ModelSpec
+from .model_spec import ModelSpec, ParallelMixerSpec, block_layout, round_up
 
 VERSION = 2
 KINDS = ["step_init", "embed_lookup_decode", "rmsnorm_qkv", "qk_norm_rope_store", "sdpa_decode", "linear_residual",
          "rmsnorm_gateup_act", "final_rmsnorm_lm_head", "argmax_finalize", "allreduce", "residual_add", "rmsnorm_rows",
          "rope_store_rows", "argmax_rows", "kv_store_quant", "sdpa_decode_quant", "embed_rows", "residual_norm_rows", "linear_rows",
-         "qk_norm_store_rows", "attention_rows", "moe_route_rows", "norm_linear", "attention_decode", "moe_up", "moe_down", "argmax_row"]
+         "qk_norm_store_rows", "attention_rows", "moe_route_rows", "norm_linear", "attention_decode", "moe_up", "moe_down", "argmax_row",
+         "block_norm_rows", "block_linear_rows", "rotary_store_rows", "window_attention_rows", "window_attention_decode", "recurrence_rows",
+         "recurrence_decode", "norm_gate_rows", "segment_linear"]
 KERNEL = {k: "fusekit_" + k for k in KINDS}
 (K_STEP, K_EMBED, K_QKV, K_QKNORM, K_SDPA, K_LIN, K_GATEUP, K_HEAD, K_ARGMAX, K_ALLREDUCE, K_RESADD, K_NORMROWS, K_ROPEROWS,
  K_ARGMAXROWS, K_KVQ, K_SDPAQ, K_EMBEDROWS, K_RESNORM, K_LINROWS, K_QKSTORE, K_ATTROWS, K_ROUTE, K_NORMLIN, K_ATTDEC, K_MOEUP,
- K_MOEDOWN, K_ARGMAXROW) = range(27)
+ K_MOEDOWN, K_ARGMAXROW, K_BLOCKNORM, K_BLOCKLIN, K_ROTSTORE, K_WINROWS, K_WINDEC, K_RECROWS, K_RECDEC, K_NORMGATE, K_SEGLIN) = range(36)
 
 
 def _bf16_round(v: float) -> float:
@@ -207,10 +209,6 @@ def _envelope(tasks: list, out_slots: dict, target: dict) -> dict:
 
 
 # ------------------------------------------------------------------ layered decoders (model_spec.LayeredSpec)
-def round_up(v: int, m: int) -> int:
-    return (v + m - 1) // m * m
-
-
 def _task(tasks, kind, layer, bufs, iargs, fargs=()):
     tasks.append({"kind": kind, "layer": layer, "bufs": {int(k): v for k, v in bufs.items() if v}, "iargs": [int(v) for v in iargs],
                   "fargs": [float(v) for v in fargs]})
@@ -220,13 +218,15 @@ def key_splits(mixer, capacity: int, sm: int) -> int:
     """Blocks the keys of a decode step are split over: two blocks per SM over all kv heads, at most 64 (the last
     block to finish folds the others' results) and at least 64 keys of capacity each."""
     tiles = -(-(mixer.heads // mixer.kv_heads * mixer.maps) // 8)
-    return max(1, min(-(-2 * sm // (mixer.kv_heads * tiles)), -(-capacity // 64), 64))
+    return max(1, min(-(-2 * sm // (mixer.kv_heads * tiles)), -(-mixer.visible(capacity) // 64), 64))
 
 
 def layered_decode_tasks(spec, capacity: int, lambdas: dict, dtype: int = 0, sm: int = 148) -> list:
     """One decoded position: per layer run q|k|v|gate projection (previous sublayer's post-norm, residual add and this one's
     pre-norm in its prologue), attention with the q/k norm and the cache store in its prologue, output projection, router and
     shared up-projection in one product, the chosen experts' up- and down-projections; then the head with the greedy choice."""
+    if spec.block == "parallel":
+        return parallel_decode_tasks(spec, capacity, dtype, sm)
     D, eps, t = spec.hidden, spec.eps, []
     x = lambda r: f"global_scratch.x_in.{r}"
     _task(t, K_EMBEDROWS, -1, {0: "param.embed_tokens", 1: x(0)}, [D, 1, spec.vocab])
@@ -262,6 +262,8 @@ def layered_decode_tasks(spec, capacity: int, lambdas: dict, dtype: int = 0, sm:
 def layered_rows_tasks(spec, capacity: int, lambdas: dict, rows: int, wanted: int, greedy: bool, dtype: int = 0) -> list:
     """``rows`` consecutive positions: the same layers on row kernels; logits of the ``wanted`` rows of the index buffer, and with
     ``greedy`` the token after the first of them (the position then advances by ``rows``)."""
+    if spec.block == "parallel":
+        return parallel_rows_tasks(spec, capacity, rows, wanted, greedy, dtype)
     D, V, M, eps, t = spec.hidden, spec.vocab, rows, spec.eps, []
     ld = round_up(D, 64)
     emb, xb, h = "rows_scratch.embedding", "rows_scratch.x", "rows_scratch.h"
@@ -310,9 +312,140 @@ def layered_rows_tasks(spec, capacity: int, lambdas: dict, rows: int, wanted: in
     return t
 
 
+def _pair(a: int, b: int) -> int:
+    return a | b << 16
+
+
+def _limit(layer) -> float:
+    return layer.mlp.limit if layer.mlp is not None else 0.0
+
+
+def _recurrence(layer):
+    """The recurrent mixer of a parallel block's layer, the tensors' prefix, the factor on its queries and its gate cap."""
+    m = layer.mixer
+    if isinstance(m, ParallelMixerSpec):
+        return m.right, "mix.right.", 1.0, 0.0
+    return m, "mix.", m.dim ** -0.5, m.gate_cap
+
+
+def _recurrence_bufs(lp: str, pre: str, buf: str, run: int, memory: bool, logits: str, out: str) -> dict:
+    bufs = {0: buf + "q", 1: buf + "k", 2: buf + "v", 6: f"layer_state.{run}", 7: out}
+    return {**bufs, **({3: logits, 4: lp + pre + "bias"} if memory else {5: lp + pre + "log_decay"})}
+
+
+def parallel_decode_tasks(spec, capacity: int, dtype: int = 0, sm: int = 148) -> list:
+    """One decoded position of a model of parallel blocks, three or four kernels a layer: the joint projection of everything that
+    reads the normed input (the layer before is added up and normed in its prologue, silu and gated unit at its end), attention with
+    joint q/k norm, rotation and cache store in its prologue, the recurrence, and the output projections of mixer and feed-forward in
+    one launch (the recurrence's norm and gate in its prologue)."""
+    D, eps, t = spec.hidden, spec.eps, []
+    x = lambda r: f"global_scratch.x_in.{r}"
+    _task(t, K_EMBEDROWS, -1, {1: x(0), 3: "param.lm_head"}, [D, 1, spec.vocab])
+    cur, pend, post, np_, nn = x(0), None, None, 0, 0
+    for run, (i, _) in enumerate(spec.runs()):
+        l, lp = spec.layers[i], f"layer_param.{i}."
+        m, f, lay, buf = l.mixer, l.mlp, block_layout(l), f"layer_scratch.block.{i}."
+        _task(t, K_NORMLIN, run, {0: cur, 1: pend, 2: post, 4: x(run) if run else None, 5: lp + "norm1", 6: lp + "block", 7: "layer_scratch.block", 11: lp + "norm1.b"},
+              [D, lay.rows, 3 if lay.silu else 0, 0, np_, nn, lay.exact if f is not None else 0, lay.silu], [eps, 0.5, _limit(l)])
+        cur = x(run)
+        rec, pre, qs, cap = _recurrence(l)
+        both, seg = isinstance(m, ParallelMixerSpec), []
+        if both:
+            a = m.left
+            _task(t, K_WINDEC, run, {0: buf + "attention", 1: lp + "mix.left.q.norm", 2: lp + "mix.left.k.norm", 3: f"layer_cache_k.{run}", 4: f"layer_cache_v.{run}",
+                                     5: "layer_scratch.attention", 6: "global_scratch.attention_partials", 7: "global_scratch.attention_counters",
+                                     8: f"rotation.{i}" if a.rotary is not None else None},
+                  [_pair(a.heads, a.kv_heads), _pair(a.dim, a.vdim), capacity, dtype, key_splits(a, capacity, sm), a.window or 0, a.keep_first, a.rotary.dims if a.rotary else 0],
+                  [a.scale, eps])
+            seg.append(("layer_scratch.attention", lp + "mix.left.o", a.out_rows))
+        _task(t, K_RECDEC, run, _recurrence_bufs(lp, pre, buf, run, not both, buf + "logits", "layer_scratch.memory"), [rec.heads, rec.dim, rec.vdim], [qs, cap])
+        seg.append(("layer_scratch.memory", lp + pre + "o", rec.out_rows))
+        normed = len(seg) - 1
+        if f is not None:
+            seg.append((buf + "ff", lp + "mlp.down", f.ff))
+        bufs = {6: "layer_scratch.sums", 7: lp + pre + "norm", 8: buf + "gate"}
+        for j, (src, w, _) in enumerate(seg):
+            bufs[2 * j], bufs[2 * j + 1] = src, w
+        ks = [k for _, _, k in seg] + [0] * (3 - len(seg))
+        _task(t, K_SEGLIN, run, bufs, [D, len(seg), *ks, normed, rec.norm_group], [eps])
+        pend, post, np_, nn = "layer_scratch.sums", lp + "mix.out" if both else None, len(seg), 2 if both else 0
+    _task(t, K_NORMLIN, -1, {0: cur, 1: pend, 2: post, 4: x(len(spec.runs())), 5: "param.final_norm", 6: "param.lm_head", 7: "global_scratch.logits",
+                             9: "global_scratch.argmax_scratch", 10: "global_scratch.head_counter", 11: "param.final_norm.b"},
+          [D, spec.vocab, 0, 0, np_, nn, 0, 0], [eps, 0.5, 0.0, spec.logit_scale])
+    return t
+
+
+def parallel_rows_tasks(spec, capacity: int, rows: int, wanted: int, greedy: bool, dtype: int = 0) -> list:
+    """``rows`` consecutive positions of a model of parallel blocks (see layered_rows_tasks)."""
+    D, V, M, eps, t = spec.hidden, spec.vocab, rows, spec.eps, []
+    ld = round_up(D, 64)
+    emb, xb, h, r = "rows_scratch.embedding", "rows_scratch.x", "rows_scratch.h", "rows_scratch."
+    _task(t, K_EMBEDROWS, -1, {1: emb, 2: "rows_scratch.tokens", 3: "param.lm_head"}, [D, M, V])
+    cur, pend, post, nn = emb, [], None, 0
+
+    def norm(run, w, n, out, x_out=None, index=None):
+        _task(t, K_BLOCKNORM, run, {0: cur, **{1 + j: y for j, y in enumerate(pend)}, 4: x_out, 5: w, 6: out, 7: index, 8: w + ".b", 9: post},
+              [D, n, dtype, ld, ld, len(pend), nn], [eps, 0.5])
+
+    def linear(run, x, w, y, n, ldx, ldy, f32=0, m=M, scale=0.0):
+        _task(t, K_LINROWS, run, {0: x, 1: w, 2: y}, [m, 0, n, ldx, ldy, dtype, f32 << 8, 0], [scale])
+
+    for run, (i, _) in enumerate(spec.runs()):
+        l, lp = spec.layers[i], f"layer_param.{i}."
+        m, f, lay, buf = l.mixer, l.mlp, block_layout(l), f"rows_scratch.block.{i}."
+        norm(run, lp + "norm1", M, h, xb if run else None)
+        cur = xb if run else emb
+        ldb, ldf, both = round_up(lay.plain, 64), round_up(f.ff, 64) if f is not None else 64, isinstance(m, ParallelMixerSpec)
+        _task(t, K_BLOCKLIN, run, {0: h, 1: lp + "block", 2: r + "block", 3: r + "gate_logits" if lay.exact > lay.plain else None, 4: r + "ff" if f is not None else None},
+              [M, lay.plain, lay.exact, lay.rows, ldb, ldf, dtype, lay.silu], [_limit(l)])
+        pend, post, nn = [], None, 0
+        if both:
+            a = m.left
+            ha, da, lda = _pair(a.heads, a.kv_heads), _pair(a.dim, a.vdim), round_up(a.out_rows, 64)
+            _task(t, K_ROTSTORE, run, {0: buf + "attention", 1: lp + "mix.left.q.norm", 2: lp + "mix.left.k.norm", 3: r + "q", 4: f"layer_cache_k.{run}", 5: f"layer_cache_v.{run}",
+                                       6: f"rotation.{i}" if a.rotary is not None else None}, [ha, da, capacity, M, ldb, a.rotary.dims if a.rotary else 0, dtype], [eps])
+            _task(t, K_WINROWS, run, {0: r + "q", 1: f"layer_cache_k.{run}", 2: f"layer_cache_v.{run}", 3: r + "attention"},
+                  [ha, da, capacity, M, dtype, a.window or 0, a.keep_first], [a.scale])
+            linear(run, r + "attention", lp + "mix.left.o", r + "y", D, lda, ld)
+            pend, post, nn = [r + "y", r + "y1"], lp + "mix.out", 2
+        else:
+            pend = [r + "y"]
+        rec, pre, qs, cap = _recurrence(l)
+        ldm, ldg = round_up(rec.out_rows, 8), round_up(rec.out_rows, 64)
+        _task(t, K_RECROWS, run, {**_recurrence_bufs(lp, pre, buf, run, not both, r + "gate_logits", r + "memory"), 8: r + "runs"},
+              [_pair(rec.heads, dtype), rec.dim, rec.vdim, M, ldb, lay.exact - lay.plain, ldm, recurrence_scratch(rec, M)], [qs, cap])
+        _task(t, K_NORMGATE, run, {0: r + "memory", 1: lp + pre + "norm", 2: buf + "gate", 3: r + "gated"}, [rec.out_rows, rec.norm_group, M, ldm, ldb, ldg, dtype], [eps])
+        linear(run, r + "gated", lp + pre + "o", pend[-1], D, ldg, ld)
+        if f is not None:
+            pend.append(r + "y2")
+            linear(run, r + "ff", lp + "mlp.down", pend[-1], D, ldf, ld)
+    if wanted:
+        norm(-1, "param.final_norm", wanted, "rows_scratch.h_wanted", None, "rows_scratch.index")
+        linear(-1, "rows_scratch.h_wanted", "param.lm_head", "rows_scratch.logits", V, ld, V, f32=1, m=wanted, scale=spec.logit_scale)
+        if greedy:
+            _task(t, K_ARGMAXROW, -1, {0: "rows_scratch.logits"}, [V, M])
+    return t
+
+
+def recurrence_cell(rec) -> int:
+    """Floats of a recurrence's state per (head, slice of 64 value columns)."""
+    return rec.dim * 64 + (round_up(rec.dim + 1, 4) if hasattr(rec, "gate_cap") else 0)
+
+
+def recurrence_state(rec) -> int:
+    return rec.heads * -(-rec.vdim // 64) * recurrence_cell(rec)
+
+
+def recurrence_scratch(rec, rows: int) -> int:
+    """Floats of scratch that let a prompt's chunks be worked on in several runs side by side (at most 16 of at least 4 chunks)."""
+    runs = min(16, -(-rows // 64) // 4)
+    return 0 if runs < 2 else (runs + 1) * recurrence_state(rec) + runs * rec.heads * -(-rec.vdim // 64)
+
+
 def emit_layered(spec, capacity: int, lambdas: dict, dtype: int = 0, sm: int = 148) -> dict:
     """The decode step of a layered decoder as a v2 document (``lambdas``: layer -> combination constant of its two maps)."""
-    out_slots = {K_EMBEDROWS: [1], K_NORMLIN: [4, 7, 8, 9, 10], K_ATTDEC: [3, 4, 5, 6, 7], K_MOEUP: [3, 4, 5], K_MOEDOWN: [6]}
+    out_slots = {K_EMBEDROWS: [1], K_NORMLIN: [4, 7, 8, 9, 10], K_ATTDEC: [3, 4, 5, 6, 7], K_MOEUP: [3, 4, 5], K_MOEDOWN: [6],
+                 K_WINDEC: [3, 4, 5, 6, 7], K_RECDEC: [6, 7], K_SEGLIN: [6]}
     return _envelope(layered_decode_tasks(spec, capacity, lambdas, dtype, sm), out_slots,
                      {"chip": "b200", "arch": "sm_100a", "tensor_parallel": 1, "rank": 0, "bits": 32 if dtype else 16,
                       "launch": "grid and block sizes are chosen by the runtime from the SM count"})

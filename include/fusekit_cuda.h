@@ -67,13 +67,23 @@ enum {
     FK_TASK_MOE_UP = 24,
     FK_TASK_MOE_DOWN = 25,
     FK_TASK_ARGMAX_ROW = 26,
-    FK_TASK_KIND_COUNT = 27
+    /* parallel blocks of the layered decoders (no reference counterpart): layer norm, rotary windowed attention, linear recurrences */
+    FK_TASK_BLOCK_NORM_ROWS = 27,
+    FK_TASK_BLOCK_LINEAR_ROWS = 28,
+    FK_TASK_ROTARY_STORE_ROWS = 29,
+    FK_TASK_WINDOW_ATTENTION_ROWS = 30,
+    FK_TASK_WINDOW_ATTENTION_DECODE = 31,
+    FK_TASK_RECURRENCE_ROWS = 32,
+    FK_TASK_RECURRENCE_DECODE = 33,
+    FK_TASK_NORM_GATE_ROWS = 34,
+    FK_TASK_SEGMENT_LINEAR = 35,
+    FK_TASK_KIND_COUNT = 36
 };
 
 /* activation selector for FK_TASK_RMSNORM_GATEUP_ACT */
 enum { FK_ACT_SWIGLU = 0, FK_ACT_GEGLU_TANH = 1 };
-/* activation selector of the layered decoders' products: none, square of relu */
-enum { FK_ACT_NONE = 0, FK_ACT_RELU_SQUARED = 2 };
+/* activation selector of the layered decoders' products: none, square of relu, silu */
+enum { FK_ACT_NONE = 0, FK_ACT_RELU_SQUARED = 2, FK_ACT_SILU = 3 };
 
 /*
  * One entry of the per-token dispatch list (reference: the (kernel, buffers,
@@ -153,13 +163,15 @@ enum { FK_ACT_NONE = 0, FK_ACT_RELU_SQUARED = 2 };
  * Layered decoders.  A = bf16 or (dtype = 1) fp32 activations; weights are dense rows kept as uploaded (fk_weight_keep_rows), K
  * padded with zeros to a multiple of 64; `maps` = 2 for differential attention (two sub-heads per head), else 1; dpad / vpad =
  * dim / vdim rounded up to 8.  ROWS tasks work on M consecutive positions offset .. offset + M - 1 of one sequence.
- * EMBED_ROWS           buf0 table T[V,D]  buf1 x f32[M,D]  buf2 token ids u32[M] | 0 (the decode state's)   i0 D  i1 M  i2 V
+ * EMBED_ROWS           buf0 table T[V,D]  buf1 x f32[M,D]  buf2 token ids u32[M] | 0 (the decode state's)  buf3 weight|0 (its rows are the
+ *                      table, buf0 0)   i0 D  i1 M  i2 V
  * RESIDUAL_NORM_ROWS   x' = x + norm(y) * post (+ add), h = norm(x') * w.  buf0 x f32[M,D]  buf1 y A[M,ldy]|0  buf2 post T[D]
  *                      buf3 add f32[M,D]|0  buf4 x' out|0 (may be buf0)  buf5 w T[D]  buf6 h A[M,ldh]  buf7 row index u32|0 (output
  *                      row r is input row index[r])  buf8 grouped expert rows A[M*top,ldy]|0  buf9 slots  buf10 expert weights
  *                      (y += sum_j weight[j] * buf8[slot[j]])   i0 D  i1 output rows  i2 dtype  i3 ldh  i4 top  i5 ldy   f0 eps
  * LINEAR_ROWS          buf0 x A[M,ldx]  buf1 weight  buf2 y [M,ldy]  buf3 expert offsets i32[E+1]|0 (rows grouped by expert, weight
- *                      rows e*N ..)   i0 M  i1 first weight row  i2 N  i3 ldx  i4 ldy  i5 dtype  i6 act | 256 (y is fp32)  i7 E
+ *                      rows e*N ..)   i0 M  i1 first weight row  i2 N  i3 ldx  i4 ldy  i5 dtype  i6 act | 256 (y is fp32)  i7 E   f0 factor on y
+ *                      (0 = 1)
  * QK_NORM_STORE_ROWS   buf0 q|k|v rows A[M,ld]  buf1 q norm T[dim]  buf2 k norm  buf3 q out A[M,H*maps,dpad]  buf4 cache k
  *                      A[G*maps,capacity,dpad]  buf5 cache v A[G,capacity,vpad]   i0 H  i1 G  i2 dim  i3 vdim  i4 capacity  i5 M
  *                      i6 dtype | maps << 8  i7 ld   f0 eps
@@ -171,7 +183,10 @@ enum { FK_ACT_NONE = 0, FK_ACT_RELU_SQUARED = 2 };
  * NORM_LINEAR          one row, fp32 activations: y = act(W h), h = norm(x') * w with x' as in RESIDUAL_NORM_ROWS, or h = x when buf5 = 0.
  *                      buf0 x f32[K]  buf1 pending y f32|0  buf2 post  buf3 add|0  buf4 x' out|0 (not buf0)  buf5 w|0  buf6 weight
  *                      buf7 y f32[N]  buf8 h out f32|0  buf9 argmax scratch u64[2*SMs]|0  buf10 counter   i0 K  i1 N  i2 act  i3 first row with
- *                      act   f0 eps      (with buf9 the last block picks the greedy token of y and advances the decode state)
+ *                      act   f0 eps   Several pending sublayer outputs: i4 their number (1..3), buf1 f32[i4][K], the first i5 of them normed with
+ *                      buf2[j] and scaled by f1, the others added as they are.  buf11 bias T[K]: h is a layer norm.  i6 > 0: from row i6 (even)
+ *                      on rows are (gate, up) neighbours, y[i6 + j] the clamped gated value of pair j with limit f2.  i7 > 0: end of the
+ *                      rows with act.  f3 factor on y (0 = 1)      (with buf9 the last block picks the greedy token of y and advances the decode state)
  * ATTENTION_DECODE     one position: q/k norm, cache store, attention.  buf0 q|k|v|gate f32  buf1 q norm  buf2 k norm  buf3 cache k
  *                      buf4 cache v  buf5 out f32[H*vdim]  buf6 partials f32  buf7 counters (zero before first use)   i0 H  i1 G  i2 dim
  *                      i3 vdim  i4 capacity  i5 gate present  i6 dtype | maps << 8 (dtype of the caches)  i7 key splits
@@ -181,6 +196,34 @@ enum { FK_ACT_NONE = 0, FK_ACT_RELU_SQUARED = 2 };
  * MOE_DOWN             buf0 act f32[top*ff]  buf1 chosen  buf2 weights  buf3 weight [E*D, ff]  buf4 shared act f32|0  buf5 shared weight [D, ffs]
  *                      buf6 y f32[D]   i0 D  i1 E  i2 top  i3 ff  i4 ffs
  * ARGMAX_ROW           buf0 logits f32[V]   i0 V  i1 positions to advance by
+ * Parallel blocks.  A recurrence state is [heads][ceil(vdim / 64)] cells of dim * 64 floats (S by rows of 64 value columns), for the
+ * matrix memory followed by round4(dim + 1) more (normaliser, running maximum); it is not read at position 0.
+ * BLOCK_NORM_ROWS      x' = x + f1 * sum of the normed y_p * post_p + the other y_p, h = norm(x').  buf0 x f32[M,D]  buf1, buf2, buf3 y_p A[M,ldy]|0
+ *                      buf4 x' out|0 (may be buf0)  buf5 w T[D]  buf6 h A[rows,ldh]  buf7 row index u32|0  buf8 bias T[D]|0 (with it a layer
+ *                      norm, else an RMS norm)  buf9 post T[normed][D]   i0 D  i1 output rows  i2 dtype  i3 ldh  i4 ldy  i5 pending  i6 normed
+ *                      f0 eps  f1 factor
+ * BLOCK_LINEAR_ROWS    the joint projection, x A[M, weight columns]: columns [0, i1) go to buf2 A[M,ldy] (the first i7 behind a silu), [i1, i2) to
+ *                      buf3 f32[M, i2 - i1], from i2 on (gate, up) neighbours are folded into buf4 A[M,ld3] with limit f0.  buf0 x  buf1 weight
+ *                      i0 M  i1  i2 (multiples of 32)  i3 columns  i4 ldy  i5 ld3  i6 dtype  i7 columns with silu
+ * ROTARY_STORE_ROWS    buf0 q|k|v rows A[M,ld]  buf1 q norm T[H*dim]  buf2 k norm T[G*dim] (all rows normed together)  buf3 q out A[M,H,dpad]  buf4
+ *                      cache k  buf5 cache v  buf6 rotation table f32[capacity][i5 / 2][cos, sin]|0   i0 H | G << 16  i1 dim | vdim << 16
+ *                      i2 capacity  i3 M  i4 ld  i5 rotated dimensions  i6 dtype   f0 eps
+ * WINDOW_ATTENTION_ROWS  buf0 q  buf1 cache k  buf2 cache v  buf3 out A[M, round64(H*vdim)]   i0, i1, i2, i3 as above  i4 dtype  i5 window (0: none;
+ *                      position i sees j <= i with i - j < window or j < keep)  i6 keep   f0 scale
+ * WINDOW_ATTENTION_DECODE  one position: joint q/k norm, rotation, cache store, attention.  buf0 q|k|v f32  buf1 q norm  buf2 k norm  buf3 cache k
+ *                      buf4 cache v  buf5 out f32[H*vdim]  buf6 partials  buf7 counters (as ATTENTION_DECODE)  buf8 rotation table|0
+ *                      i0 H | G << 16  i1 dim | vdim << 16  i2 capacity  i3 dtype of the caches  i4 key splits  i5 window  i6 keep
+ *                      i7 rotated dimensions   f0 scale  f1 eps
+ * RECURRENCE_ROWS      buf0 q A[M,ld] (heads one after the other)  buf1 k  buf2 v  buf3 gate logits f32[M,i5] (input gates, then forget gates)|0  buf4 their
+ *                      biases T[2*heads]|0  buf5 log decays f32[heads]|0  buf6 state  buf7 out A[M,i6]  buf8 scratch|0 (i7 floats of it)
+ *                      i0 heads | dtype << 16  i1 dim  i2 vdim  i3 M  i4 ld  i5 ld of the logits  i6 ld of out  i7 scratch floats
+ *                      f0 factor on q  f1 gate cap.  With buf5 the decay form, with buf3 and buf4 the matrix memory
+ * RECURRENCE_DECODE    one position, the same with f32 vectors (buf0 .. buf7; strides and scratch are not used)
+ * NORM_GATE_ROWS       out = norm(o) * w * sigmoid(gate), the norm over groups of i1 values.  buf0 o A[M,ldo]  buf1 w T[n]  buf2 gate A[M,ldg]
+ *                      buf3 out A[M,ld]   i0 n  i1 group  i2 M  i3 ldo  i4 ldg  i5 ld  i6 dtype   f0 eps
+ * SEGMENT_LINEAR       one row, up to three products y_s = W_s x_s of i0 rows: buf(2s) x_s f32, buf(2s + 1) weight  buf6 y f32[i1][i0]  buf7 w T, buf8
+ *                      gate f32: input i5 is staged as norm(x) * w * sigmoid(gate), the norm over groups of i6 (i5 = -1: none)
+ *                      i0 rows  i1 products  i2..i4 values of x_s   f0 eps
  *
  * Batch decode (M = 2..16 independent sequences at one position): EMBED with i1 = M, LINEAR_RESIDUAL / RMSNORM_GATEUP_ACT
  * with their row counts, SDPA_DECODE with i5 = M (q and out T[M, n_q*hd], caches [M, n_kv, capacity, hd]).

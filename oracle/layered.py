@@ -131,3 +131,169 @@ class LayeredOracle:
             self.residuals.append(x)
         self.pos += len(tokens)
         return rms_norm(x, t["final.norm"], eps) @ t["head"].T
+
+
+# ---------------------------------------------------------------- parallel blocks: layer norm, rotation, windows, recurrences
+def layer_norm(x, w, b, eps):
+    """Mean and variance along the last axis; eps inside the root."""
+    d = x - np.mean(x, axis=-1, keepdims=True)
+    return d / np.sqrt(np.mean(d * d, axis=-1, keepdims=True) + eps) * w + b
+
+
+def silu(z):
+    return z * sigmoid(z)
+
+
+def clamped_glu(gate, up, limit):
+    """s(g) (u + 1) with s(g) = g sigmoid(1.702 g), the gate bounded from above and the up value on both sides."""
+    g, u = np.minimum(gate, limit), np.clip(up, -limit, limit)
+    return g * sigmoid(1.702 * g) * (u + 1.0)
+
+
+def rotation_frequencies(dims, base, scaling=None):
+    """Angle per position of every rotated pair; ``scaling`` = (factor, low, high, original) stretches the long wavelengths."""
+    out = []
+    for i in range(dims // 2):
+        f = float(base) ** (-2.0 * i / dims)
+        if scaling is not None:
+            factor, low, high, original = scaling
+            wave = 2.0 * np.pi / f
+            if wave > original / low:
+                f = f / factor
+            elif wave >= original / high:
+                s = (original / wave - low) / (high - low)
+                f = (1.0 - s) * f / factor + s * f
+        out.append(f)
+    return np.array(out)
+
+
+def rotate_pairs(x, positions, freqs):
+    """x [T, heads, d]: neighbours (2i, 2i + 1) turned by position * freqs[i]; dimensions past the last pair are kept."""
+    out = x.copy()
+    for i, f in enumerate(freqs):
+        a = np.asarray(positions, np.float64) * f
+        c, s = np.cos(a)[:, None].astype(x.dtype), np.sin(a)[:, None].astype(x.dtype)
+        u, v = x[..., 2 * i], x[..., 2 * i + 1]
+        out[..., 2 * i], out[..., 2 * i + 1] = u * c - v * s, v * c + u * s
+    return out
+
+
+def window_attention(q, k, v, scale, pos0, window=None, keep_first=0):
+    """One head, as softmax_attention, where position i sees j <= i with i - j < window or j < keep_first."""
+    out = np.zeros((q.shape[0], v.shape[1]), q.dtype)
+    for i in range(q.shape[0]):
+        p = pos0 + i
+        j = np.arange(p + 1)
+        see = j[(p - j < window) | (j < keep_first)] if window is not None else j
+        s = (k[see] @ q[i]) * scale
+        e = np.exp(s - s.max())
+        out[i] = (e / e.sum()) @ v[see]
+    return out
+
+
+def decay_recurrence(q, k, v, decay, state):
+    """One head: S <- decay S + k v^T, o = S^T q.  ``state``: S [dim, vdim].  Returns (o, S)."""
+    out = np.zeros((q.shape[0], v.shape[1]), q.dtype)
+    for t in range(q.shape[0]):
+        state = decay * state + np.outer(k[t], v[t])
+        out[t] = state.T @ q[t]
+    return out, state
+
+
+def matrix_memory(q, k, v, log_i, log_f, state):
+    """One head of a matrix memory with exponential gates kept in range by a running maximum.  ``state``: (S, n, m)."""
+    S, n, m = state
+    out = np.zeros((q.shape[0], v.shape[1]), q.dtype)
+    for t in range(q.shape[0]):
+        new = max(log_f[t] + m, log_i[t])
+        keep, add = np.exp(log_f[t] + m - new), np.exp(log_i[t] - new)
+        S, n, m = keep * S + add * np.outer(k[t], v[t]), keep * n + add * k[t], new
+        out[t] = (S.T @ q[t]) / (max(abs(n @ q[t]), np.exp(-m)) + 1e-6)
+    return out, (S, n, m)
+
+
+def soft_cap(z, cap):
+    return cap * np.tanh(z / cap)
+
+
+def log_sigmoid(z):
+    return -np.logaddexp(0.0, -z)
+
+
+class ParallelBlockOracle:
+    """Layers in which the mixer and the feed-forward read one layer norm and are added together.  Same interface as
+    LayeredOracle; only the numbers of ``spec`` are read, and a mixer is told by the fields it has."""
+
+    def __init__(self, spec, tensors, dtype=np.float64):
+        self.spec, self.dt = spec, dtype
+        self.t = {k: np.asarray(v, dtype) for k, v in tensors.items()}
+        self.reset()
+
+    def reset(self):
+        self.pos, self.mem = 0, {}
+
+    def attention(self, key, p, m, h):
+        t, eps, T = self.t, self.spec.eps, h.shape[0]
+        H, G, d, dv = m.heads, m.kv_heads, m.dim, m.vdim
+        q = rms_norm(h @ t[p + "q"].T, t[p + "q.norm"], eps).reshape(T, H, d)
+        k = rms_norm(h @ t[p + "k"].T, t[p + "k.norm"], eps).reshape(T, G, d)
+        v = (h @ t[p + "v"].T).reshape(T, G, dv)
+        if m.rotary is not None:
+            r = m.rotary
+            s = None if r.scaling is None else (r.scaling.factor, r.scaling.low, r.scaling.high, r.scaling.original)
+            f = rotation_frequencies(r.dims, r.base, s)
+            at = self.pos + np.arange(T)
+            q, k = rotate_pairs(q, at, f), rotate_pairs(k, at, f)
+        if key in self.mem:
+            k, v = np.concatenate([self.mem[key][0], k]), np.concatenate([self.mem[key][1], v])
+        self.mem[key] = (k, v)
+        o = [window_attention(q[:, i], k[:, i // (H // G)], v[:, i // (H // G)], m.scale, self.pos, m.window, m.keep_first) for i in range(H)]
+        return np.concatenate(o, 1) @ t[p + "o"].T
+
+    def lightning(self, key, p, m, h):
+        t, T = self.t, h.shape[0]
+        q, k, v = (silu(h @ t[p + n].T).reshape(T, m.heads, -1) for n in "qkv")
+        S, o = self.mem.get(key, np.zeros((m.heads, m.dim, m.vdim), self.dt)).copy(), []
+        for i in range(m.heads):
+            y, S[i] = decay_recurrence(q[:, i], k[:, i], v[:, i], m.decay[i], S[i])
+            o.append(y)
+        self.mem[key] = S
+        o = rms_norm(np.concatenate(o, 1), t[p + "norm"], self.spec.eps) * sigmoid(h @ t[p + "g"].T)
+        return o @ t[p + "o"].T
+
+    def mlstm(self, key, p, m, h):
+        t, T, eps = self.t, h.shape[0], self.spec.eps
+        q = (h @ t[p + "q"].T).reshape(T, m.heads, m.dim) * m.dim ** -0.5
+        k, v = (h @ t[p + "k"].T).reshape(T, m.heads, m.dim), (h @ t[p + "v"].T).reshape(T, m.heads, m.vdim)
+        gi = soft_cap(h @ t[p + "i"].T + t[p + "i.b"], m.gate_cap)
+        gf = log_sigmoid(soft_cap(h @ t[p + "f"].T + t[p + "f.b"], m.gate_cap))
+        st = self.mem.get(key) or [(np.zeros((m.dim, m.vdim), self.dt), np.zeros(m.dim, self.dt), 0.0) for _ in range(m.heads)]
+        o, new = [], []
+        for i in range(m.heads):
+            y, s = matrix_memory(q[:, i], k[:, i], v[:, i], gi[:, i], gf[:, i], st[i])
+            o.append(rms(y, eps)); new.append(s)
+        self.mem[key] = new
+        return (np.concatenate(o, 1) * t[p + "norm"] * sigmoid(h @ t[p + "g"].T)) @ t[p + "o"].T
+
+    def mixer(self, i, m, h):
+        p = f"l{i}.mix."
+        if hasattr(m, "left"):
+            a = self.attention((i, "left"), p + "left.", m.left, h)
+            b = self.lightning((i, "right"), p + "right.", m.right, h)
+            return 0.5 * (rms_norm(a, self.t[p + "left.out"], self.spec.eps) + rms_norm(b, self.t[p + "right.out"], self.spec.eps))
+        return self.mlstm(i, p, m, h)
+
+    def feed_forward(self, i, f, h):
+        p = f"l{i}.mlp."
+        return clamped_glu(h @ self.t[p + "gate"].T, h @ self.t[p + "up"].T, f.limit) @ self.t[p + "down"].T
+
+    def forward(self, tokens):
+        t, eps = self.t, self.spec.eps
+        x, self.residuals = t["embed"][np.asarray(tokens, np.int64)].copy(), []
+        for i, l in enumerate(self.spec.layers):
+            h = layer_norm(x, t[f"l{i}.norm1"], t[f"l{i}.norm1.b"], eps)
+            y = self.mixer(i, l.mixer, h)
+            x = x + (y if l.mlp is None else y + self.feed_forward(i, l.mlp, h))
+            self.residuals.append(x)
+        self.pos += len(tokens)
+        return layer_norm(x, t["final.norm"], t["final.norm.b"], eps) @ t["embed"].T * self.spec.logit_scale

@@ -4,7 +4,7 @@ from __future__ import annotations
 import numpy as np
 
 from fusekit_b200 import checkpoint as CK
-from fusekit_b200.layered import LayeredEngine, vector_plan, weight_plan
+from fusekit_b200.layered import LayeredEngine, tensor_shapes
 from fusekit_b200.model_spec import AttentionSpec, LayeredSpec, LayerSpec, LoopSpec, MoeSpec
 from oracle.layered import LayeredOracle
 
@@ -24,20 +24,6 @@ def rounded(a):
 
 def spec(layers, hidden=96, vocab=211, loop=None, eps=1e-5, name="test"):
     return LayeredSpec(name, "Fatulix", hidden, vocab, tuple(layers), eps=eps, loop=loop)
-
-
-def tensor_shapes(s):
-    out = {}
-    for _, parts, k in weight_plan(s):
-        for n, rows in parts:
-            out[n] = (rows, k)
-    for _, n, shape, _, _ in vector_plan(s):
-        out[n] = shape
-    for i, l in enumerate(s.layers):
-        if l.mixer.diff is not None:
-            for n in ("lq1", "lk1", "lq2", "lk2"):
-                out[f"l{i}.mix.{n}"] = (l.mixer.dim,)
-    return out
 
 
 def random_tensors(s, seed=0, router=6.0):
