@@ -154,7 +154,7 @@ __global__ void __launch_bounds__(256) k_norm_gate_rows(const FkState *st, NormG
 }
 
 // ---------------------------------------------------------------- linear recurrences, position by position
-// S_t = keep_t S_(t-1) + add_t k_t v_t^T, o_t = S_t^T (qscale q_t).  Decay form (log_decay set): keep = exp(log_decay[head]), add = 1.  Matrix
+// S_t = keep_t S_(t-1) + add_t k_t v_t^T, o_t = S_t^T (qscale q_t).  Decay form (log_decay set: the heads' logarithms, then the decays themselves): keep = decay, add = 1.  Matrix
 // memory (MEM): log gates i = cap tanh((zi + bi) / cap), f = log sigmoid(cap tanh((zf + bf) / cap)), m_t = max(f + m_(t-1), i),
 // keep = exp(f + m_(t-1) - m_t), add = exp(i - m_t), n_t like S with k alone, and o_t over max(|n_t . q_t|, exp(-m_t)) + 1e-6.
 // One block per (slice of 64 value columns, head); a thread holds RPT rows of one column in registers through all positions.
@@ -183,7 +183,7 @@ __global__ void __launch_bounds__(FKL_RC_THREADS) k_recurrence(FkState *st, RecA
     for (int j = 0; j < RPT; ++j) { const int d = part * RPT + j; s[j] = !fresh && d < a.dim ? __ldcg(S + d * FKL_RC_COLS + c) : 0.0f; }
     const bool own_n = MEM && c < RPT && part * RPT + c < a.dim;         // this thread keeps row part * RPT + c of the normaliser
     if (MEM && !fresh) { if (own_n) n = __ldcg(S + a.dim * FKL_RC_COLS + part * RPT + c); m = __ldcg(S + a.dim * FKL_RC_COLS + a.dim); }
-    const float bi = MEM ? bf2f(a.bias[head]) : 0.0f, bf = MEM ? bf2f(a.bias[a.heads + head]) : 0.0f, decay = MEM ? 0.0f : expf(a.log_decay[head]);
+    const float bi = MEM ? bf2f(a.bias[head]) : 0.0f, bf = MEM ? bf2f(a.bias[a.heads + head]) : 0.0f, decay = MEM ? 0.0f : a.log_decay[a.heads + head];
     pdl_wait(); pdl_launch_dependents();
     const T *q = (const T *)a.q + head * a.dim, *k = (const T *)a.k + head * a.dim, *v = (const T *)a.v + head * a.vdim;
     float rq = 0.0f, rk = 0.0f, rv = 0.0f, ri = 0.0f, rf = 0.0f;

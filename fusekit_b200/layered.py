@@ -226,8 +226,9 @@ class LayeredEngine(EngineBase):
                     tables[rot] = rt.to_device(rotation_table(rot, self.capacity)) if rot.dims else 0
                 self.scratch[f"rotation.{i}"] = tables[rot]
             if isinstance(l.mixer, ParallelMixerSpec):
+                d = np.array(l.mixer.right.decay, np.float64)
                 with np.errstate(divide="ignore"):
-                    self.V[f"layer_param.{i}.mix.right.log_decay"] = rt.to_device(np.maximum(np.log(np.array(l.mixer.right.decay, np.float64)), -1e4).astype(np.float32))
+                    self.V[f"layer_param.{i}.mix.right.decay"] = rt.to_device(np.concatenate([np.maximum(np.log(d), -1e4), d]).astype(np.float32))
 
     def _grow_logits(self, wanted: int):
         if wanted > self.wanted_rows:

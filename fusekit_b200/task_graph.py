@@ -330,7 +330,7 @@ def _recurrence(layer):
 
 def _recurrence_bufs(lp: str, pre: str, buf: str, run: int, memory: bool, logits: str, out: str) -> dict:
     bufs = {0: buf + "q", 1: buf + "k", 2: buf + "v", 6: f"layer_state.{run}", 7: out}
-    return {**bufs, **({3: logits, 4: lp + pre + "bias"} if memory else {5: lp + pre + "log_decay"})}
+    return {**bufs, **({3: logits, 4: lp + pre + "bias"} if memory else {5: lp + pre + "decay"})}
 
 
 def parallel_decode_tasks(spec, capacity: int, dtype: int = 0, sm: int = 148) -> list:

@@ -215,7 +215,7 @@ enum { FK_ACT_NONE = 0, FK_ACT_RELU_SQUARED = 2, FK_ACT_SILU = 3 };
  *                      i0 H | G << 16  i1 dim | vdim << 16  i2 capacity  i3 dtype of the caches  i4 key splits  i5 window  i6 keep
  *                      i7 rotated dimensions   f0 scale  f1 eps
  * RECURRENCE_ROWS      buf0 q A[M,ld] (heads one after the other)  buf1 k  buf2 v  buf3 gate logits f32[M,i5] (input gates, then forget gates)|0  buf4 their
- *                      biases T[2*heads]|0  buf5 log decays f32[heads]|0  buf6 state  buf7 out A[M,i6]  buf8 scratch|0 (i7 floats of it)
+ *                      biases T[2*heads]|0  buf5 f32[2][heads] log decays, decays|0  buf6 state  buf7 out A[M,i6]  buf8 scratch|0 (i7 floats of it)
  *                      i0 heads | dtype << 16  i1 dim  i2 vdim  i3 M  i4 ld  i5 ld of the logits  i6 ld of out  i7 scratch floats
  *                      f0 factor on q  f1 gate cap.  With buf5 the decay form, with buf3 and buf4 the matrix memory
  * RECURRENCE_DECODE    one position, the same with f32 vectors (buf0 .. buf7; strides and scratch are not used)

@@ -5,8 +5,9 @@ import numpy as np
 
 from fusekit_b200 import checkpoint as CK
 from fusekit_b200.layered import LayeredEngine, tensor_shapes
-from fusekit_b200.model_spec import AttentionSpec, LayeredSpec, LayerSpec, LoopSpec, MoeSpec
-from oracle.layered import LayeredOracle
+from fusekit_b200.model_spec import (AttentionSpec, ClampedGluSpec, FrequencyScaling, LayeredSpec, LayerSpec, LightningSpec, LoopSpec, MatrixMemorySpec, MoeSpec,
+                                     ParallelMixerSpec, RotarySpec)
+from oracle.layered import LayeredOracle, ParallelBlockOracle
 
 
 def bits(a):
@@ -39,6 +40,10 @@ def random_tensors(s, seed=0, router=6.0):
             a *= 0.25
         elif n.endswith(("q.norm", "k.norm")):
             a = 1.3 + 0.3 * a
+        elif n.endswith(".f.b"):
+            a = 3.0 + a                                  # long memories
+        elif n.endswith(".b"):
+            a *= 0.5
         elif len(shape) == 1:
             a = 1.0 + 0.2 * a
         else:
@@ -58,7 +63,20 @@ def engine(s, tensors, capacity, dtype="float32", **kw):
 
 
 def oracle(s, tensors):
-    return LayeredOracle(s, {k: values(v) for k, v in tensors.items()})
+    return (ParallelBlockOracle if s.block == "parallel" else LayeredOracle)(s, {k: values(v) for k, v in tensors.items()})
+
+
+def parallel_entry(m, f):
+    if isinstance(m, ParallelMixerSpec):
+        l, r, rot = m.left, m.right, m.left.rotary
+        left = {"heads": l.heads, "kv_heads": l.kv_heads, "dim": l.dim, "vdim": l.vdim, "scale": l.scale,
+                "mask": None if l.window is None else {"size": l.window, "keep_first": l.keep_first},
+                "rot": None if rot is None else {"dims": rot.dims, "base": rot.base, "scaling": None if rot.scaling is None else vars(rot.scaling)}}
+        e = {"type": "parallel", "mixer": {"left": left, "right": {"heads": r.heads, "dim": r.dim, "vdim": r.vdim, "decay": list(r.decay)}}}
+    else:
+        e = {"type": "mlstm", "mixer": {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "gate_cap": m.gate_cap}}
+    e["mlp"] = None if f is None else {"kind": "dense", "ff": f.ff, "limit": f.limit}
+    return e
 
 
 def write_model(path, s, tensors):
@@ -69,10 +87,15 @@ def write_model(path, s, tensors):
     layers = []
     for l in s.layers:
         m, f = l.mixer, l.mlp
+        if s.block == "parallel":
+            layers.append(parallel_entry(m, f))
+            continue
         layers.append({"type": "attention", "mixer": {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale, "diff": m.diff},
                        "mlp": None if f is None else {"kind": "moe", "router": {"experts": f.experts, "top": f.top}, "expert": {"ff": f.ff},
                                                       "shared": {"ff": f.shared_ff} if f.shared_ff else None}})
     cfg = {"architecture": s.arch, "width": s.hidden, "vocab": s.vocab, "norm": {"eps": s.eps}, "layers": layers}
+    if s.block == "parallel":
+        cfg["logit_scale"] = s.logit_scale
     if s.loop is not None:
         cfg["loop"] = {"start": s.loop.start, "stop": s.loop.stop, "times": s.loop.times}
     with open(os.path.join(path, "config.json"), "w") as f:
@@ -92,6 +115,33 @@ SPECS = {
     "many-rows": spec([LayerSpec(A(10, 1, 20, 16, 0.3, 0.25), M(70, 5, 16, 24)), LayerSpec(A(12, 3, 64, 64, 0.15, 0.6), M(33, 6, 72, 8))], hidden=200, vocab=97),
     "plain-maps": spec([LayerSpec(A(4, 2, 48, 64, 0.2, None), M(8, 2, 64, 96))], hidden=128, vocab=130),
     "one-layer": spec([LayerSpec(A(1, 1, 8, 8, 0.6, 0.3), M(1, 1, 8, 8))], hidden=16, vocab=33, loop=LoopSpec(0, 1, 1)),
+}
+
+
+def parallel_spec(layers, hidden=96, vocab=211, eps=1e-5, logit_scale=1.0, name="test"):
+    return LayeredSpec(name, "Kakunex", hidden, vocab, tuple(layers), eps=eps, block="parallel", logit_scale=logit_scale)
+
+
+def windowed(heads, kv_heads, dim, vdim, scale, window=None, keep=0, rot=None, scaling=None, base=1e4):
+    r = None if rot is None else RotarySpec(rot, base, None if scaling is None else FrequencyScaling(*scaling))
+    return AttentionSpec(heads, kv_heads, dim, vdim, scale, norm="projection", gate=False, rotary=r, window=window, keep_first=keep)
+
+
+P, L, MM, G = ParallelMixerSpec, LightningSpec, MatrixMemorySpec, ClampedGluSpec
+# sizes off every tile, unequal layers, windows of one / none / larger than a tile, no kept keys / more than a tile of them, rotation of all / some / no
+# dimensions, with and without stretching, decays of 0 and 1, layers without feed-forward, widths that no vector load fits
+PARALLEL_SPECS = {
+    "mixed": parallel_spec([LayerSpec(P(windowed(4, 2, 24, 40, 0.3, 20, 5, 16, (4.0, 1.0, 4.0, 50.0)), L(3, 16, 24, (0.5, 0.9, 1.0))), G(72, 0.8)),
+                            LayerSpec(MM(3, 24, 40, 8.0), None), LayerSpec(P(windowed(3, 1, 20, 12, 0.25, 1, 0, 20), L(1, 40, 72, (0.97,))), None),
+                            LayerSpec(MM(1, 8, 136, 20.0), G(40, 3.0)), LayerSpec(P(windowed(5, 5, 8, 16, 0.5, None, 0, None), L(5, 8, 8, (0.0, 0.3, 0.6, 0.8, 0.999))), G(24, 100.0))],
+                           hidden=88, logit_scale=1.7),
+    "memory-first": parallel_spec([LayerSpec(MM(2, 72, 16, 5.0), G(136, 1.0)), LayerSpec(MM(4, 16, 64, 15.0), G(8, 0.5)),
+                                   LayerSpec(P(windowed(2, 2, 40, 64, 0.2, 70, 66, 40, (8.0, 1.0, 2.0, 30.0)), L(2, 136, 64, (0.99, 0.8))), G(64, 2.0))], hidden=136, vocab=130),
+    "odd-sizes": parallel_spec([LayerSpec(P(windowed(6, 3, 18, 22, 0.25, 33, 3, 6, (2.0, 1.0, 3.0, 40.0)), L(3, 10, 14, (0.7, 0.95, 0.2))), G(37, 1.2)),
+                                LayerSpec(MM(3, 14, 18, 11.0), G(21, 0.9)), LayerSpec(MM(2, 5, 7, 6.0), None)], hidden=75, vocab=99, eps=1e-3, logit_scale=0.4),
+    "wide-heads": parallel_spec([LayerSpec(P(windowed(12, 1, 136, 200, 0.1, 40, 10, 136), L(1, 264, 130, (0.9,))), G(48, 4.0)),
+                                 LayerSpec(MM(1, 200, 72, 15.0), G(33, 2.0))], hidden=64, vocab=80),
+    "one-layer": parallel_spec([LayerSpec(P(windowed(1, 1, 8, 8, 0.6, 4, 2, 8), L(1, 8, 8, (0.9,))), G(8, 1.0))], hidden=16, vocab=33, logit_scale=3.0),
 }
 
 
