@@ -107,9 +107,11 @@ class AttentionCase:
         self.qq = OL.rotate_pairs(OL.rms_norm(self.q.reshape(n, -1), self.qn, self.eps).reshape(n, H, dim), at, f)
         self.kk = OL.rotate_pairs(OL.rms_norm(self.k.reshape(n, -1), self.kn, self.eps).reshape(n, G, dim), at, f)
 
-    def want(self, lo, hi, window=..., keep=None):
+    def want(self, lo, hi, window=..., keep=None, f32=1, q16=False):
+        """Outputs of positions lo .. hi - 1; in bf16 the keys are taken as a cache holds them (and the queries as a buffer does)."""
+        kk, qq = (self.kk, self.qq) if f32 else (LM.rounded(self.kk).astype(np.float64), LM.rounded(self.qq).astype(np.float64) if q16 else self.qq)
         w, kp = self.window if window is ... else window, self.keep if keep is None else keep
-        o = [OL.window_attention(self.qq[lo:hi, h], self.kk[:hi, h // (self.H // self.G)], self.v[:hi, h // (self.H // self.G)], self.scale, lo, w, kp) for h in range(self.H)]
+        o = [OL.window_attention(qq[lo:hi, h], kk[:hi, h // (self.H // self.G)], self.v[:hi, h // (self.H // self.G)], self.scale, lo, w, kp) for h in range(self.H)]
         return np.concatenate(o, 1)
 
     def caches(self, dev, cap, filled, f32, noise):
@@ -138,7 +140,7 @@ WINDOWS = [(None, 0), (1, 0), (7, 3), (64, 0), (40, 70), (130, 5)]
 def test_rotary_store_and_window_attention_rows(runtime, dev, H, G, dim, vdim, rot, f32, before, rows):
     rng = np.random.default_rng(H * 1000 + dim + before)
     n, cap = before + rows, before + rows + 3
-    sz, tol, ld, ldo, dp, vp = 4 if f32 else 2, 4e-5 if f32 else 2e-2, up((H + G) * dim + G * vdim, 64), up(H * vdim, 64), up(dim, 8), up(vdim, 8)
+    sz, tol, ld, ldo, dp, vp = 4 if f32 else 2, 4e-5 if f32 else 1.2e-2, up((H + G) * dim + G * vdim, 64), up(H * vdim, 64), up(dim, 8), up(vdim, 8)
     for window, keep in WINDOWS:
         for far in edges(window, keep, n - 1):
             c = AttentionCase(rng, H, G, dim, vdim, rot, n, [n - 1], far, window, keep)
@@ -154,7 +156,7 @@ def test_rotary_store_and_window_attention_rows(runtime, dev, H, G, dim, vdim, r
             kc = dev.get(ck, (G, cap, dp), f32)
             close(kc[:, before:n, :dim], c.kk[before:].transpose(1, 0, 2), 3e-6 if f32 else 5e-3, "stored keys")
             assert (kc[:, n:, :dim] == 3.0).all()
-            want, got = c.want(before, n), dev.get(out, (rows, ldo), f32)[:, :H * vdim]
+            want, got = c.want(before, n, f32=f32, q16=True), dev.get(out, (rows, ldo), f32)[:, :H * vdim]
             close(got, want, tol, f"window {window} keep {keep} far {far}")
             close(got[-1], want[-1], tol, f"last position, window {window} keep {keep} far {far}")
             # the cases tell a window or a kept prefix that is one off
@@ -185,22 +187,30 @@ def test_window_attention_decode(runtime, dev, H, G, dim, vdim, rot, f32):
                                 {0: dev.put(raw), 1: dev.put(LM.bits(c.qn)), 2: dev.put(LM.bits(c.kn)), 3: ck, 4: cv, 5: out, 6: part, 7: cnt, 8: dev.put(rotation_table(c.rot, cap)) if rot else 0},
                                 [H | G << 16, dim | vdim << 16, cap, f32, splits, window or 0, keep, rot], [c.scale, c.eps])
                 runtime.state_set(0, pos)
-                want = c.want(pos, pos + 1)[0]
+                want = c.want(pos, pos + 1, f32=f32)[0]
                 for _ in range(2):                       # the split counters are left as they were found
                     runtime.launch(t)
                     assert runtime.state_get()[2] == 0
-                    close(runtime.download(out, (H * vdim,), np.float32), want, 4e-5 if f32 else 1e-2, f"window {window} keep {keep} pos {pos} splits {splits} far {far}")
+                    close(runtime.download(out, (H * vdim,), np.float32), want, 4e-5 if f32 else 8e-3, f"window {window} keep {keep} pos {pos} splits {splits} far {far}")
                 kc, vc = dev.get(ck, (G, cap, dp), f32), dev.get(cv, (G, cap, vp), f32)
                 close(kc[:, pos, :dim], c.kk[pos], 3e-6 if f32 else 5e-3, "stored key")
                 assert np.array_equal(vc[:, pos, :vdim], c.v[pos].astype(np.float32)) and (kc[:, pos + 1:, :dim] == 3.0).all()
 
 
 def memory_want(q, k, v, zi, zf, bi, bf, cap, states):
-    out = np.zeros(v.shape)
+    """Outputs and, for each, the magnitude that rounding errors are a fraction of: the sums of the numerator and of the divisor taken
+    with absolute values (the divisor |n . q| may come close to zero and blow up the output together with its error)."""
+    out, size = np.zeros(v.shape), np.zeros(v.shape)
     for h in range(q.shape[1]):
         gi, gf = OL.soft_cap(zi[:, h] + bi[h], cap), OL.log_sigmoid(OL.soft_cap(zf[:, h] + bf[h], cap))
         out[:, h], states[h] = OL.matrix_memory(q[:, h], k[:, h], v[:, h], gi, gf, states[h])
-    return out
+        n, A, B, m = np.zeros(q.shape[2]), np.zeros((q.shape[2], v.shape[2])), np.zeros(q.shape[2]), 0.0
+        for t in range(len(q)):
+            new = max(gf[t] + m, gi[t])
+            keep, add, m = np.exp(gf[t] + m - new), np.exp(gi[t] - new), new
+            n, A, B = keep * n + add * k[t, h], keep * A + add * np.outer(abs(k[t, h]), abs(v[t, h])), keep * B + add * abs(k[t, h])
+            size[t, h] = (A.T @ abs(q[t, h]) + abs(out[t, h]) * (B @ abs(q[t, h]))) / (max(abs(n @ q[t, h]), np.exp(-m)) + 1e-6)
+    return out, size
 
 
 REC = [(1, 8, 8), (3, 16, 24), (2, 40, 72), (2, 64, 64), (4, 128, 128), (1, 200, 136), (2, 256, 64), (1, 264, 16), (3, 10, 14), (1, 5, 130)]
@@ -225,10 +235,11 @@ def test_recurrence(runtime, dev, heads, dim, vdim, form, dtype):
     rec = LM.MM(heads, dim, vdim, cap) if mem else LM.L(heads, dim, vdim, tuple(decay))
     if mem:
         states = [(np.zeros((dim, vdim)), np.zeros(dim), 0.0) for _ in range(heads)]
-        want = memory_want(q * float(qs), k.astype(np.float64), v.astype(np.float64), zi.astype(np.float64), zf.astype(np.float64), bi, bf, cap, states)
+        want, size = memory_want(q * float(qs), k.astype(np.float64), v.astype(np.float64), zi.astype(np.float64), zf.astype(np.float64), bi, bf, cap, states)
     else:
-        states, want = np.zeros((heads, dim, vdim)), np.zeros((T, heads, vdim))
+        states, want, size = np.zeros((heads, dim, vdim)), np.zeros((T, heads, vdim)), np.zeros((T, heads, vdim))
         for h in range(heads):
+            size[:, h] = OL.decay_recurrence(abs(q[:, h]) * float(qs), abs(k[:, h]).astype(np.float64), abs(v[:, h]).astype(np.float64), decay[h], states[h])[0]
             want[:, h], states[h] = OL.decay_recurrence(q[:, h] * float(qs), k[:, h].astype(np.float64), v[:, h].astype(np.float64), decay[h], states[h])
     slices, cell = -(-vdim // 64), TG.recurrence_cell(rec)
     state = dev.put(np.full(TG.recurrence_state(rec), np.nan, np.float32))
@@ -250,12 +261,8 @@ def test_recurrence(runtime, dev, heads, dim, vdim, form, dtype):
         assert runtime.state_get()[2] == 0
         got.append(dev.get(out, (n, ldo), f32)[:, :heads * vdim].reshape(n, heads, vdim)); at += n
     got = np.concatenate(got)
-    for h in range(heads):
-        # every stretch by itself, so that a fault at a border is not lost in what follows
-        for lo in range(0, T, 50):
-            a, b = got[lo:lo + 50, h], want[lo:lo + 50, h]
-            spread = max(np.abs(b).max(), 0.05 * np.abs(want[:, h]).max())
-            assert np.abs(a - b).max() <= (3e-5 if f32 else 1e-2) * spread, (h, lo, np.abs(a - b).max() / spread)
+    err = np.abs(got - want) / ((3e-6 if f32 else 2e-5) * size + (0.0 if f32 else 2.0 ** -8) * np.abs(want) + 1e-9)
+    assert err.max() <= 1.0, (np.unravel_index(err.argmax(), err.shape), err.max())
     st = runtime.download(state, (heads, slices, cell), np.float32)
     for h in range(heads):
         S = np.concatenate(list(st[h, :, :dim * 64].reshape(slices, dim, 64)), 1)[:, :vdim]
@@ -421,14 +428,15 @@ def test_a_key_at_the_edge_of_what_is_seen_decides_the_output(runtime, dtype):
     u = np.random.default_rng(0).standard_normal(16)
     q[:, 1] = np.tile(u, 2) * 3; k[:, 0] = u * 3
     t["l0.mix.left.q"], t["l0.mix.left.k"] = LM.bits(q), LM.bits(k)
-    t["l0.mix.right.out"] = LM.bits(np.full(64, 0.01))
+    t["l0.mix.right.out"], t["l0.mix.left.out"] = LM.bits(np.full(64, 0.01)), LM.bits(3 * LM.values(t["l0.mix.left.out"]))
     n = 150
     e = LM.engine(s, t, n + 4, dtype, runtime=runtime)
     for far, seen in ((0, 1), (K - 1, 1), (K, 0), (n - 1 - W, 0), (n - W, 1), (n - 2, 1), (64, 0)):
         toks = np.random.default_rng(far).integers(10, s.vocab, n); toks[far] = 7; toks[-1] = 8
         without = toks.copy(); without[far] = 11
         want, blind = (LM.oracle(s, t).forward(x)[-1:] for x in (toks, without))
-        assert (LM.logit_error(blind, want)[0] > 0.15) == bool(seen), far
+        change = LM.logit_error(blind, want)[0]
+        assert change > 0.3 if seen else change < 0.01, far
         for cut in (0, n - 1, n - 2, 64):
             seq = e.open_sequence()
             if cut:
