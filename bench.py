@@ -321,6 +321,8 @@ def run_layered(args, local: int):
     def chunks(eng, seed, base):
         tok, dev, wall = seed, 0.0, 0.0
         for i in range(args.warmup + args.steps):
+            if hasattr(eng, "at"):
+                eng.at[eng.slot] = base                  # the same positions again: what a state holds does not matter here
             t0 = time.perf_counter()
             out, s = eng.decode_chunk(base, tok, CHUNK)
             tok = int(out[-1])
@@ -330,6 +332,9 @@ def run_layered(args, local: int):
 
     for name in names:
         spec = LAYERED_CONFIGS[name]
+        if spec.block == "parallel":
+            run_parallel(args, local, name, spec, frac, chunks, peak, flops_peak, peak_kind)
+            continue
         m, f, D, L = spec.layers[0].mixer, spec.layers[0].mlp, spec.hidden, len(spec.layers)
         runs = spec.runs()
         first = {i: r for r, (i, _) in reversed(list(enumerate(runs)))}       # a layer's first run
@@ -429,6 +434,112 @@ def run_layered(args, local: int):
             "like_model": {"model": q.name, "layers": L, "inter": inter, "decode_tok_s_bf16": odec, "decode_roofline_frac": obytes * odec / 1e9 / peak,
                            "prompt_tok_s_q4_16_rows": P / osecs},
             "peaks": {"hbm_gbs": peak, "bf16_tflops": flops_peak, "kind": peak_kind}, "clocks": clocks, "kernels": kern, "like_kernels": like}), flush=True)
+
+
+def run_parallel(args, local, name, spec, frac, chunks, peak, flops_peak, peak_kind):
+    """run_layered for a model of parallel blocks.  Like kernels: decode against a Qwen-shaped bf16 decoder of the same width, heads and
+    feed-forward size (as many layers), prompt rows against the sandwich-block decoder registered at the same width."""
+    from fusekit_b200 import _native as N
+    from fusekit_b200.model_spec import LAYERED_CONFIGS, ModelSpec, ParallelMixerSpec, block_layout
+    from fusekit_b200.runtime import DecodeEngine, attach
+    ctx, P, D, L = LAYERED_CTX, LAYERED_PROMPT, spec.hidden, len(spec.layers)
+    both = [i for i, l in enumerate(spec.layers) if isinstance(l.mixer, ParallelMixerSpec)]
+    mems = [i for i in range(L) if i not in both]
+    a, r, mm, f = spec.layers[both[0]].mixer.left, spec.layers[both[0]].mixer.right, spec.layers[mems[0]].mixer, spec.layers[0].mlp
+    joint = {k: sum(n for _, _, n in block_layout(spec.layers[g[0]]).sources) + 2 * f.ff for k, g in (("parallel", both), ("memory", mems))}
+    eng = attach(spec, max(ctx + CHUNK, P) + 8, device=local, max_rows=P)
+    eng.load_synthetic(); eng.prefill_kv_synthetic(ctx); eng.capture()
+    rt, kern = eng.rt, {}
+    sampler = ClockSampler(local); sampler.start()
+    dec, dec_e2e = chunks(eng, 3, ctx)
+    rt.state_set(3, ctx)
+
+    def add(key, tasks, nbytes, flops=0.0, e=None, table=None):
+        secs = (e or eng).time_tasks(tasks, 5) / len(tasks)
+        (kern if table is None else table)[key] = {"us": secs * 1e6, "frac": frac(secs, nbytes, flops), "bytes": nbytes, "flops": flops}
+
+    pick = lambda kind, of, group, w=None: [t for t in of if t.kind == kind and t.layer in group and (w is None or t.buf[1] in [eng.W[f"layer_param.{i}.{w}"] for i in group])]
+    lin = lambda n, k: (2 * (P * k + n * k + P * n), 2.0 * P * n * k)
+    state = lambda x: 8 * x.heads * x.dim * x.vdim
+    for k, g in (("parallel", both), ("memory", mems)):
+        add(f"decode joint projection, {k} layer", pick(N.TASK_NORM_LINEAR, eng.replay, g), 2 * D * joint[k])
+    add("decode attention", pick(N.TASK_WINDOW_ATTENTION_DECODE, eng.replay, both), 2 * a.visible(ctx) * (a.k_rows + a.v_rows))
+    add("decode linear attention", pick(N.TASK_RECURRENCE_DECODE, eng.replay, both), state(r))
+    add("decode matrix memory", pick(N.TASK_RECURRENCE_DECODE, eng.replay, mems), state(mm))
+    add("decode output projections, parallel layer", pick(N.TASK_SEGMENT_LINEAR, eng.replay, both), 2 * D * (a.out_rows + r.out_rows + f.ff))
+    add("decode output projections, memory layer", pick(N.TASK_SEGMENT_LINEAR, eng.replay, mems), 2 * D * (mm.out_rows + f.ff))
+    add("decode head", [eng.replay[-1]], 2 * D * spec.vocab)
+    rows = eng.rows_dispatches(P, 0, False)
+    rt.upload(eng.scratch["rows_scratch.tokens"], np.random.default_rng(0).integers(0, spec.vocab, P).astype(np.uint32))
+    rt.state_set(0, 0)
+    pre_secs = eng.time_tasks(rows, max(2, args.steps))
+    for k, g in (("parallel", both), ("memory", mems)):
+        add(f"rows joint projection, {k} layer", pick(N.TASK_BLOCK_LINEAR_ROWS, rows, g), *(lambda b, fl: (b - 2 * P * f.ff, fl))(*lin(joint[k], D)))
+    pairs = sum(a.visible(p + 1) for p in range(P))
+    add("rows attention", pick(N.TASK_WINDOW_ATTENTION_ROWS, rows, both), 2 * P * (a.q_rows + a.k_rows + a.v_rows + a.out_rows), 2.0 * a.heads * (a.dim + a.vdim) * pairs)
+    add("rows joint q/k norm + rotation + store", pick(N.TASK_ROTARY_STORE_ROWS, rows, both), 4 * P * a.rows)
+    add("rows linear attention", pick(N.TASK_RECURRENCE_ROWS, rows, both), 2 * P * (r.qkv_rows + r.out_rows), 4.0 * P * r.heads * r.dim * r.vdim)
+    add("rows matrix memory", pick(N.TASK_RECURRENCE_ROWS, rows, mems), 2 * P * (mm.qkv_rows + mm.out_rows), 4.0 * P * mm.heads * mm.dim * mm.vdim)
+    add("rows norm + gate", pick(N.TASK_NORM_GATE_ROWS, rows, both), 6 * P * r.out_rows)
+    add("rows attention output projection", pick(N.TASK_LINEAR_ROWS, rows, both, "mix.left.o"), *lin(D, a.out_rows))
+    add("rows linear attention output projection", pick(N.TASK_LINEAR_ROWS, rows, both, "mix.right.o"), *lin(D, r.out_rows))
+    add("rows down", pick(N.TASK_LINEAR_ROWS, rows, range(L), "mlp.down"), *lin(D, f.ff))
+    add("rows residual + norm", [t for t in pick(N.TASK_BLOCK_NORM_ROWS, rows, both[1:]) if t.iarg[5] == 3], P * D * (3 * 2 + 2 + 4 + 4))
+    clocks = sampler.stop()
+    for _ in range(2):
+        t0 = time.perf_counter(); eng.prefill(np.arange(P) % spec.vocab); wall = time.perf_counter() - t0
+    eng.close()
+
+    q, like = ModelSpec(f"qwen-like-{D}", "qwen2", L, D, a.heads, a.kv_heads, 128, f.ff // 64 * 64, spec.vocab, bits=16), {}
+    old = DecodeEngine(q, ctx + CHUNK + 8, device=local)
+    old.load_synthetic(); old.prefill_kv_synthetic(ctx); old.capture()
+    odec, _ = chunks(old, 3, ctx)
+    old.rt.state_set(3, ctx)
+    okind = lambda k, n=None: [t for t in old.tasks if t.kind == k and (n is None or (t.iarg[0], t.iarg[1]) == n)]
+    add("qkv", okind(2), q.linear_bytes(D, (q.n_q + 2 * q.n_kv) * 128), e=old, table=like)
+    add("attention", okind(4), 4 * q.n_kv * 128 * ctx, e=old, table=like)
+    add("o", okind(5, (q.n_q * 128, D)), q.linear_bytes(q.n_q * 128, D, True), e=old, table=like)
+    add("gate/up", okind(6), 2 * q.linear_bytes(D, q.inter), e=old, table=like)
+    add("down", okind(5, (q.inter, D)), q.linear_bytes(q.inter, D, True), e=old, table=like)
+    add("head", okind(7), q.linear_bytes(D, q.vocab), e=old, table=like)
+    obytes = q.bytes_per_token(ctx)
+    old.close()
+    sname = f"fatulix-{D}"
+    sw = LAYERED_CONFIGS[sname]
+    m, g = sw.layers[0].mixer, sw.layers[0].mlp
+    se = attach(sw, P + 8, device=local, max_rows=P)
+    se.load_synthetic()
+    srows = se.rows_dispatches(P, 0, False)
+    se.rt.upload(se.scratch["rows_scratch.tokens"], np.random.default_rng(0).integers(0, sw.vocab, P).astype(np.uint32))
+    se.rt.state_set(0, 0)
+    spre = se.time_tasks(srows, max(2, args.steps))
+    ids = lambda w: [se.W[f"layer_param.{i}.{w}"] for i in range(len(sw.layers))]
+    sp = lambda kind, w=None, row0=0: [t for t in srows if t.kind == kind and (w is None or (t.buf[1] in ids(w) and t.iarg[1] == row0))]
+    add("s rows q|k|v|gate", sp(N.TASK_LINEAR_ROWS, "mix.qkvg"), *lin(m.rows, D), e=se, table=like)
+    add("s rows shared up", sp(N.TASK_LINEAR_ROWS, "mlp.router_shared", g.experts), *lin(g.shared_ff, D), e=se, table=like)
+    add("s rows attention", sp(N.TASK_ATTENTION_ROWS), 2 * P * (m.q_rows + m.k_rows + m.v_rows + m.heads * m.vdim), m.heads * m.maps * (m.dim + m.vdim) * float(P) * P, e=se, table=like)
+    add("s rows output projection", sp(N.TASK_LINEAR_ROWS, "mix.o"), *lin(D, m.heads * m.vdim), e=se, table=like)
+    add("s rows shared down", sp(N.TASK_LINEAR_ROWS, "mlp.shared_down"), *lin(D, g.shared_ff), e=se, table=like)
+    add("s rows residual + norm", [t for t in sp(N.TASK_RESIDUAL_NORM_ROWS) if t.buf[1] and not t.buf[8] and t.buf[4]], P * D * (2 + 2 + 4 + 4), e=se, table=like)
+    add("s rows q/k norm + store", sp(N.TASK_QK_NORM_STORE_ROWS), 4 * P * (m.rows - m.heads), e=se, table=like)
+    se.close()
+    pair = {"decode joint projection, parallel layer": "gate/up", "decode joint projection, memory layer": "gate/up", "decode attention": "attention", "decode linear attention": "attention",
+            "decode matrix memory": "attention", "decode output projections, parallel layer": "down", "decode output projections, memory layer": "down", "decode head": "head",
+            "rows joint projection, parallel layer": "s rows shared up", "rows joint projection, memory layer": "s rows shared up", "rows attention": "s rows attention",
+            "rows linear attention": "s rows attention", "rows matrix memory": "s rows attention", "rows joint q/k norm + rotation + store": "s rows q/k norm + store",
+            "rows norm + gate": "s rows q/k norm + store", "rows attention output projection": "s rows output projection", "rows linear attention output projection": "s rows output projection",
+            "rows down": "s rows shared down", "rows residual + norm": "s rows residual + norm"}
+    for k, v in kern.items():
+        v["like"], v["like_frac"], v["like_frac_over_frac"] = pair[k], like[pair[k]]["frac"], like[pair[k]]["frac"] / v["frac"]
+    print(json.dumps({
+        "metric": f"layered decoder {name}: decode tok/s at context {ctx}, prompt tok/s at {P}", "value": dec, "unit": "tok/s", "n_gpus": 1, "steps": args.steps,
+        "warmup": args.warmup, "higher_is_better": True, "dtype": "bf16", "data": "synthetic",
+        "config": {"model": name, "layers": L, "l2": "one launch per layer: products read weights larger than L2 in all, caches and states stay in it"},
+        "decode": {"tok_s": dec, "e2e_tok_s": dec_e2e, "roofline_frac": spec.bytes_per_token(ctx) * dec / 1e9 / peak, "bytes_per_token": spec.bytes_per_token(ctx)},
+        "prompt": {"tok_s": P / pre_secs, "e2e_tok_s": P / wall, "tflops": spec.flops_per_token(P / 2) * P / pre_secs / 1e12},
+        "like_model": {"model": q.name, "layers": L, "inter": q.inter, "decode_tok_s_bf16": odec, "decode_roofline_frac": obytes * odec / 1e9 / peak},
+        "like_rows_model": {"model": sname, "runs": len(sw.runs()), "prompt_tok_s": P / spre, "tflops": sw.flops_per_token(P / 2) * P / spre / 1e12},
+        "peaks": {"hbm_gbs": peak, "bf16_tflops": flops_peak, "kind": peak_kind}, "clocks": clocks, "kernels": kern, "like_kernels": like}), flush=True)
 
 
 def main():

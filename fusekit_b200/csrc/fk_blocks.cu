@@ -53,10 +53,12 @@ fk_status fkb_run(FklEnv &c, const fk_task &t, char *err, size_t ecap) {
         if ((size_t)a.d * 4 > 200 * 1024) return bad(err, ecap, "block_norm_rows: width above 51200");
         const dim3 g(i[1]);
         if (a.d % 4 == 0 && a.d <= 8192 && a.ldh % 4 == 0 && a.ldy % 4 == 0) {
-            const dim3 blk(a.d <= 512 ? 128 : 256);
-#define BN(T, NV) launch(c, (k_block_norm_rows4<T, NV>), g, blk, 0, st, a)
-            if (i[2]) e = a.d <= 1024 ? BN(float, 1) : a.d <= 2048 ? BN(float, 2) : a.d <= 4096 ? BN(float, 4) : BN(float, 8);
-            else e = a.d <= 1024 ? BN(uint16_t, 1) : a.d <= 2048 ? BN(uint16_t, 2) : a.d <= 4096 ? BN(uint16_t, 4) : BN(uint16_t, 8);
+            // one round of four values per thread up to 2048, two above; as many threads as that takes
+            const int nv = a.d <= 2048 ? 1 : 2;
+            const dim3 blk(round_up((a.d / 4 + nv - 1) / nv, 32));
+#define BN(T, NV, NT, BLOCKS) launch(c, (k_block_norm_rows4<T, NV, NT, BLOCKS>), g, blk, 0, st, a)
+            if (i[2]) e = a.d <= 2048 ? BN(float, 1, 512, 2) : a.d <= 4096 ? BN(float, 2, 512, 2) : BN(float, 2, 1024, 1);
+            else e = a.d <= 2048 ? BN(uint16_t, 1, 512, 3) : a.d <= 4096 ? BN(uint16_t, 2, 512, 2) : a.d <= 5120 ? BN(uint16_t, 2, 640, 2) : BN(uint16_t, 2, 1024, 1);
 #undef BN
             break;
         }
@@ -91,9 +93,9 @@ fk_status fkb_run(FklEnv &c, const fk_task &t, char *err, size_t ecap) {
         a.sstride = rec_state_stride(a.dim, mem);
         const bool aligned = ((b[0] | b[1] | b[2]) & 15) == 0 && a.ld % 8 == 0 && a.dim % 8 == 0 && a.vdim % 8 == 0 && (b[7] & 3) == 0 && a.ldo % 2 == 0;
         if (!f32 && a.rows >= FKB_CHUNK_MIN_ROWS && a.dim <= 256 && aligned) {
-            // runs of chunks side by side: as many as it takes to give every SM a block, at least four chunks each
+            // runs of chunks side by side: as many as it takes to fill every SM, at least four chunks each
             const int chunks = (a.rows + FKL_CH - 1) / FKL_CH, cells = a.heads * ((a.vdim + FKL_RC_COLS - 1) / FKL_RC_COLS);
-            int runs = b[8] ? c.sm_count / cells : 1;
+            int runs = b[8] ? (a.dim <= 128 ? 2 : 1) * c.sm_count / cells : 1;
             if (runs > chunks / 4) runs = chunks / 4;
             if (runs > FKB_MAX_SEGMENTS) runs = FKB_MAX_SEGMENTS;
             while (runs > 1 && (long long)(runs + 1) * cells * a.sstride + (long long)runs * cells > i[7]) --runs;

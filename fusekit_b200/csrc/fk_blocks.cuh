@@ -13,20 +13,35 @@ struct BlockNormArgs {
     const float *x; const void *y[3]; const uint16_t *post; float *x_out; const uint16_t *w, *b; void *h; const uint32_t *index;
     int d, ldh, ldy, np, nnorm; float eps, scale;
 };
-template <typename T, int NV>
-__global__ void __launch_bounds__(256) k_block_norm_rows4(const FkState *st, BlockNormArgs a) {
+// four values as they are stored
+template <typename T> struct Raw4;
+template <> struct Raw4<uint16_t> {
+    uint2 v;
+    __device__ __forceinline__ void load(const uint16_t *p) { v = __ldcg(reinterpret_cast<const uint2 *>(p)); }
+    __device__ __forceinline__ void zero() { v = make_uint2(0, 0); }
+    __device__ __forceinline__ float4 get() const { return make_float4(bf_lo(v.x), bf_hi(v.x), bf_lo(v.y), bf_hi(v.y)); }
+};
+template <> struct Raw4<float> {
+    float4 v;
+    __device__ __forceinline__ void load(const float *p) { v = __ldcg(reinterpret_cast<const float4 *>(p)); }
+    __device__ __forceinline__ void zero() { v = make_float4(0.0f, 0.0f, 0.0f, 0.0f); }
+    __device__ __forceinline__ float4 get() const { return v; }
+};
+// rows of a multiple of 4 and at most NV * 4 * blockDim.x values: everything in registers, one round of loads
+template <typename T, int NV, int NT, int BLOCKS>
+__global__ void __launch_bounds__(NT, BLOCKS) k_block_norm_rows4(const FkState *st, BlockNormArgs a) {
     __shared__ float red[66];
     const int tid = threadIdx.x, nt = blockDim.x;
     pdl_wait(); pdl_launch_dependents();
     const size_t row = a.index ? a.index[blockIdx.x] : blockIdx.x;
-    const float4 zero = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
-    float4 x[NV], y[3][NV];
+    float4 x[NV];
+    Raw4<T> y[3][NV];
 #pragma unroll
     for (int v = 0; v < NV; ++v) {
         const int i = (v * nt + tid) * 4;
-        x[v] = i < a.d ? ld4(a.x + row * a.d + i) : zero;
+        x[v] = i < a.d ? ld4(a.x + row * a.d + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
-        for (int p = 0; p < 3; ++p) y[p][v] = p < a.np && i < a.d ? ld4((const T *)a.y[p] + row * a.ldy + i) : zero;
+        for (int p = 0; p < 3; ++p) { if (p < a.np && i < a.d) y[p][v].load((const T *)a.y[p] + row * a.ldy + i); else y[p][v].zero(); }
     }
     float f[3] = {1.0f, 1.0f, 1.0f};
     if (a.nnorm > 0) {
@@ -34,7 +49,7 @@ __global__ void __launch_bounds__(256) k_block_norm_rows4(const FkState *st, Blo
 #pragma unroll
         for (int p = 0; p < 3; ++p)
 #pragma unroll
-            for (int v = 0; v < NV; ++v) ss[p] = fmaf(y[p][v].x, y[p][v].x, fmaf(y[p][v].y, y[p][v].y, fmaf(y[p][v].z, y[p][v].z, fmaf(y[p][v].w, y[p][v].w, ss[p]))));
+            for (int v = 0; v < NV; ++v) { const float4 e = y[p][v].get(); ss[p] = fmaf(e.x, e.x, fmaf(e.y, e.y, fmaf(e.z, e.z, fmaf(e.w, e.w, ss[p])))); }
         const float2 s01 = block_sum2(ss[0], ss[1], red);
         f[0] = a.scale * inv_rms(s01.x, a.d, a.eps);
         if (a.nnorm > 1) f[1] = a.scale * inv_rms(s01.y, a.d, a.eps);
@@ -46,9 +61,9 @@ __global__ void __launch_bounds__(256) k_block_norm_rows4(const FkState *st, Blo
         const int i = (v * nt + tid) * 4;
 #pragma unroll
         for (int p = 0; p < 3; ++p) if (p < a.np && i < a.d) {
-            const float4 w = p < a.nnorm ? ld4(a.post + (size_t)p * a.d + i) : make_float4(1.0f, 1.0f, 1.0f, 1.0f);
-            x[v].x = fmaf(y[p][v].x * f[p], w.x, x[v].x); x[v].y = fmaf(y[p][v].y * f[p], w.y, x[v].y);
-            x[v].z = fmaf(y[p][v].z * f[p], w.z, x[v].z); x[v].w = fmaf(y[p][v].w * f[p], w.w, x[v].w);
+            const float4 w = p < a.nnorm ? ld4(a.post + (size_t)p * a.d + i) : make_float4(1.0f, 1.0f, 1.0f, 1.0f), e = y[p][v].get();
+            x[v].x = fmaf(e.x * f[p], w.x, x[v].x); x[v].y = fmaf(e.y * f[p], w.y, x[v].y);
+            x[v].z = fmaf(e.z * f[p], w.z, x[v].z); x[v].w = fmaf(e.w * f[p], w.w, x[v].w);
         }
         sum += (x[v].x + x[v].y) + (x[v].z + x[v].w);
     }
@@ -65,7 +80,7 @@ __global__ void __launch_bounds__(256) k_block_norm_rows4(const FkState *st, Blo
         const int i = (v * nt + tid) * 4;
         if (i >= a.d) continue;
         if (a.x_out) st4(a.x_out + row * a.d + i, x[v]);
-        const float4 w = ld4(a.w + i), b = a.b ? ld4(a.b + i) : zero;
+        const float4 w = ld4(a.w + i), b = a.b ? ld4(a.b + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
         st4((T *)a.h + (size_t)blockIdx.x * a.ldh + i, make_float4(fmaf((x[v].x - mean) * r, w.x, b.x), fmaf((x[v].y - mean) * r, w.y, b.y),
                                                                    fmaf((x[v].z - mean) * r, w.z, b.z), fmaf((x[v].w - mean) * r, w.w, b.w)));
     }
@@ -252,13 +267,17 @@ __global__ void __launch_bounds__(FKL_RC_THREADS) k_recurrence(FkState *st, RecA
 // are four small matrix products on the tensor cores (mma.m16n8k16).  fp32 factors (scores, weighted keys, the state) enter as two bf16 terms
 // (hi + lo); the state itself stays in fp32 accumulators.
 //
-// One block per (slice of 64 value columns, head, run of chunks).  With several runs, a first pass (OUT = false) leaves each run's
-// own end state in scratch and the second starts every run from the fold of those before it.
+// The normaliser rides along as one more value column that is always 1.  exp(a_s - M_t) needs only F, a and the running maximum of a inside the
+// chunk besides m_0, so the gates of several chunks are worked out at once, a warp each.
+//
+// One block per (slice of 64 value columns, head, run of chunks), two to an SM up to keys of 128.  With several runs, a first pass
+// (OUT = false) leaves each run's own end state in scratch and the second starts every run from the fold of those before it.
 #define FKL_CH 64
 #define FKL_CH_THREADS 256
+#define FKL_CH_GATES 4                // chunks whose gates are worked out together
 template <int KD> struct ChunkSmem {
     static constexpr int KS = KD + 8, VS = FKL_RC_COLS + 8;
-    static constexpr int QK = FKL_CH * KS * 2, V = FKL_CH * VS * 2, STAGE = 2 * QK + V, SH = KD * VS * 2, TOTAL = 2 * STAGE + 2 * SH;
+    static constexpr int K = FKL_CH * KS * 2, V = FKL_CH * VS * 2, Q = 2 * (K + V), SHI = Q + K, SLO = SHI + KD * VS * 2, TOTAL = SLO + KD * VS * 2;
 };
 __device__ __forceinline__ void ch_mma(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
@@ -275,14 +294,13 @@ __device__ __forceinline__ uint32_t ch_pack(float lo, float hi) { const __nv_bfl
 __device__ __forceinline__ void ch_split(float x, float y, uint32_t &hi, uint32_t &lo) { hi = ch_pack(x, y); lo = ch_pack(x - bf_lo(hi), y - bf_hi(hi)); }
 
 template <int KD, bool MEM, bool OUT>
-__global__ void __launch_bounds__(FKL_CH_THREADS) k_recurrence_chunks(FkState *st, RecArgs a) {
+__global__ void __launch_bounds__(FKL_CH_THREADS, KD <= 128 ? 2 : 1) k_recurrence_chunks(FkState *st, RecArgs a) {
     using L = ChunkSmem<KD>;
-    constexpr int KS = L::KS, VS = L::VS;
-    // state tiles of 16 rows: with fewer tiles than warps several warps share one, 8 columns at a time
+    constexpr int KS = L::KS, VS = L::VS, GR = FKL_CH_GATES;
+    // state tiles of 16 rows: with fewer tiles than warps several warps share one, some columns each
     constexpr int TILES = KD / 16, MT = TILES > 8 ? TILES / 8 : 1, SHARE = TILES >= 8 ? 1 : 8 / TILES, NT = 8 / SHARE;
     extern __shared__ __align__(128) unsigned char ch_smem[];
-    __shared__ float sa[2][FKL_CH], sM[2][FKL_CH], sF[2][FKL_CH], sw[FKL_CH], sn[MEM ? KD : 1], sden[FKL_CH];
-    __shared__ float s_end[2][2];                       // F and M at the end of a chunk
+    __shared__ float sF[GR][FKL_CH], sa[GR][FKL_CH], sX[GR][FKL_CH];      // F, a, running maximum of a inside the chunk
     const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5, g8 = lane >> 2, t4 = lane & 3;
     const int slice = blockIdx.x, head = blockIdx.y, run = blockIdx.z, col0 = slice * FKL_RC_COLS;
     const int chunk0 = run * a.per, nchunk = min((a.rows + FKL_CH - 1) / FKL_CH - chunk0, a.per);
@@ -291,72 +309,63 @@ __global__ void __launch_bounds__(FKL_CH_THREADS) k_recurrence_chunks(FkState *s
     const bool fresh = st->offset == 0;
     const float lgd = MEM ? 0.0f : a.log_decay[head], bi = MEM ? bf2f(a.bias[head]) : 0.0f, bf = MEM ? bf2f(a.bias[a.heads + head]) : 0.0f;
     pdl_wait(); pdl_launch_dependents();
-    const uint32_t sbase = (uint32_t)__cvta_generic_to_shared(ch_smem), shi = sbase + 2 * L::STAGE, slo = shi + L::SH;
+    const uint32_t sbase = (uint32_t)__cvta_generic_to_shared(ch_smem), qb = sbase + L::Q, shi = sbase + L::SHI, slo = sbase + L::SLO;
     const uint16_t *gq = (const uint16_t *)a.q + head * a.dim, *gk = (const uint16_t *)a.k + head * a.dim, *gv = (const uint16_t *)a.v + head * a.vdim + col0;
     const int vcols = min(FKL_RC_COLS, a.vdim - col0);
-    auto fetch = [&](int c) {                           // chunk c of this run; rows past the end and padding columns are zeros
-        const uint32_t kb = sbase + (uint32_t)((c & 1) * L::STAGE), qb = kb + L::QK, vb = qb + L::QK;
+    // rows of chunk c of this run; past the end and in padding columns zeros
+    auto fetch_rows = [&](const uint16_t *g, uint32_t dst, int c) {
         const int r0 = (chunk0 + c) * FKL_CH;
         for (int i = tid; i < FKL_CH * (KD / 8); i += FKL_CH_THREADS) {
             const int r = i / (KD / 8), cc = (i - r * (KD / 8)) * 8; const bool v = r0 + r < a.rows && cc < a.dim;
-            const size_t at = (size_t)(r0 + r) * a.ld + cc;
-            cp16_zfill(kb + (uint32_t)((r * KS + cc) * 2), v ? gk + at : gk, v);
-            if (OUT) cp16_zfill(qb + (uint32_t)((r * KS + cc) * 2), v ? gq + at : gq, v);
+            cp16_zfill(dst + (uint32_t)((r * KS + cc) * 2), v ? g + (size_t)(r0 + r) * a.ld + cc : g, v);
         }
+    };
+    auto fetch_kv = [&](int c) {
+        const uint32_t kb = sbase + (uint32_t)((c & 1) * (L::K + L::V)), vb = kb + L::K;
+        const int r0 = (chunk0 + c) * FKL_CH;
+        fetch_rows(gk, kb, c);
         for (int i = tid; i < FKL_CH * (FKL_RC_COLS / 8); i += FKL_CH_THREADS) {
             const int r = i >> 3, cc = (i & 7) * 8; const bool v = r0 + r < a.rows && cc < vcols;
             cp16_zfill(vb + (uint32_t)((r * VS + cc) * 2), v ? gv + (size_t)(r0 + r) * a.ld + cc : gv, v);
         }
-        asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    fetch(0);
-    // log gates of a chunk, two positions per lane of warp 0 (requested a chunk ahead)
-    float zi[2] = {}, zf[2] = {};
-    auto gates_request = [&](int c) {
-        if (MEM && wid == 0) {
-#pragma unroll
-            for (int j = 0; j < 2; ++j) {
-                const int r = (chunk0 + c) * FKL_CH + 2 * lane + j;
-                if (r < a.rows) { zi[j] = a.logits[(size_t)r * a.ldl + head]; zf[j] = a.logits[(size_t)r * a.ldl + a.heads + head]; }
-            }
-        }
-    };
-    auto gates = [&](int c, float m0) {                 // warp 0: F, a and M of chunk c, and the weights that lead to its end
-        if (wid != 0) return;
-        const int r0 = (chunk0 + c) * FKL_CH + 2 * lane, p = c & 1;
+    fetch_kv(0);
+    if (OUT) fetch_rows(gq, qb, 0);
+    asm volatile("cp.async.commit_group;" ::: "memory");
+    auto gates = [&](int c) {                           // this warp: F, a and X of chunk c, two positions per lane
+        const int r0 = (chunk0 + c) * FKL_CH + 2 * lane, p = c % GR;
         float f[2], i2[2];
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
             const bool v = r0 + j < a.rows;
-            f[j] = v ? (MEM ? log_sigmoid_f(soft_cap_f(zf[j] + bf, a.cap)) : lgd) : 0.0f;
-            i2[j] = v ? (MEM ? soft_cap_f(zi[j] + bi, a.cap) : 0.0f) : -INFINITY;
+            if (MEM) {
+                const float zi = v ? a.logits[(size_t)(r0 + j) * a.ldl + head] : 0.0f, zf = v ? a.logits[(size_t)(r0 + j) * a.ldl + a.heads + head] : 0.0f;
+                f[j] = v ? log_sigmoid_f(soft_cap_f(zf + bf, a.cap)) : 0.0f; i2[j] = v ? soft_cap_f(zi + bi, a.cap) : -INFINITY;
+            } else { f[j] = v ? lgd : 0.0f; i2[j] = v ? 0.0f : -INFINITY; }
         }
         float F = f[0] + f[1];
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) { const float t = __shfl_up_sync(0xffffffffu, F, o); if (lane >= o) F += t; }
-        const float F1 = F, F0 = F - f[1];
-        const float a0 = i2[0] - F0, a1 = i2[1] - F1;
-        float M0 = -F0, M1 = -F1;
+        const float F0 = F - f[1], a0 = i2[0] - F0, a1 = i2[1] - F;
+        sF[p][2 * lane] = F0; sF[p][2 * lane + 1] = F; sa[p][2 * lane] = a0; sa[p][2 * lane + 1] = a1;
         if (MEM) {
             float x = fmaxf(a0, a1);
 #pragma unroll
             for (int o = 1; o < 32; o <<= 1) { const float t = __shfl_up_sync(0xffffffffu, x, o); if (lane >= o) x = fmaxf(x, t); }
-            float before = __shfl_up_sync(0xffffffffu, x, 1);
-            before = lane == 0 ? m0 : fmaxf(before, m0);
-            M0 = fmaxf(before, a0); M1 = fmaxf(M0, a1);
+            const float before = __shfl_up_sync(0xffffffffu, x, 1);
+            sX[p][2 * lane] = lane == 0 ? a0 : fmaxf(before, a0); sX[p][2 * lane + 1] = x;
         }
-        const float Fe = __shfl_sync(0xffffffffu, F1, 31), Me = __shfl_sync(0xffffffffu, M1, 31);
-        sa[p][2 * lane] = a0; sa[p][2 * lane + 1] = a1; sM[p][2 * lane] = M0; sM[p][2 * lane + 1] = M1; sF[p][2 * lane] = F0; sF[p][2 * lane + 1] = F1;
-        sw[2 * lane] = expf(a0 - Me); sw[2 * lane + 1] = expf(a1 - Me);
-        if (lane == 0) { s_end[p][0] = Fe; s_end[p][1] = Me; }
     };
-    // ---- the state before the run: tile rows (16 of dim) x columns in accumulators, and as hi + lo in shared memory
+    // ---- the state before the run: tile rows (16 of dim) x columns in accumulators; the normaliser in column 0 of a tile of its own
     const int tile0 = SHARE > 1 ? wid / SHARE : wid * MT, n0 = SHARE > 1 ? (wid % SHARE) * NT : 0;
-    float acc[MT][NT][4];
+    const uint32_t ones = g8 == 0 ? 0x3f803f80u : 0u;   // B fragment whose column 0 is 1
+    float acc[MT][NT][4], accn[MEM ? MT : 1][4];
 #pragma unroll
-    for (int i = 0; i < MT; ++i)
+    for (int i = 0; i < MT; ++i) {
 #pragma unroll
         for (int j = 0; j < NT; ++j) acc[i][j][0] = acc[i][j][1] = acc[i][j][2] = acc[i][j][3] = 0.0f;
+        if (MEM) accn[i][0] = accn[i][1] = accn[i][2] = accn[i][3] = 0.0f;
+    }
     float m0 = 0.0f;
     auto add_state = [&](const float *src, float fa, float fb) {         // acc <- fa acc + fb src, the same for n
 #pragma unroll
@@ -370,8 +379,8 @@ __global__ void __launch_bounds__(FKL_CH_THREADS) k_recurrence_chunks(FkState *s
                     const float2 v = __ldcg(reinterpret_cast<const float2 *>(src + d * FKL_RC_COLS + (n0 + j) * 8 + t4 * 2));
                     acc[i][j][2 * h] = fmaf(fa, acc[i][j][2 * h], fb * v.x); acc[i][j][2 * h + 1] = fmaf(fa, acc[i][j][2 * h + 1], fb * v.y);
                 }
+                if (MEM && t4 == 0) accn[i][2 * h] = fmaf(fa, accn[i][2 * h], fb * __ldcg(src + a.dim * FKL_RC_COLS + d));
             }
-        if (MEM) for (int d = tid; d < a.dim; d += FKL_CH_THREADS) sn[d] = fmaf(fa, sn[d], fb * __ldcg(src + a.dim * FKL_RC_COLS + d));
     };
     auto put_state = [&](float *dst, float m) {
 #pragma unroll
@@ -382,10 +391,10 @@ __global__ void __launch_bounds__(FKL_CH_THREADS) k_recurrence_chunks(FkState *s
                 if (d >= a.dim) continue;
 #pragma unroll
                 for (int j = 0; j < NT; ++j) *reinterpret_cast<float2 *>(dst + d * FKL_RC_COLS + (n0 + j) * 8 + t4 * 2) = make_float2(acc[i][j][2 * h], acc[i][j][2 * h + 1]);
+                if (MEM && n0 == 0 && t4 == 0) dst[a.dim * FKL_RC_COLS + d] = accn[i][2 * h];
             }
-        if (MEM) { for (int d = tid; d < a.dim; d += FKL_CH_THREADS) dst[a.dim * FKL_RC_COLS + d] = sn[d]; if (tid == 0) dst[a.dim * FKL_RC_COLS + a.dim] = m; }
+        if (MEM && tid == 0) dst[a.dim * FKL_RC_COLS + a.dim] = m;
     };
-    if (MEM) for (int d = tid; d < KD; d += FKL_CH_THREADS) sn[d] = 0.0f;
     // scratch: [runs + 1][cells][sstride], entry 0 the stored state, entry r + 1 what run r leaves (run 0: from the stored state); then
     // [runs][cells] sums of log keeps
     float *fsum = a.seg + (size_t)(a.segments + 1) * cells * a.sstride;
@@ -413,51 +422,49 @@ __global__ void __launch_bounds__(FKL_CH_THREADS) k_recurrence_chunks(FkState *s
             add_state(seg(r + 1), fa, fb);
         }
     }
-    gates_request(0);
     float Ftotal = 0.0f;
     for (int c = 0; c < nchunk; ++c) {
-        const int p = c & 1;
-        gates(c, m0);
-        gates_request(c + 1);
-        if (c + 1 < nchunk) { fetch(c + 1); asm volatile("cp.async.wait_group 1;" ::: "memory"); }
-        else asm volatile("cp.async.wait_group 0;" ::: "memory");
+        const int p = c % GR;
+        if (p == 0) {
+            if (c > 0) __syncthreads();                 // the last chunks' gates have been read
+            if (wid < GR && c + wid < nchunk) gates(c + wid);
+        }
         if (OUT) {                                      // the state before this chunk as hi + lo
 #pragma unroll
             for (int i = 0; i < MT; ++i)
 #pragma unroll
-                for (int h = 0; h < 2; ++h)
+                for (int h = 0; h < 2; ++h) {
+                    const uint32_t row = (uint32_t)(((tile0 + i) * 16 + g8 + h * 8) * VS * 2);
+                    uint32_t hi, lo;
 #pragma unroll
                     for (int j = 0; j < NT; ++j) {
-                        uint32_t hi, lo; ch_split(acc[i][j][2 * h], acc[i][j][2 * h + 1], hi, lo);
-                        const uint32_t at = (uint32_t)((((tile0 + i) * 16 + g8 + h * 8) * VS + (n0 + j) * 8 + t4 * 2) * 2);
+                        ch_split(acc[i][j][2 * h], acc[i][j][2 * h + 1], hi, lo);
+                        const uint32_t at = row + (uint32_t)(((n0 + j) * 8 + t4 * 2) * 2);
                         asm volatile("st.shared.b32 [%0], %1;" ::"r"(shi + at), "r"(hi) : "memory");
                         asm volatile("st.shared.b32 [%0], %1;" ::"r"(slo + at), "r"(lo) : "memory");
                     }
-        }
-        __syncthreads();
-        const uint32_t kb = sbase + (uint32_t)(p * L::STAGE), qb = kb + L::QK, vb = qb + L::QK;
-        const float Fe = s_end[p][0], Me = s_end[p][1];
-        if (OUT) {
-            if (MEM) {                                  // n . q of every position: four threads each
-                const int r = tid >> 2, q4 = tid & 3; const uint16_t *qr = reinterpret_cast<const uint16_t *>(ch_smem + p * L::STAGE + L::QK) + r * KS;
-                float d = 0.0f;
-#pragma unroll 4
-                for (int i = q4 * 8; i < KD; i += 32) {
-                    float f[8]; unpack8f(*reinterpret_cast<const uint4 *>(qr + i), f);
-#pragma unroll
-                    for (int j = 0; j < 8; ++j) d = fmaf(f[j], sn[i + j], d);
+                    if (MEM && n0 == 0) {               // columns 64 .. 71 (row padding): the normaliser and zeros
+                        ch_split(accn[i][2 * h], 0.0f, hi, lo);
+                        const uint32_t at = row + (uint32_t)((FKL_RC_COLS + t4 * 2) * 2);
+                        asm volatile("st.shared.b32 [%0], %1;" ::"r"(shi + at), "r"(hi) : "memory");
+                        asm volatile("st.shared.b32 [%0], %1;" ::"r"(slo + at), "r"(lo) : "memory");
+                    }
                 }
-                d += __shfl_xor_sync(0xffffffffu, d, 1); d += __shfl_xor_sync(0xffffffffu, d, 2);
-                if (q4 == 0) sden[r] = d;
-                __syncthreads();
-            }
-            const int wr = wid & 3, hc = wid >> 2, row0 = wr * 16;      // 16 positions x 32 columns of this warp
-            float s[8][4], o[4][4];
+        }
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+        if (c + 1 < nchunk) { fetch_kv(c + 1); asm volatile("cp.async.commit_group;" ::: "memory"); }      // its stage was read a chunk ago
+        const uint32_t kb = sbase + (uint32_t)((c & 1) * (L::K + L::V)), vb = kb + L::K;
+        const float Fe = sF[p][FKL_CH - 1], Me = MEM ? fmaxf(m0, sX[p][FKL_CH - 1]) : -Fe;
+        if (OUT) {
+            // 16 positions x 32 columns of this warp; later positions have more to do, so the two warps of a scheduler take opposite ends
+            const int hc = wid >> 2, wr = hc ? 3 - (wid & 3) : wid & 3, row0 = wr * 16;
+            float s[8][4], o[4][4], nd[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
             for (int i = 0; i < 8; ++i) s[i][0] = s[i][1] = s[i][2] = s[i][3] = 0.0f;
 #pragma unroll
             for (int i = 0; i < 4; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
-#pragma unroll 4
+#pragma unroll 2
             for (int k = 0; k < KD / 16; ++k) {
                 uint32_t q[4], b[4];
                 ch_ldsm(q, qb + (uint32_t)(((row0 + (lane & 15)) * KS + k * 16 + (lane >> 4) * 8) * 2));
@@ -472,9 +479,13 @@ __global__ void __launch_bounds__(FKL_CH_THREADS) k_recurrence_chunks(FkState *s
                     ch_ldsm_t(b, shi + at); ch_mma(o[2 * n], q, b[0], b[1]); ch_mma(o[2 * n + 1], q, b[2], b[3]);
                     ch_ldsm_t(b, slo + at); ch_mma(o[2 * n], q, b[0], b[1]); ch_mma(o[2 * n + 1], q, b[2], b[3]);
                 }
+                if (MEM) {                              // n . q: hi in the first two matrices, lo in the others
+                    const uint32_t at = (uint32_t)(((k * 16 + (lane & 15)) * VS + FKL_RC_COLS) * 2);
+                    ch_ldsm_t(b, (lane < 16 ? shi : slo) + at); ch_mma(nd, q, b[0], b[1]); ch_mma(nd, q, b[2], b[3]);
+                }
             }
             const int ra = row0 + g8, rb = ra + 8;
-            const float Ma = sM[p][ra], Mb = sM[p][rb], fa = expf(m0 - Ma) * a.qscale, fb = expf(m0 - Mb) * a.qscale;
+            const float Ma = MEM ? fmaxf(m0, sX[p][ra]) : -sF[p][ra], Mb = MEM ? fmaxf(m0, sX[p][rb]) : -sF[p][rb], fa = expf(m0 - Ma) * a.qscale, fb = expf(m0 - Mb) * a.qscale;
 #pragma unroll
             for (int i = 0; i < 4; ++i) { o[i][0] *= fa; o[i][1] *= fa; o[i][2] *= fb; o[i][3] *= fb; }
             float da = 0.0f, db = 0.0f;
@@ -498,11 +509,13 @@ __global__ void __launch_bounds__(FKL_CH_THREADS) k_recurrence_chunks(FkState *s
                     ch_mma(o[2 * v], pl, b[0], b[1]); ch_mma(o[2 * v + 1], pl, b[2], b[3]);
                 }
             }
+            __syncthreads();                            // q and the shared copy of the state have been read
+            if (c + 1 < nchunk) { fetch_rows(gq, qb, c + 1); asm volatile("cp.async.commit_group;" ::: "memory"); }
             float na = 1.0f, nb = 1.0f;
             if (MEM) {
                 da += __shfl_xor_sync(0xffffffffu, da, 1); da += __shfl_xor_sync(0xffffffffu, da, 2);
                 db += __shfl_xor_sync(0xffffffffu, db, 1); db += __shfl_xor_sync(0xffffffffu, db, 2);
-                da = fmaf(fa, sden[ra], da); db = fmaf(fb, sden[rb], db);
+                da = fmaf(fa, __shfl_sync(0xffffffffu, nd[0], lane & 28), da); db = fmaf(fb, __shfl_sync(0xffffffffu, nd[2], lane & 28), db);
                 na = 1.0f / (fmaxf(fabsf(da), expf(-(sF[p][ra] + Ma))) + 1e-6f); nb = 1.0f / (fmaxf(fabsf(db), expf(-(sF[p][rb] + Mb))) + 1e-6f);
             }
             const int r0 = (chunk0 + c) * FKL_CH;
@@ -518,9 +531,11 @@ __global__ void __launch_bounds__(FKL_CH_THREADS) k_recurrence_chunks(FkState *s
         // ---- the state after the chunk
         const float decay = expf(m0 - Me);
 #pragma unroll
-        for (int i = 0; i < MT; ++i)
+        for (int i = 0; i < MT; ++i) {
 #pragma unroll
             for (int j = 0; j < NT; ++j) { acc[i][j][0] *= decay; acc[i][j][1] *= decay; acc[i][j][2] *= decay; acc[i][j][3] *= decay; }
+            if (MEM) { accn[i][0] *= decay; accn[i][2] *= decay; }
+        }
 #pragma unroll
         for (int k = 0; k < 4; ++k) {                   // 16 positions
             uint32_t b[NT][2];
@@ -530,7 +545,8 @@ __global__ void __launch_bounds__(FKL_CH_THREADS) k_recurrence_chunks(FkState *s
                 ch_ldsm_t(r, vb + (uint32_t)(((k * 16 + (lane & 15)) * VS + (n0 + j) * 8 + (lane >> 4) * 8) * 2));
                 b[j][0] = r[0]; b[j][1] = r[1]; b[j + 1][0] = r[2]; b[j + 1][1] = r[3];
             }
-            const float w0 = sw[k * 16 + t4 * 2], w1 = sw[k * 16 + t4 * 2 + 1], w2 = sw[k * 16 + t4 * 2 + 8], w3 = sw[k * 16 + t4 * 2 + 9];
+            const float *ak = sa[p] + k * 16 + t4 * 2;
+            const float w0 = expf(ak[0] - Me), w1 = expf(ak[1] - Me), w2 = expf(ak[8] - Me), w3 = expf(ak[9] - Me);
 #pragma unroll
             for (int i = 0; i < MT; ++i) {
                 uint32_t x[4], hi[4], lo[4];
@@ -539,21 +555,11 @@ __global__ void __launch_bounds__(FKL_CH_THREADS) k_recurrence_chunks(FkState *s
                 ch_split(bf_lo(x[2]) * w2, bf_hi(x[2]) * w3, hi[2], lo[2]); ch_split(bf_lo(x[3]) * w2, bf_hi(x[3]) * w3, hi[3], lo[3]);
 #pragma unroll
                 for (int j = 0; j < NT; ++j) { ch_mma(acc[i][j], hi, b[j][0], b[j][1]); ch_mma(acc[i][j], lo, b[j][0], b[j][1]); }
+                if (MEM) { ch_mma(accn[i], hi, ones, ones); ch_mma(accn[i], lo, ones, ones); }
             }
         }
-        if (MEM) {
-            if (OUT) __syncthreads();                   // n has been read
-            for (int d = tid; d < KD; d += FKL_CH_THREADS) {
-                const uint16_t *kc = reinterpret_cast<const uint16_t *>(ch_smem + p * L::STAGE) + d;
-                float v = decay * sn[d];
-#pragma unroll 8
-                for (int r = 0; r < FKL_CH; ++r) v = fmaf(sw[r], bf2f(kc[r * KS]), v);
-                sn[d] = v;
-            }
-            m0 = Fe + Me;
-        }
+        if (MEM) m0 = Fe + Me;
         Ftotal += Fe;
-        __syncthreads();                                // the stage, the gate arrays and the shared copy of the state are free
     }
     if (a.segments == 1) put_state(S, m0);
     else if (!OUT) { put_state(seg(run + 1), m0); if (tid == 0) fsum[(size_t)run * cells + cell] = Ftotal; }

@@ -52,7 +52,7 @@ __device__ __forceinline__ Visible visible_keys(int pos, int window, int keep) {
 // dimension i of a head after rotation by a position's table row (cos, sin of pair 0, of pair 1, ..); v: the value, other: its pair's
 __device__ __forceinline__ float rotate_dim(float v, float other, int i, int dims, const float *row) {
     if (i >= dims) return v;
-    const float2 cs = __ldg(reinterpret_cast<const float2 *>(row) + (i >> 1));
+    const float2 cs = reinterpret_cast<const float2 *>(row)[i >> 1];
     return (i & 1) ? fmaf(v, cs.x, other * cs.y) : fmaf(v, cs.x, -(other * cs.y));
 }
 __device__ __forceinline__ void unpack8f(uint4 v, float (&f)[8]) {

@@ -405,6 +405,7 @@ __global__ void __launch_bounds__(FKL_ATT_WARPS * 32) k_attention(FkState *st, A
 // block of a (kv head, row tile) folds them, combines the maps and applies the gate.
 #define FKL_AD_KEYS 64
 #define FKL_AD_THREADS 256
+#define FKL_AD_ROT 256               // rotated dimensions whose table row fits in shared memory
 struct AdLayout { int ks, vs, stage, q, sc, pr, nk, nv, of, total; };      // byte offsets; ks / vs: row strides in elements
 __host__ __device__ inline AdLayout ad_layout(int maps, int dpad, int vpad) {
     AdLayout l; l.ks = ((dpad / 8) | 1) * 8; l.vs = ((vpad / 8) | 1) * 8;           // odd multiples of 16 bytes
@@ -423,7 +424,7 @@ __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st
     float *qs = reinterpret_cast<float *>(ad_smem + L.q), *sc = reinterpret_cast<float *>(ad_smem + L.sc), *pr = reinterpret_cast<float *>(ad_smem + L.pr);
     uint16_t *nk = reinterpret_cast<uint16_t *>(ad_smem + L.nk), *nv = reinterpret_cast<uint16_t *>(ad_smem + L.nv);
     float *of = reinterpret_cast<float *>(ad_smem + L.of);
-    __shared__ float s_corr[RT], s_m[RT], s_l[RT], s_fac[256 * RT], s_red[66]; __shared__ int s_last;
+    __shared__ float s_corr[RT], s_m[RT], s_l[RT], s_fac[256 * RT], s_red[66], s_rot[FKL_AD_ROT]; __shared__ int s_last;
     const int tid = threadIdx.x, lane = tid & 31, wid = tid >> 5;
     const int g = blockIdx.y / a.tiles, tile = blockIdx.y - g * a.tiles, group = a.H / a.G, nrow_kv = group * a.maps, r0 = tile * RT, nr = min(RT, nrow_kv - r0);
     const uint32_t upos = st->offset;                   // advanced by the head of the token before, long since finished
@@ -447,49 +448,76 @@ __global__ void __launch_bounds__(FKL_AD_THREADS) k_attention_decode(FkState *st
         }
     };
     if (fits) for (int c = 0; c < 2; ++c) { if (c < nchunk) request(c); asm volatile("cp.async.commit_group;" ::: "memory"); }
+    // what else does not depend on the kernel before: rows without a query, the position's rotation, the norm weights of the warp's first item
+    const bool mine = newest >= k0 && newest < k1;
+    const int items = nr + (mine ? a.maps + 1 : 0);     // query rows, new keys, new value
+    auto weight_of = [&](int it) { const bool is_q = it < nr; return (is_q ? a.qn : a.kn) + (a.joint ? (is_q ? g * nrow_kv + r0 + it : g) * a.dim : 0); };
+    auto source_of = [&](int it) { return a.qkv + (it < nr ? (g * nrow_kv + r0 + it) : (a.H * a.maps + g * a.maps + (it - nr))) * a.dim; };
+    float xv[4], wv[4];                                 // the first 128 values of the warp's item
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { const int i = lane + j * 32; wv[j] = wid < items && wid != nr + a.maps && i < a.dim ? bf2f(weight_of(wid)[i]) : 0.0f; }
+    for (int i = tid; i < (RT - nr) * a.dpad; i += NT) qs[nr * a.dpad + i] = 0.0f;
+    const float *rot = a.rot && fits ? a.rot + (size_t)pos * a.rot_dims : nullptr;
+    if (rot && a.rot_dims <= FKL_AD_ROT) { for (int i = tid; i < a.rot_dims; i += NT) s_rot[i] = rot[i]; rot = s_rot; __syncthreads(); }
     pdl_wait(); pdl_launch_dependents();
     if (!fits) { if (tid == 0) atomicOr(&st->error, FKL_ERR_CAPACITY); return; }
     if (nchunk == 0) return;                            // more splits than this many keys need
     // ---- query rows, and where the position falls here the new key and value
-    const bool mine = newest >= k0 && newest < k1;
+#pragma unroll
+    for (int j = 0; j < 4; ++j) { const int i = lane + j * 32; xv[j] = wid < items && wid != nr + a.maps && i < a.dim ? __ldcg(source_of(wid) + i) : 0.0f; }
     float2 joint = make_float2(0.0f, 0.0f);
     if (a.joint) {
+        const int nq = a.H * a.dim, nk = a.G * a.dim;
         float sq = 0.0f, sk = 0.0f;
-        for (int i = tid; i < a.H * a.dim; i += NT) { const float v = __ldcg(a.qkv + i); sq = fmaf(v, v, sq); }
-        for (int i = tid; i < a.G * a.dim; i += NT) { const float v = __ldcg(a.qkv + a.H * a.dim + i); sk = fmaf(v, v, sk); }
+        if ((((uintptr_t)a.qkv | (uintptr_t)(a.qkv + nq)) & 15) == 0 && (nq & 3) == 0 && (nk & 3) == 0) {
+            const float4 *p = reinterpret_cast<const float4 *>(a.qkv);
+            for (int b = tid; b < (nq + nk) / 4; b += 4 * NT) {
+                float4 v[4];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) v[j] = b + j * NT < (nq + nk) / 4 ? __ldcg(p + b + j * NT) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float e = fmaf(v[j].x, v[j].x, fmaf(v[j].y, v[j].y, fmaf(v[j].z, v[j].z, v[j].w * v[j].w)));
+                    if (b + j * NT < nq / 4) sq += e; else sk += e;
+                }
+            }
+        } else {
+            for (int i = tid; i < nq; i += NT) { const float v = __ldcg(a.qkv + i); sq = fmaf(v, v, sq); }
+            for (int i = tid; i < nk; i += NT) { const float v = __ldcg(a.qkv + nq + i); sk = fmaf(v, v, sk); }
+        }
         joint = block_sum2(sq, sk, s_red);
-        joint = make_float2(inv_rms(joint.x, a.H * a.dim, a.eps), inv_rms(joint.y, a.G * a.dim, a.eps));
+        joint = make_float2(inv_rms(joint.x, nq, a.eps), inv_rms(joint.y, nk, a.eps));
     }
-    const float *rot = a.rot ? a.rot + (size_t)pos * a.rot_dims : nullptr;
-    for (int it = wid; it < RT + (mine ? a.maps + 1 : 0); it += NT / 32) {
-        if (it >= nr && it < RT) { for (int i = lane; i < a.dpad; i += 32) qs[it * a.dpad + i] = 0.0f; continue; }
-        if (it == RT + a.maps) {
+    for (int it = wid; it < items; it += NT / 32) {
+        if (it == nr + a.maps) {
             const float *src = a.qkv + (a.H + a.G) * a.maps * a.dim + g * a.vdim;
             for (int i = lane; i < a.vpad; i += 32) { const uint16_t v = i < a.vdim ? f2bf(__ldcg(src + i)) : (uint16_t)0; nv[i] = v; if (i < a.vdim) cv[(size_t)pos * a.vpad + i] = v; }
             continue;
         }
-        const bool is_q = it < RT;
-        const float *src = a.qkv + (is_q ? (g * nrow_kv + r0 + it) : (a.H * a.maps + g * a.maps + (it - RT))) * a.dim;
-        const uint16_t *w = (is_q ? a.qn : a.kn) + (a.joint ? (is_q ? g * nrow_kv + r0 + it : g) * a.dim : 0);
-        float ss = 0.0f, xv[4], wv[4];                  // the first 128 values stay in registers
+        const bool is_q = it < nr;
+        const float *src = source_of(it);
+        const uint16_t *w = weight_of(it);
+        if (it != wid) {
 #pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const int i = lane + j * 32;
-            xv[j] = i < a.dim ? __ldcg(src + i) : 0.0f; wv[j] = i < a.dim ? bf2f(w[i]) : 0.0f;
+            for (int j = 0; j < 4; ++j) { const int i = lane + j * 32; xv[j] = i < a.dim ? __ldcg(src + i) : 0.0f; wv[j] = i < a.dim ? bf2f(w[i]) : 0.0f; }
         }
+        float r = is_q ? joint.x : joint.y;
+        if (!a.joint) {
+            float ss = 0.0f;
 #pragma unroll
-        for (int j = 0; j < 4; ++j) ss = fmaf(xv[j], xv[j], ss);
-        for (int i = lane + 128; i < a.dim; i += 32) { const float v = __ldcg(src + i); ss = fmaf(v, v, ss); }
-        const float r = a.joint ? (is_q ? joint.x : joint.y) : inv_rms(warp_sum(ss), a.dim, a.eps);
-#pragma unroll 4
-        for (int j = 0; j * 32 < a.dpad; ++j) {
-            const int i = lane + j * 32;
-            float v = j < 4 ? xv[j & 3] * r * wv[j & 3] : i < a.dim ? __ldcg(src + i) * r * bf2f(w[i]) : 0.0f;
+            for (int j = 0; j < 4; ++j) ss = fmaf(xv[j], xv[j], ss);
+            for (int i = lane + 128; i < a.dim; i += 32) { const float v = __ldcg(src + i); ss = fmaf(v, v, ss); }
+            r = inv_rms(warp_sum(ss), a.dim, a.eps);
+        }
+        auto put = [&](int i, float v) {
             if (rot) v = rotate_dim(v, __shfl_xor_sync(0xffffffffu, v, 1), i, a.rot_dims, rot);
-            if (i >= a.dpad) continue;
+            if (i >= a.dpad) return;
             if (is_q) qs[it * a.dpad + i] = v * a.scale;
-            else { nk[(it - RT) * a.dpad + i] = f2bf(v); if (i < a.dim) ck[((size_t)(it - RT) * a.cap + pos) * a.dpad + i] = f2bf(v); }
-        }
+            else { nk[(it - nr) * a.dpad + i] = f2bf(v); if (i < a.dim) ck[((size_t)(it - nr) * a.cap + pos) * a.dpad + i] = f2bf(v); }
+        };
+#pragma unroll
+        for (int j = 0; j < 4; ++j) if (j * 32 < a.dpad) put(lane + j * 32, xv[j] * r * wv[j]);
+        for (int i = lane + 128; i - lane < a.dpad; i += 32) put(i, i < a.dim ? __ldcg(src + i) * r * bf2f(w[i]) : 0.0f);
     }
     // ---- chunks
     int tpc = 1; while (tpc < NT && tpc < a.vpad / 2) tpc <<= 1;        // threads over pairs of value columns
