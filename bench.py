@@ -455,6 +455,7 @@ def run_parallel(args, local, name, spec, frac, chunks, peak, flops_peak, peak_k
     rt.state_set(3, ctx)
 
     def add(key, tasks, nbytes, flops=0.0, e=None, table=None):
+        time.sleep(0.3)          # each kernel by itself and from a rested chip: a long run of products lowers the clocks (power cap)
         secs = (e or eng).time_tasks(tasks, 5) / len(tasks)
         (kern if table is None else table)[key] = {"us": secs * 1e6, "frac": frac(secs, nbytes, flops), "bytes": nbytes, "flops": flops}
 

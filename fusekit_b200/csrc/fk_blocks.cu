@@ -57,7 +57,7 @@ fk_status fkb_run(FklEnv &c, const fk_task &t, char *err, size_t ecap) {
             const int nv = a.d <= 2048 ? 1 : 2;
             const dim3 blk(round_up((a.d / 4 + nv - 1) / nv, 32));
 #define BN(T, NV, NT, BLOCKS) launch(c, (k_block_norm_rows4<T, NV, NT, BLOCKS>), g, blk, 0, st, a)
-            if (i[2]) e = a.d <= 2048 ? BN(float, 1, 512, 2) : a.d <= 4096 ? BN(float, 2, 512, 2) : BN(float, 2, 1024, 1);
+            if (i[2]) e = a.d <= 2048 ? BN(float, 1, 512, 2) : a.d <= 4096 ? BN(float, 2, 512, 1) : BN(float, 2, 1024, 1);
             else e = a.d <= 2048 ? BN(uint16_t, 1, 512, 3) : a.d <= 4096 ? BN(uint16_t, 2, 512, 2) : a.d <= 5120 ? BN(uint16_t, 2, 640, 2) : BN(uint16_t, 2, 1024, 1);
 #undef BN
             break;

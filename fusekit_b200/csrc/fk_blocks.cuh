@@ -27,60 +27,80 @@ template <> struct Raw4<float> {
     __device__ __forceinline__ void zero() { v = make_float4(0.0f, 0.0f, 0.0f, 0.0f); }
     __device__ __forceinline__ float4 get() const { return v; }
 };
-// rows of a multiple of 4 and at most NV * 4 * blockDim.x values: everything in registers, one round of loads
+// sums over a block of up to 32 warps with one barrier: every warp adds up all warps' parts.  Each call of a kernel has buffers of its own.
+template <int N> __device__ __forceinline__ void block_sums(float (&v)[N], float (*buf)[32]) {
+    const int lane = threadIdx.x & 31, wid = threadIdx.x >> 5, nw = blockDim.x >> 5;
+#pragma unroll
+    for (int i = 0; i < N; ++i) { v[i] = warp_sum(v[i]); if (lane == 0) buf[i][wid] = v[i]; }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < N; ++i) v[i] = warp_sum(lane < nw ? buf[i][lane] : 0.0f);
+}
+__device__ __forceinline__ float4 bf4(uint2 v) { return make_float4(bf_lo(v.x), bf_hi(v.x), bf_lo(v.y), bf_hi(v.y)); }
+// rows of a multiple of 4 and at most NV * 4 * blockDim.x values: everything in registers, one round of loads, weights ahead of the sums
 template <typename T, int NV, int NT, int BLOCKS>
 __global__ void __launch_bounds__(NT, BLOCKS) k_block_norm_rows4(const FkState *st, BlockNormArgs a) {
-    __shared__ float red[66];
+    __shared__ float red[5][32];
     const int tid = threadIdx.x, nt = blockDim.x;
     pdl_wait(); pdl_launch_dependents();
     const size_t row = a.index ? a.index[blockIdx.x] : blockIdx.x;
     float4 x[NV];
     Raw4<T> y[3][NV];
+    uint2 w0[NV], w1[NV];                               // post weights, then the norm's weights
 #pragma unroll
     for (int v = 0; v < NV; ++v) {
         const int i = (v * nt + tid) * 4;
         x[v] = i < a.d ? ld4(a.x + row * a.d + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
 #pragma unroll
         for (int p = 0; p < 3; ++p) { if (p < a.np && i < a.d) y[p][v].load((const T *)a.y[p] + row * a.ldy + i); else y[p][v].zero(); }
+        w0[v] = a.nnorm > 0 && i < a.d ? __ldg(reinterpret_cast<const uint2 *>(a.post + i)) : make_uint2(0, 0);
+        w1[v] = a.nnorm > 1 && i < a.d ? __ldg(reinterpret_cast<const uint2 *>(a.post + a.d + i)) : make_uint2(0, 0);
     }
-    float f[3] = {1.0f, 1.0f, 1.0f};
     if (a.nnorm > 0) {
-        float ss[3] = {};
+        float f[3] = {};
 #pragma unroll
         for (int p = 0; p < 3; ++p)
 #pragma unroll
-            for (int v = 0; v < NV; ++v) { const float4 e = y[p][v].get(); ss[p] = fmaf(e.x, e.x, fmaf(e.y, e.y, fmaf(e.z, e.z, fmaf(e.w, e.w, ss[p])))); }
-        const float2 s01 = block_sum2(ss[0], ss[1], red);
-        f[0] = a.scale * inv_rms(s01.x, a.d, a.eps);
-        if (a.nnorm > 1) f[1] = a.scale * inv_rms(s01.y, a.d, a.eps);
-        if (a.nnorm > 2) f[2] = a.scale * inv_rms(block_sum(ss[2], red), a.d, a.eps);
+            for (int v = 0; v < NV; ++v) { const float4 e = y[p][v].get(); f[p] = fmaf(e.x, e.x, fmaf(e.y, e.y, fmaf(e.z, e.z, fmaf(e.w, e.w, f[p])))); }
+        block_sums(f, red);
+#pragma unroll
+        for (int p = 0; p < 3; ++p) {
+            const float s = a.scale * inv_rms(f[p], a.d, a.eps);
+#pragma unroll
+            for (int v = 0; v < NV; ++v) {
+                const int i = (v * nt + tid) * 4;
+                if (p >= a.nnorm || i >= a.d) continue;
+                const float4 e = y[p][v].get(), w = p == 0 ? bf4(w0[v]) : p == 1 ? bf4(w1[v]) : ld4(a.post + (size_t)2 * a.d + i);
+                x[v].x = fmaf(e.x * s, w.x, x[v].x); x[v].y = fmaf(e.y * s, w.y, x[v].y); x[v].z = fmaf(e.z * s, w.z, x[v].z); x[v].w = fmaf(e.w * s, w.w, x[v].w);
+            }
+        }
     }
-    float sum = 0.0f;
+    float sum[1] = {0.0f};
 #pragma unroll
     for (int v = 0; v < NV; ++v) {
         const int i = (v * nt + tid) * 4;
 #pragma unroll
-        for (int p = 0; p < 3; ++p) if (p < a.np && i < a.d) {
-            const float4 w = p < a.nnorm ? ld4(a.post + (size_t)p * a.d + i) : make_float4(1.0f, 1.0f, 1.0f, 1.0f), e = y[p][v].get();
-            x[v].x = fmaf(e.x * f[p], w.x, x[v].x); x[v].y = fmaf(e.y * f[p], w.y, x[v].y);
-            x[v].z = fmaf(e.z * f[p], w.z, x[v].z); x[v].w = fmaf(e.w * f[p], w.w, x[v].w);
-        }
-        sum += (x[v].x + x[v].y) + (x[v].z + x[v].w);
+        for (int p = 0; p < 3; ++p) if (p >= a.nnorm && p < a.np) { const float4 e = y[p][v].get(); x[v].x += e.x; x[v].y += e.y; x[v].z += e.z; x[v].w += e.w; }
+        sum[0] += (x[v].x + x[v].y) + (x[v].z + x[v].w);
+        if (a.x_out && i < a.d) st4(a.x_out + row * a.d + i, x[v]);
+        w0[v] = i < a.d ? __ldg(reinterpret_cast<const uint2 *>(a.w + i)) : make_uint2(0, 0);
+        w1[v] = a.b && i < a.d ? __ldg(reinterpret_cast<const uint2 *>(a.b + i)) : make_uint2(0, 0);
     }
-    const float mean = a.b ? block_sum(sum, red) / (float)a.d : 0.0f;
-    float ss = 0.0f;
+    float mean = 0.0f;
+    if (a.b) { block_sums(sum, red + 3); mean = sum[0] / (float)a.d; }
+    float ss[1] = {0.0f};
 #pragma unroll
     for (int v = 0; v < NV; ++v) if ((v * nt + tid) * 4 < a.d) {
         const float d0 = x[v].x - mean, d1 = x[v].y - mean, d2 = x[v].z - mean, d3 = x[v].w - mean;
-        ss = fmaf(d0, d0, fmaf(d1, d1, fmaf(d2, d2, fmaf(d3, d3, ss))));
+        ss[0] = fmaf(d0, d0, fmaf(d1, d1, fmaf(d2, d2, fmaf(d3, d3, ss[0]))));
     }
-    const float r = inv_rms(block_sum(ss, red), a.d, a.eps);
+    block_sums(ss, red + 4);
+    const float r = inv_rms(ss[0], a.d, a.eps);
 #pragma unroll
     for (int v = 0; v < NV; ++v) {
         const int i = (v * nt + tid) * 4;
         if (i >= a.d) continue;
-        if (a.x_out) st4(a.x_out + row * a.d + i, x[v]);
-        const float4 w = ld4(a.w + i), b = a.b ? ld4(a.b + i) : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        const float4 w = bf4(w0[v]), b = bf4(w1[v]);
         st4((T *)a.h + (size_t)blockIdx.x * a.ldh + i, make_float4(fmaf((x[v].x - mean) * r, w.x, b.x), fmaf((x[v].y - mean) * r, w.y, b.y),
                                                                    fmaf((x[v].z - mean) * r, w.z, b.z), fmaf((x[v].w - mean) * r, w.w, b.w)));
     }

@@ -113,7 +113,7 @@ class AttentionSpec:
     """Softmax attention with RMS-normed queries and keys.  ``diff`` set: differential attention -- every head has two query/key
     maps over the same values, combined as a1 - lambda a2.  ``norm``: "head" (every (sub-)head by itself, one weight of size dim)
     or "projection" (all rows at once, a weight for every row).  ``gate``: a sigmoid output gate per head.  ``window`` set:
-    position i sees j <= i with i - j < window or j < keep_first."""
+    a position sees the newest ``window`` positions up to itself and the first ``keep_first`` of the sequence."""
     heads: int
     kv_heads: int
     dim: int                  # query/key size of a map

@@ -208,8 +208,8 @@ enum { FK_ACT_NONE = 0, FK_ACT_RELU_SQUARED = 2, FK_ACT_SILU = 3 };
  * ROTARY_STORE_ROWS    buf0 q|k|v rows A[M,ld]  buf1 q norm T[H*dim]  buf2 k norm T[G*dim] (all rows normed together)  buf3 q out A[M,H,dpad]  buf4
  *                      cache k  buf5 cache v  buf6 rotation table f32[capacity][i5 / 2][cos, sin]|0   i0 H | G << 16  i1 dim | vdim << 16
  *                      i2 capacity  i3 M  i4 ld  i5 rotated dimensions  i6 dtype   f0 eps
- * WINDOW_ATTENTION_ROWS  buf0 q  buf1 cache k  buf2 cache v  buf3 out A[M, round64(H*vdim)]   i0, i1, i2, i3 as above  i4 dtype  i5 window (0: none;
- *                      position i sees j <= i with i - j < window or j < keep)  i6 keep   f0 scale
+ * WINDOW_ATTENTION_ROWS  buf0 q  buf1 cache k  buf2 cache v  buf3 out A[M, round64(H*vdim)]   i0, i1, i2, i3 as above  i4 dtype  i5 window (0: none; else the
+ *                      newest i5 positions and the first i6 are seen)  i6 keep   f0 scale
  * WINDOW_ATTENTION_DECODE  one position: joint q/k norm, rotation, cache store, attention.  buf0 q|k|v f32  buf1 q norm  buf2 k norm  buf3 cache k
  *                      buf4 cache v  buf5 out f32[H*vdim]  buf6 partials  buf7 counters (as ATTENTION_DECODE)  buf8 rotation table|0
  *                      i0 H | G << 16  i1 dim | vdim << 16  i2 capacity  i3 dtype of the caches  i4 key splits  i5 window  i6 keep

@@ -179,7 +179,7 @@ def rotate_pairs(x, positions, freqs):
 
 
 def window_attention(q, k, v, scale, pos0, window=None, keep_first=0):
-    """One head, as softmax_attention, where position i sees j <= i with i - j < window or j < keep_first."""
+    """One head, as softmax_attention over the newest ``window`` positions up to the query and the first ``keep_first`` of all."""
     out = np.zeros((q.shape[0], v.shape[1]), q.dtype)
     for i in range(q.shape[0]):
         p = pos0 + i

@@ -141,6 +141,7 @@ PARALLEL_SPECS = {
                                 LayerSpec(MM(3, 14, 18, 11.0), G(21, 0.9)), LayerSpec(MM(2, 5, 7, 6.0), None)], hidden=75, vocab=99, eps=1e-3, logit_scale=0.4),
     "wide-heads": parallel_spec([LayerSpec(P(windowed(12, 1, 136, 200, 0.1, 40, 10, 136), L(1, 264, 130, (0.9,))), G(48, 4.0)),
                                  LayerSpec(MM(1, 200, 72, 15.0), G(33, 2.0))], hidden=64, vocab=80),
+    "memory-only": parallel_spec([LayerSpec(MM(2, 12, 20, 6.0), None)], hidden=36, vocab=50),
     "one-layer": parallel_spec([LayerSpec(P(windowed(1, 1, 8, 8, 0.6, 4, 2, 8), L(1, 8, 8, (0.9,))), G(8, 1.0))], hidden=16, vocab=33, logit_scale=3.0),
 }
 
